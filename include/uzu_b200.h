@@ -481,7 +481,7 @@ typedef struct uzu_dense_linear_args {
                                       min(g, limit) * sigmoid(alpha * min(g, limit)) * (clamp(u, -limit, limit) + 1) */
     float glu_limit, glu_alpha;
     uint32_t glu_kind;             /* paired epilogue: 0 the clamped unit above, 1 g * sigmoid(g) * u */
-    uint32_t reserved0;
+    uint32_t d_op;                 /* applied to the finished element (after scale, gate and bias): 0 none, 1 the exact gelu z * Phi(z) */
     uint64_t gate_bias;            /* optional f32 [n] (with gate): sigmoid(gate[row, col] + gate_bias[col]) */
     uint64_t col_scale;            /* optional f32 [n]: the product is multiplied by col_scale[col] (a per-channel layer scale) */
     uint64_t row_scale;            /* optional f32 [compact rows]: the product of compact row p is multiplied by row_scale[p] before any
@@ -498,6 +498,18 @@ typedef struct uzu_dense_linear_args {
     uint32_t token_table_stride, token_column, token_vocab;
     uint32_t a_bf16;               /* 1: A is bf16 [m, k] (lda = k, 16-byte aligned), e.g. rows of a bf16 cache; only the tcgen05 form takes it
                                       (bf16 weights, batch 1, m >= 128, k a multiple of 64, n >= 64), no A operation */
+    /* Stream epilogue (streams 1..4; batch = 1, no accumulate; not on the tcgen05 form): the finished product y is a sublayer's result over a
+     * residual kept as `streams` copies x_s (f32 [rows, streams, n], stream_x). Element by element, from the old copies,
+     *   x_t <- sum_s stream_mix[s, t] x_s + stream_out[t] y,   stream_u[row, col] = sum_t stream_in[t] x_t   (stream_in 0: all ones)
+     * stream_u (f32 [rows, n]) is what the next sublayer's norm reads. D is not written. */
+    uint64_t stream_x, stream_mix, stream_out, stream_in, stream_u;
+    /* Layer-norm prologue (a_norm_weight != 0): every A row is replaced by (x - mean) / sqrt(variance + a_norm_epsilon) * a_norm_weight[k]
+     * as it is staged. Passes of at most 8 rows whose rows fit the staging buffer (m * k <= 8192, k a multiple of 8, dense 16-byte rows). */
+    uint64_t a_norm_weight;
+    float a_norm_epsilon;
+    uint32_t streams;
+    uint32_t d_bf16;               /* 1: D is bf16 [m, ldd] (tcgen05 form only, no accumulate): the next product's A rows */
+    uint32_t reserved1;
 } uzu_dense_linear_args;
 UZU_API void uzu_dense_linear_encode(uzu_command_buffer* cmd, const uzu_dense_linear_args* args);
 /* 0, or the code of the first bounded barrier wait that ran out inside a tensor-memory dense product (the kernel gives up and returns) */
@@ -518,6 +530,7 @@ UZU_API void uzu_group_rms_norm_encode(uzu_command_buffer* cmd, const uzu_group_
 /* A norm of `input`, optionally added into a residual stream, optionally followed by the next sublayer's norm of the updated stream:
  *   norm(x)  = x / sqrt(mean(x^2) + epsilon) * weight (+ bias)          (kind 0: RMS norm)
  *            = tanh(alpha * x) * weight + bias                          (kind 1: Dynamic Tanh, no mean and no variance)
+ *            = (x - mean(x)) / sqrt(mean((x - mean(x))^2) + epsilon) * weight (+ bias)     (kind 2: layer norm)
  *   residual == 0:  output = norm(input)
  *   residual != 0:  residual += mult * norm(input);  output (optional) = next_norm(residual), of kind next_kind with next_weight /
  *                   next_bias / next_alpha.
@@ -529,6 +542,20 @@ typedef struct uzu_norm_add_args {
     uint32_t reserved;
 } uzu_norm_add_args;
 UZU_API void uzu_norm_add_encode(uzu_command_buffer* cmd, const uzu_norm_add_args* args);
+
+/* Residual kept as `streams` copies x_s of every row (f32 [rows, streams, n]), one launch between two sublayers. Steps, each optional:
+ *   begin  (token_ids != 0): x_s = embedding row of the token, for all s (table [vocab, n] of type table_dt; ids >= vocab read 0)
+ *   update (y != 0):         x_t <- sum_s mix[s, t] x_s + out[t] y, all t from the old copies
+ *   read:                    u = sum_s read[s] x_s   (read = 0: all ones); stored to `u` when given
+ *   norm   (output != 0):    output = (u - mean(u)) / sqrt(mean((u - mean(u))^2) + epsilon) * weight   (f32 rows, or bf16 with output_bf16)
+ * mix f32 [streams, streams] (from, to), out / read f32 [streams]; all sums f32. At most 16 streams. */
+typedef struct uzu_stream_mix_args {
+    uint64_t x, y, mix, out, read, u, weight, output, token_ids, table;
+    uint32_t rows, n, streams, vocab, table_dt, output_bf16;
+    float epsilon;
+    uint32_t reserved;
+} uzu_stream_mix_args;
+UZU_API void uzu_stream_mix_encode(uzu_command_buffer* cmd, const uzu_stream_mix_args* args);
 
 /* Per-layer token input, the elementwise part: out[r, i] = gelu_tanh(z[r, i]) * table[token[r], column + i] for i < n, with
  * gelu_tanh(z) = z/2 (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))); table is weights_dt [vocab, table_stride]; z, out f32 [rows, n]. */
@@ -731,6 +758,44 @@ typedef struct uzu_exp_gates_args {
 } uzu_exp_gates_args;
 UZU_API void uzu_exp_gates_encode(uzu_command_buffer* cmd, const uzu_exp_gates_args* args);
 
+/* Inputs of a gated delta rule, for `rows` tokens of one sequence at positions p = prefix + t (prefix read from dynamic_position when
+ * non-zero). proj f32 [rows, stride] holds per row the projections [q: kv_heads*dim | k: kv_heads*dim | v: heads*vdim] from column 0 and, at
+ * a_offset and b_offset, one decay and one step-size projection per head.
+ *   q, k, v each pass a causal convolution over the tokens per channel, y[c] = sum_j conv[c, j] x_(p - taps + 1 + j)[c] (zero before
+ *   position 0), then silu; q and k become unit vectors per head, x / sqrt(sum x^2 + 1e-6), and q is multiplied by dim^(-1/2);
+ *   decay[t, h] = exp(-exp(a_log[h]) softplus(a + dt_bias[h]));  beta[t, h] = sigmoid(b)
+ * Inputs of earlier passes come from `ring` (f32 [taps, 2*kv_heads*dim + heads*vdim]): the input of position p lies in slot p % taps.
+ * Outputs f32: q, k [rows, kv_heads, dim4] (dim4 = dim rounded up to a multiple of 4, the pad is zero), v [rows, heads*vdim], decay, beta
+ * [rows, heads]. The ring is not advanced here (uzu_gated_delta_encode and uzu_gated_delta_step_encode do that). */
+typedef struct uzu_delta_prepare_args {
+    uint64_t proj, conv /* f32 [2*kv_heads*dim + heads*vdim, taps] */, ring, a_log, dt_bias /* f32 [heads] */, dynamic_position;
+    uint64_t q, k, v, decay, beta;
+    uint32_t rows, heads, kv_heads, dim, vdim, taps, stride, a_offset, b_offset, prefix;
+} uzu_delta_prepare_args;
+UZU_API void uzu_delta_prepare_encode(uzu_command_buffer* cmd, const uzu_delta_prepare_args* args);
+
+/* Gated delta rule over the prepared inputs of uzu_delta_prepare_encode, token by token; per head (reading q / k head h / (heads / kv_heads)):
+ *   S <- decay S;  S <- S + k (beta (v - S^T k))^T;  out[t, h, :] = S^T q
+ * state f32 [heads, vdim, dim4] (the dim entries of a value column are contiguous), read and written back; out f32 [rows, heads*vdim].
+ * prep.rows tokens in one launch, which also stores the pass's last inputs of the convolution into prep.ring. */
+typedef struct uzu_gated_delta_args {
+    uzu_delta_prepare_args prep;
+    uint64_t state, out;
+} uzu_gated_delta_args;
+UZU_API void uzu_gated_delta_encode(uzu_command_buffer* cmd, const uzu_gated_delta_args* args);
+
+/* One token of a whole gated-delta-rule mixer between its projections, in one launch: the convolution, unit vectors and gates of
+ * uzu_delta_prepare_encode, the state update and read-out of uzu_gated_delta_encode, then per head o / sqrt(mean(o^2) + epsilon) * norm[vdim]
+ * * silu(gate) with the gate at gate_offset of the projection row (heads*vdim columns). out f32 [heads*vdim]. prep.rows must be 1; prep.q .. beta
+ * are not used. */
+typedef struct uzu_gated_delta_step_args {
+    uzu_delta_prepare_args prep;
+    uint64_t state, norm, out;
+    uint32_t gate_offset;
+    float epsilon;
+} uzu_gated_delta_step_args;
+UZU_API void uzu_gated_delta_step_encode(uzu_command_buffer* cmd, const uzu_gated_delta_step_args* args);
+
 /* Windowed softmax attention, cache side and query side of one pass. Per token row t at position p = prefix + t (prefix read from
  * dynamic_position when non-zero), per head: optional RMS norm over the head's `dim` channels times q_scales / k_scales [dim] (shared by
  * all heads), then rotation of the first 2 * rot_pairs channels (interleaved pairs, or two halves with rot_halves) by cos / sin rows
@@ -743,11 +808,15 @@ typedef struct uzu_window_attention_prepare_args {
     uint32_t rows, heads, kv_heads, dim, vdim, rot_pairs, v_pairs, q_stride, k_stride, v_stride, prefix, cache_dt;
     float epsilon;
     uint32_t rot_halves;           /* 1: q / k pair channel i with channel i + rot_pairs (two halves) instead of (2i, 2i + 1); values keep the interleaved pairs */
+    uint32_t unit_rms;             /* 1: q and k are divided by their root mean square per head also without a weight row (a rotation keeps the norm, so
+                                      the order of norm and rotation does not matter then) */
+    uint32_t reserved;
 } uzu_window_attention_prepare_args;
 UZU_API void uzu_window_attention_prepare_encode(uzu_command_buffer* cmd, const uzu_window_attention_prepare_args* args);
 
 /* Causal softmax attention of `rows` queries (positions p = prefix + t) over cached keys / values with a sliding window that keeps the
- * first tokens: key j is visible when j <= p and (p - j < window or j < keep_first); window = 0 means no window. Query head h reads
+ * first tokens: key j is visible when j <= p and (p - j < window or j < keep_first); window = 0 means no window; a chunk bounds the
+ * window's keys to the query's own chunk. Query head h reads
  * key / value head h / (heads / kv_heads).
  *   s = scale * head_temp[h] * query . key;  softcap > 0: s <- softcap * tanh(s / softcap);  weights = softmax over the visible keys
  *   out[t, h, :] = rotate_(-p)(sum_j weight_j * values[j, g, :])   (the rotation back over 2 * v_pairs channels only when v_pairs > 0)
@@ -765,6 +834,8 @@ typedef struct uzu_window_attention_args {
     uint32_t splits, head_gate_stride;
     uint64_t sinks;                /* optional f32 [heads]: the softmax denominator also holds exp(sinks[h]) (no key, no value, not scaled) */
     uint64_t head_gate;            /* optional f32 [rows, head_gate_stride]: head h's output is multiplied by sigmoid(head_gate[t, h]) */
+    uint32_t chunk;                /* > 0: only keys of the query's own chunk are visible, floor(j / chunk) = floor(p / chunk), counted from position 0 */
+    uint32_t reserved;
 } uzu_window_attention_args;
 UZU_API void uzu_window_attention_encode(uzu_command_buffer* cmd, const uzu_window_attention_args* args);
 
@@ -798,6 +869,8 @@ typedef struct uzu_model_info {
     uint64_t weight_bytes_per_token;      /* algorithmic bytes of quantised weights one decode step streams */
     uint64_t kv_bytes_per_token_per_ctx;  /* K+V bytes read per context token per decode step */
     uint64_t state_bytes_per_token;       /* DeltaNet state read+write bytes per decode step */
+    uint32_t num_layer_runs;              /* layer runs of a pass: num_layers, or more when a range of layers runs several times */
+    uint32_t reserved;
 } uzu_model_info;
 
 UZU_API uzu_status uzu_engine_create(uzu_context* ctx, const char* model_dir, const uzu_engine_options* opts, uzu_engine** out);
@@ -836,7 +909,8 @@ UZU_API uzu_status uzu_engine_slot_acquire(uzu_engine* e, uint32_t* out_slot);
 UZU_API uzu_status uzu_engine_slot_release(uzu_engine* e, uint32_t slot);
 UZU_API uzu_status uzu_engine_forward_rows(uzu_engine* e, uint32_t slot, const uint32_t* tokens, uint32_t count, const uint32_t* rows,
                                            uint32_t nrows, float* out_logits);
-/* f32 residual stream after every layer of the last pass (models of the parallel-block family; debug / parity): [layers, count, model_dim] */
+/* f32 residual stream (the sum of the streams, if there are several) after every layer run of the last pass (models of the parallel-block
+ * family; debug / parity): [num_layer_runs, count, model_dim] */
 UZU_API uzu_status uzu_engine_debug_layer_outputs(uzu_engine* e, uint32_t enable, float* out, uint32_t capacity_floats, uint32_t* out_count);
 /* Multi-sequence batched decode (extension -- the reference decodes ONE sequence; BASELINE config 4 "batch = 8"): `sequences` (<= 16)
  * independent sequence states (own KV caches / DeltaNet states / positions) advance by one token per step and share one pass over the

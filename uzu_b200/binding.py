@@ -121,7 +121,7 @@ SamplingMethod = _struct("uzu_sampling_method", [
 ModelInfo = _struct("uzu_model_info", [
     ("model_dim", u32), ("hidden_dim", u32), ("vocab_size", u32), ("num_layers", u32), ("num_attention_layers", u32),
     ("num_delta_net_layers", u32), ("weight_bytes_per_token", u64), ("kv_bytes_per_token_per_ctx", u64),
-    ("state_bytes_per_token", u64)])
+    ("state_bytes_per_token", u64), ("num_layer_runs", u32), ("reserved", u32)])
 
 TpAllGatherArgs = _struct("uzu_tp_all_gather_args", [("src", u64), ("dst", u64), ("scratch", u64), ("rows", u32), ("cols_local", u32)])
 
@@ -136,10 +136,12 @@ DenseLinearArgs = _struct("uzu_dense_linear_args", [
     ("a_z_stride", u64), ("w_z_stride", u64), ("d_z_stride", u64), ("gate", u64), ("workspace", u64),
     ("m", u32), ("n", u32), ("k", u32), ("lda", u32), ("ldd", u32), ("batch", u32),
     ("weights_dt", u32), ("accumulate", u32), ("scale", f32), ("a_op", u32), ("gate_ld", u32), ("pair_rows", u32),
-    ("glu_limit", f32), ("glu_alpha", f32), ("glu_kind", u32), ("reserved0", u32), ("gate_bias", u64), ("col_scale", u64), ("row_scale", u64),
+    ("glu_limit", f32), ("glu_alpha", f32), ("glu_kind", u32), ("d_op", u32), ("gate_bias", u64), ("col_scale", u64), ("row_scale", u64),
     ("post_weight", u64), ("post_bias", u64), ("next_weight", u64), ("next_bias", u64), ("next_out", u64),
     ("post_alpha", f32), ("post_mult", f32), ("next_alpha", f32), ("token_gate_dt", u32), ("token_ids", u64), ("token_table", u64),
-    ("token_table_stride", u32), ("token_column", u32), ("token_vocab", u32), ("a_bf16", u32)])
+    ("token_table_stride", u32), ("token_column", u32), ("token_vocab", u32), ("a_bf16", u32),
+    ("stream_x", u64), ("stream_mix", u64), ("stream_out", u64), ("stream_in", u64), ("stream_u", u64), ("a_norm_weight", u64), ("a_norm_epsilon", f32),
+    ("streams", u32), ("d_bf16", u32), ("reserved1", u32)])
 
 GroupRmsNormArgs = _struct("uzu_group_rms_norm_args", [
     ("input", u64), ("scales", u64), ("output", u64), ("row_indices", u64),
@@ -218,17 +220,33 @@ WindowAttentionPrepareArgs = _struct("uzu_window_attention_prepare_args", [
     ("q", u64), ("k", u64), ("v", u64), ("q_scales", u64), ("k_scales", u64), ("query", u64), ("keys", u64), ("values", u64),
     ("cosines", u64), ("sines", u64), ("v_cosines", u64), ("v_sines", u64), ("dynamic_position", u64),
     ("rows", u32), ("heads", u32), ("kv_heads", u32), ("dim", u32), ("vdim", u32), ("rot_pairs", u32), ("v_pairs", u32),
-    ("q_stride", u32), ("k_stride", u32), ("v_stride", u32), ("prefix", u32), ("cache_dt", u32), ("epsilon", f32), ("rot_halves", u32)])
+    ("q_stride", u32), ("k_stride", u32), ("v_stride", u32), ("prefix", u32), ("cache_dt", u32), ("epsilon", f32), ("rot_halves", u32), ("unit_rms", u32), ("reserved", u32)])
 
 WindowAttentionArgs = _struct("uzu_window_attention_args", [
     ("query", u64), ("keys", u64), ("values", u64), ("out", u64), ("dynamic_position", u64), ("head_temp", u64),
     ("v_cosines", u64), ("v_sines", u64), ("partials", u64), ("tickets", u64),
     ("rows", u32), ("heads", u32), ("kv_heads", u32), ("dim", u32), ("vdim", u32), ("prefix", u32), ("cache_dt", u32), ("window", u32),
-    ("keep_first", u32), ("v_pairs", u32), ("scale", f32), ("softcap", f32), ("splits", u32), ("head_gate_stride", u32), ("sinks", u64), ("head_gate", u64)])
+    ("keep_first", u32), ("v_pairs", u32), ("scale", f32), ("softcap", f32), ("splits", u32), ("head_gate_stride", u32), ("sinks", u64), ("head_gate", u64),
+    ("chunk", u32), ("reserved", u32)])
+
+StreamMixArgs = _struct("uzu_stream_mix_args", [
+    ("x", u64), ("y", u64), ("mix", u64), ("out", u64), ("read", u64), ("u", u64), ("weight", u64), ("output", u64), ("token_ids", u64), ("table", u64),
+    ("rows", u32), ("n", u32), ("streams", u32), ("vocab", u32), ("table_dt", u32), ("output_bf16", u32), ("epsilon", f32), ("reserved", u32)])
+
+DeltaPrepareArgs = _struct("uzu_delta_prepare_args", [
+    ("proj", u64), ("conv", u64), ("ring", u64), ("a_log", u64), ("dt_bias", u64), ("dynamic_position", u64),
+    ("q", u64), ("k", u64), ("v", u64), ("decay", u64), ("beta", u64),
+    ("rows", u32), ("heads", u32), ("kv_heads", u32), ("dim", u32), ("vdim", u32), ("taps", u32), ("stride", u32), ("a_offset", u32),
+    ("b_offset", u32), ("prefix", u32)])
+
+GatedDeltaArgs = _struct("uzu_gated_delta_args", [("prep", DeltaPrepareArgs), ("state", u64), ("out", u64)])
+
+GatedDeltaStepArgs = _struct("uzu_gated_delta_step_args", [
+    ("prep", DeltaPrepareArgs), ("state", u64), ("norm", u64), ("out", u64), ("gate_offset", u32), ("epsilon", f32)])
 
 MAIN_SLOT = 0xFFFFFFFF
 
-ABI_STRUCTS = [ExpGatesArgs, NormAddArgs, TokenGateArgs, MinGruArgs, RetentionArgs, WindowAttentionPrepareArgs, WindowAttentionArgs, TopkRouteArgs, RoutedCombineArgs, SigmoidAttentionPrepareArgs, SigmoidAttentionArgs, DenseLinearArgs, GroupRmsNormArgs, TableRouteArgs, GeneralDeltaArgs, HeadNormGateArgs, LatentPrepareArgs, LatentAttentionArgs,
+ABI_STRUCTS = [StreamMixArgs, DeltaPrepareArgs, GatedDeltaArgs, GatedDeltaStepArgs, ExpGatesArgs, NormAddArgs, TokenGateArgs, MinGruArgs, RetentionArgs, WindowAttentionPrepareArgs, WindowAttentionArgs, TopkRouteArgs, RoutedCombineArgs, SigmoidAttentionPrepareArgs, SigmoidAttentionArgs, DenseLinearArgs, GroupRmsNormArgs, TableRouteArgs, GeneralDeltaArgs, HeadNormGateArgs, LatentPrepareArgs, LatentAttentionArgs,
                DeltaNetFusedUpdateArgs, QkNormConfig, AttentionPrepareNormArgs, FusedLinearArgs, RingParams, TrieNode, KvCopy, MatmulArgs, NormalizationArgs, QkvNormArgs, AttentionPrepareArgs, AttentionArgs,
                AttentionTwoPass2Args, KvCacheUpdateArgs, GatedActMulArgs, QuantizedEmbeddingLookupArgs, UnifiedSamplingArgs,
                DeltaNetConvUpdateArgs, DeltaNetUpdateArgs, EngineOptions, SamplingMethod, ModelInfo, TpAllGatherArgs]
@@ -262,7 +280,8 @@ uzu_general_delta_encode uzu_head_norm_gate_encode uzu_latent_prepare_encode uzu
 uzu_silu_glu_encode uzu_topk_route_encode uzu_routed_combine_gated_encode uzu_sigmoid_attention_prepare_encode uzu_sigmoid_attention_encode
 uzu_engine_slot_acquire uzu_engine_slot_release uzu_engine_forward_rows uzu_engine_debug_layer_outputs uzu_debug_dense_umma_error
 uzu_min_gru_encode uzu_retention_encode uzu_window_attention_prepare_encode uzu_window_attention_encode
-uzu_exp_gates_encode uzu_norm_add_encode uzu_token_gate_encode uzu_embedding_f32_scaled_encode uzu_rows_to_bf16_encode""".split()
+uzu_exp_gates_encode uzu_norm_add_encode uzu_token_gate_encode uzu_embedding_f32_scaled_encode uzu_rows_to_bf16_encode
+uzu_stream_mix_encode uzu_delta_prepare_encode uzu_gated_delta_encode uzu_gated_delta_step_encode""".split()
 
 _lib = None
 
@@ -419,6 +438,10 @@ def load() -> C.CDLL:
         "uzu_window_attention_encode": (None, [vp, C.POINTER(WindowAttentionArgs)]),
         "uzu_exp_gates_encode": (None, [vp, C.POINTER(ExpGatesArgs)]),
         "uzu_norm_add_encode": (None, [vp, C.POINTER(NormAddArgs)]),
+        "uzu_stream_mix_encode": (None, [vp, C.POINTER(StreamMixArgs)]),
+        "uzu_delta_prepare_encode": (None, [vp, C.POINTER(DeltaPrepareArgs)]),
+        "uzu_gated_delta_encode": (None, [vp, C.POINTER(GatedDeltaArgs)]),
+        "uzu_gated_delta_step_encode": (None, [vp, C.POINTER(GatedDeltaStepArgs)]),
         "uzu_token_gate_encode": (None, [vp, C.POINTER(TokenGateArgs)]),
         "uzu_rows_to_bf16_encode": (None, [vp, u64, u32, u64, u32, u32]),
         "uzu_embedding_f32_scaled_encode": (None, [vp, u64, u64, u32, u64, u32, u32, u32, f32]),
@@ -685,14 +708,14 @@ class Engine:
         return out
 
     def debug_layer_outputs(self, enable=True) -> np.ndarray | None:
-        """Switch the per-layer residual dump on / off; with it on, returns [layers, rows, model_dim] f32 of the last pass (None before one)."""
+        """Switch the per-layer residual dump on / off; with it on, returns [layer runs, rows, model_dim] f32 of the last pass (None before one)."""
         n = u32()
         _check(self.lib.uzu_engine_debug_layer_outputs(self.h, int(enable), None, 0, C.byref(n)))
         if not enable or n.value == 0:
             return None
         out = np.zeros(n.value, dtype=np.float32)
         _check(self.lib.uzu_engine_debug_layer_outputs(self.h, 1, out.ctypes.data_as(C.POINTER(C.c_float)), n.value, C.byref(n)))
-        return out.reshape(self.info.num_layers, -1, self.info.model_dim)
+        return out.reshape(self.info.num_layer_runs, -1, self.info.model_dim)
 
     @property
     def launch_count(self):

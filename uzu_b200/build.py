@@ -46,6 +46,7 @@ SOURCES = {
     "window_attention.cu": [],
     "window_attention_mma.cu": [],
     "linear_recurrence.cu": [],
+    "gated_delta.cu": [],
     "engine.cu": [],
 }
 

@@ -106,6 +106,11 @@ inline void launch(uzu_command_buffer* cmd, const char* what, void (*kernel)(KAr
 bool prefill_gemm_applicable(const uzu_matmul_args& a);
 void encode_prefill_gemm(uzu_command_buffer* cmd, const uzu_matmul_args& a);
 
+// whether a dense product runs on the kernel that can norm its A rows as it stages them (dense_linear.cu)
+bool dense_rows_takes_norm(const uzu_dense_linear_args& a);
+// whether a dense product runs on tcgen05 with its operands in tensor memory (dense_umma.cu)
+bool dense_umma_applicable(const uzu_dense_linear_args& a);
+
 // tensor-core prefill attention (attention_prefill.cu, opt-in), tried first by uzu_attention_single_pass_encode
 bool encode_attention_prefill(uzu_command_buffer* cmd, const uzu_attention_args& a);
 

@@ -16,7 +16,6 @@
 namespace uzu {
 
 // tcgen05 form of the plain bf16 product (dense_umma.cu)
-bool dense_umma_applicable(const uzu_dense_linear_args& a);
 void encode_dense_umma(uzu_command_buffer* cmd, const uzu_dense_linear_args& a);
 
 struct DenseRows {
@@ -45,6 +44,32 @@ __device__ __forceinline__ float dense_a(const uzu_dense_linear_args& a, float x
     return x;
 }
 
+// x_t <- sum_s mix[s, t] x_s + out[t] y for one element of a row, and u = sum_t read[t] x_t
+constexpr int DL_MAX_STREAMS = 4;
+__device__ __forceinline__ void stream_store(const uzu_dense_linear_args& a, uint32_t row, uint32_t col, float y) {
+    const uint32_t S = a.streams;
+    float* x = reinterpret_cast<float*>(a.stream_x) + (size_t)row * S * a.n + col;
+    const float* mix = reinterpret_cast<const float*>(a.stream_mix);
+    const float* out = reinterpret_cast<const float*>(a.stream_out);
+    const float* in = reinterpret_cast<const float*>(a.stream_in);
+    constexpr int MAXS = DL_MAX_STREAMS;
+    float old[MAXS], u = 0.0f;
+#pragma unroll
+    for (int s = 0; s < MAXS; ++s) old[s] = (uint32_t)s < S ? x[(size_t)s * a.n] : 0.0f;
+#pragma unroll
+    for (int t = 0; t < MAXS; ++t) {
+        if ((uint32_t)t < S) {
+            float v = out[t] * y;
+#pragma unroll
+            for (int s = 0; s < MAXS; ++s)
+                if ((uint32_t)s < S) v = fmaf(mix[s * S + t], old[s], v);
+            x[(size_t)t * a.n] = v;
+            u = fmaf(in ? in[t] : 1.0f, v, u);
+        }
+    }
+    reinterpret_cast<float*>(a.stream_u)[(size_t)row * a.n + col] = u;
+}
+
 // `row` is the compact row the value belongs to (the gate is indexed like D)
 __device__ __forceinline__ void dense_store(const uzu_dense_linear_args& a, float* d, uint32_t z, uint32_t row, uint32_t col, float acc) {
     float v = acc * a.scale;
@@ -56,6 +81,11 @@ __device__ __forceinline__ void dense_store(const uzu_dense_linear_args& a, floa
     }
     if (a.col_scale) v *= reinterpret_cast<const float*>(a.col_scale)[col];
     if (a.bias && z == 0) v += reinterpret_cast<const float*>(a.bias)[col];
+    if (a.d_op == 1) v = 0.5f * v * (1.0f + erff(v * 0.70710678118654752f));
+    if (a.streams) {              // stream epilogue: the residual's copies take the product, and the next reader's weighted sum of them is formed
+        stream_store(a, row, col, v);
+        return;
+    }
     if (a.post_weight) {          // sandwich epilogue: the product's own Dynamic Tanh norm, the residual add, the next reader's norm
         float y = tanhf(a.post_alpha * v) * reinterpret_cast<const float*>(a.post_weight)[col];
         if (a.post_bias) y += reinterpret_cast<const float*>(a.post_bias)[col];
@@ -109,6 +139,31 @@ __device__ __forceinline__ float clamped_glu_value(float g, float u, float limit
 }
 
 constexpr uint32_t DL_STAGE_FLOATS = 8192;   // activation rows of a group are staged in shared memory when they fit (32 KB)
+
+// the staged rows become their layer norms: the whole CTA works on a single row, otherwise a warp takes a row
+template <int RMAX>
+__device__ __forceinline__ void layer_norm_rows(const uzu_dense_linear_args& a, float* rows, uint32_t count) {
+    __shared__ float red[32];
+    const float* w = reinterpret_cast<const float*>(a.a_norm_weight);
+    const uint32_t lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    if constexpr (RMAX == 1) {
+        float s = 0.0f, ss = 0.0f;
+        for (uint32_t i = threadIdx.x; i < a.k; i += blockDim.x) s += rows[i];
+        const float mean = block_sum(s, red) / (float)a.k;
+        for (uint32_t i = threadIdx.x; i < a.k; i += blockDim.x) { const float d = rows[i] - mean; ss = fmaf(d, d, ss); }
+        const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)a.k + a.a_norm_epsilon);
+        for (uint32_t i = threadIdx.x; i < a.k; i += blockDim.x) rows[i] = (rows[i] - mean) * inv * w[i];
+    } else if (warp < count) {
+        float* x = rows + (size_t)warp * a.k;
+        float s = 0.0f, ss = 0.0f;
+        for (uint32_t i = lane; i < a.k; i += 32) s += x[i];
+        const float mean = warp_sum(s) / (float)a.k;
+        for (uint32_t i = lane; i < a.k; i += 32) { const float d = x[i] - mean; ss = fmaf(d, d, ss); }
+        const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)a.k + a.a_norm_epsilon);
+        for (uint32_t i = lane; i < a.k; i += 32) x[i] = (x[i] - mean) * inv * w[i];
+    }
+    __syncthreads();
+}
 
 // RMAX = most activation rows of a group (1 for a plain decode step: one accumulator, no row pointers -> more CTAs per SM).
 template <typename TW, int KS, bool PAIR, int RMAX>
@@ -169,6 +224,7 @@ __global__ void __launch_bounds__(256, RMAX == 1 ? 4 : 2) dense_rows_kernel(cons
             reinterpret_cast<float4*>(a_s)[i] = x;
         }
         __syncthreads();
+        if (a.a_norm_weight) layer_norm_rows<RMAX>(a, a_s, R.count);
     }
     float acc[RMAX], acc2[PAIR ? RMAX : 1];
 #pragma unroll
@@ -574,6 +630,13 @@ __global__ void __launch_bounds__(256) dense_tensor128_kernel(const uzu_dense_li
             }
 }
 
+// the rows kernel stages its activation rows under exactly these conditions (its own test of them includes the device addresses)
+bool dense_rows_takes_norm(const uzu_dense_linear_args& a) {
+    const uint32_t vec = a.weights_dt == UZU_DT_BF16 ? 8 : 4, lda = a.lda ? a.lda : a.k;
+    return a.m <= (uint32_t)DL_MAX_ROWS && (size_t)a.m * a.k <= DL_STAGE_FLOATS && a.k % vec == 0 && lda % 4 == 0 && (a.w & 15) == 0 && (a.a & 15) == 0 &&
+           a.batch == 1 && !a.group_offsets && !a.rows_map && !a.a_op && !a.a_bf16 && (!a.pair_rows || ((uint64_t)a.pair_rows * a.k) % vec == 0);
+}
+
 }  // namespace uzu
 
 extern "C" void uzu_dense_linear_encode(uzu_command_buffer* cmd, const uzu_dense_linear_args* args) {
@@ -594,11 +657,25 @@ extern "C" void uzu_dense_linear_encode(uzu_command_buffer* cmd, const uzu_dense
         cmd->record_error(UZU_ERROR_INVALID_ARGUMENT, "dense_linear: the sandwich / token-gate epilogues take one plain product (no accumulate, no pairs, no batch)");
         return;
     }
+    if (a.d_op > 1 || (a.pair_rows && a.d_op) || (a.d_bf16 && a.accumulate) ||
+        (a.streams && (a.streams > (uint32_t)DL_MAX_STREAMS || !a.stream_x || !a.stream_mix || !a.stream_out || !a.stream_u || a.accumulate || a.batch != 1 || a.pair_rows ||
+                       a.group_offsets || a.rows_map || a.post_weight || a.token_table || a.d_bf16))) {
+        cmd->record_error(UZU_ERROR_INVALID_ARGUMENT, "dense_linear: unknown D operation, a bf16 D that accumulates, or a stream epilogue that is not one plain product");
+        return;
+    }
     if (a.m == 0 || a.n == 0) return;
+    if (a.a_norm_weight && !dense_rows_takes_norm(a)) {
+        cmd->record_error(UZU_ERROR_UNSUPPORTED, "dense_linear: the layer-norm prologue takes one plain product of at most 8 rows that fit the staging buffer");
+        return;
+    }
+    if (a.d_bf16 && (a.post_weight || a.token_table || !dense_umma_applicable(a))) {
+        cmd->record_error(UZU_ERROR_UNSUPPORTED, "dense_linear: a bf16 D needs the tcgen05 form");
+        return;
+    }
     if (a.a_bf16) {      // A rows that are bf16 already (a cache's rows): the tensor-memory form reads them as they are
         const bool dense_rows = a.lda == 0 || a.lda == a.k;
         a.lda = a.k;
-        if (!dense_rows || a.a_op || a.post_weight || a.token_table || !dense_umma_applicable(a)) {
+        if (!dense_rows || a.a_op || a.post_weight || a.token_table || a.streams || !dense_umma_applicable(a)) {
             cmd->record_error(UZU_ERROR_UNSUPPORTED, "dense_linear: bf16 activations need the tcgen05 form (bf16 weights, dense rows, a workspace pointer, m >= 128, k a multiple of 64, n >= 64, no A operation)");
             return;
         }
@@ -640,7 +717,7 @@ extern "C" void uzu_dense_linear_encode(uzu_command_buffer* cmd, const uzu_dense
         cmd->record_error(UZU_ERROR_UNSUPPORTED, "dense_linear: the paired gated-unit epilogue covers passes of at most 8 rows");
         return;
     }
-    if (!a.post_weight && !a.token_table && dense_umma_applicable(a)) {
+    if (!a.post_weight && !a.token_table && !a.streams && dense_umma_applicable(a)) {
         encode_dense_umma(cmd, a);
         return;
     }

@@ -25,7 +25,7 @@ struct DenseUmmaParams {
     const float* col_scale;    // optional [n]
     const float* bias;         // optional [n], added after scale / gate / col_scale
     const float* row_scale;    // optional [m]
-    uint32_t m, n, k, ldd, gate_ld, accumulate;
+    uint32_t m, n, k, ldd, gate_ld, accumulate, d_op, d_bf16;
     float scale;
     uint32_t desc_hi, desc_lbo, k_step, idesc;
     unsigned int* error;
@@ -168,6 +168,7 @@ __global__ void __launch_bounds__(DU_NP + 32, 1) dense_umma_kernel(const DenseUm
                 const uint32_t col0 = n0 + cb * 32u;
                 if (row >= p.m || col0 >= p.n) continue;
                 float* out = p.d + (size_t)row * p.ldd + col0;
+                __nv_bfloat16* out16 = reinterpret_cast<__nv_bfloat16*>(p.d) + (size_t)row * p.ldd + col0;
                 const float* gate = p.gate ? p.gate + (size_t)row * p.gate_ld + col0 : nullptr;
                 const float rs = p.row_scale ? p.row_scale[row] : 1.0f;
 #pragma unroll
@@ -178,6 +179,8 @@ __global__ void __launch_bounds__(DU_NP + 32, 1) dense_umma_kernel(const DenseUm
                         if (gate) val *= 1.0f / (1.0f + expf(-(gate[j] + (p.gate_bias ? p.gate_bias[col0 + j] : 0.0f))));
                         if (p.col_scale) val *= p.col_scale[col0 + j];
                         if (p.bias) val += p.bias[col0 + j];
+                        if (p.d_op == 1) val = 0.5f * val * (1.0f + erff(val * 0.70710678118654752f));
+                        if (p.d_bf16) { out16[j] = __float2bfloat16_rn(val); continue; }
                         if (p.accumulate) val += out[j];
                         out[j] = val;
                     }
@@ -263,7 +266,7 @@ void encode_dense_umma(uzu_command_buffer* cmd, const uzu_dense_linear_args& a) 
     p.col_scale = (const float*)a.col_scale;
     p.bias = (const float*)a.bias;
     p.row_scale = (const float*)a.row_scale;
-    p.m = a.m; p.n = a.n; p.k = a.k; p.ldd = a.ldd; p.gate_ld = a.gate_ld; p.accumulate = a.accumulate;
+    p.m = a.m; p.n = a.n; p.k = a.k; p.ldd = a.ldd; p.gate_ld = a.gate_ld; p.accumulate = a.accumulate; p.d_op = a.d_op; p.d_bf16 = a.d_bf16;
     p.scale = a.scale;
     // shared-memory matrix descriptor: start address >> 4 @ [0,14), LBO >> 4 @ [16,30), SBO >> 4 @ [32,46), version 1 @ [46,48), layout
     // SWIZZLE_128B = 2 @ [61,64); K-major: SBO = 1024 B between 8-row groups, LBO unused (1), UMMA_K = 16 bf16 = 32 B -> +2 per step.

@@ -286,14 +286,15 @@ struct Norm {
     Buf scales;
     uint32_t n = 0;
     bool present = false;
-    // parallel-block engine: kind 1 is the Dynamic Tanh norm tanh(alpha x) * scales + bias (no mean, no variance); kind 0 the RMS norm
+    // parallel-block engine: kind 1 is the Dynamic Tanh norm tanh(alpha x) * scales + bias (no mean, no variance); kind 0 the RMS norm; kind 2 the
+    // layer norm (mean taken off)
     uint32_t kind = 0;
     Buf bias;
     float alpha = 1.0f;
 };
 
 struct RopeCfg {
-    int kind = 0;  // 0 unscaled, 1 linear, 2 llama, 3 interleaved pairs with optional YaRN blending (table rows are [pairs], already scaled)
+    int kind = 0;  // 0 unscaled, 1 linear, 2 llama, 3 a table row holds the [pairs], already scaled: YaRN blending, or frequencies divided by scaling_factor
     float base = 10000.0f, scaling_factor = 1.0f, low = 1.0f, high = 1.0f;
     uint32_t head_dim = 0, original_context_length = 0, max_sequence_length = 0;
     bool yarn = false;          // kind 3: low / high hold the slow / fast rotation counts of the blend
@@ -398,6 +399,9 @@ struct WindowAttentionLayer {   // softmax attention with a sliding window that 
     float scale = 1.0f, softcap = 0.0f, share = 1.0f;
     int rope_index = -1, value_rope_index = -1;          // value_rope_index < 0: values are cached as they are
     bool rot_halves = false;    // q / k pair channel i with i + rot.dims / 2 instead of (2i, 2i + 1)
+    bool unit_rms = false;      // q and k are divided by their root mean square per head (no weight)
+    uint32_t chunk = 0;         // > 0: only keys of the query's own chunk of positions are visible
+    Buf sink;                   // f32 [heads] (absent: none): one more term exp(sink) in every softmax denominator
 };
 
 struct RetentionLayer {         // retention: per head S <- decay S + (k / sqrt(dim)) v^T, out = S^T q; per-head unit RMS, silu gate
@@ -408,16 +412,32 @@ struct RetentionLayer {         // retention: per head S <- decay S + (k / sqrt(
     float share = 1.0f;
 };
 
+struct GatedDeltaLayer {        // gated delta rule behind short convolutions: per head S [dim, vdim], one decay and one step size per head
+    DenseMatrix in;             // rows [query | key | value | output gate | decay | step size]; the first three parts pass the convolution
+    DenseMatrix out;
+    Buf conv;                   // f32 [2 * kv_heads * dim + heads * vdim, taps]
+    Buf a_log, dt_bias;         // f32 [heads]
+    Buf norm_weight;            // f32 [heads * vdim] (one row of vdim, repeated per head)
+    uint32_t heads = 0, kv_heads = 0, dim = 0, vdim = 0, taps = 1;
+    uint32_t gate_offset = 0, a_offset = 0, b_offset = 0;
+    uint32_t dim4() const { return (dim + 3) & ~3u; }
+    uint32_t channels() const { return 2 * kv_heads * dim + heads * vdim; }
+};
+
+struct StreamWeights {          // a sublayer over a residual of several streams: what it reads, how the streams mix, where its result goes
+    Buf read, mix, out;         // f32 [streams], [streams, streams] (from, to), [streams]
+};
+
 struct SublayerGate {           // y * scale[c] * sigmoid(gate_logit[c] + bias[c]); the gate logits are extra rows of the sublayer's stacked input projection
     bool present = false;
     Buf scale, bias;            // f32 [width]
     uint32_t offset = 0;        // first gate column of the stacked projection's output
 };
 
-struct GatedMlp {               // feed-forward: dense or routed experts; the unit is a clamped gated one, silu(g) * u, or relu(u)^2 (no gate rows)
+struct GatedMlp {               // feed-forward: dense or routed experts; the unit is a clamped gated one, silu(g) * u, relu(u)^2 or the exact gelu(u) (no gate rows)
     enum Kind { None, Dense, TableExperts, RoutedExperts } kind = None;
-    enum Unit { ClampedGlu, SiluGlu, ReluSquared } unit = ClampedGlu;
-    DenseMatrix gate_up /* experts x [2f, W]: gate rows then up rows; ReluSquared: [f (+ W gate logits), W] */, down /* experts x [W, f] */;
+    enum Unit { ClampedGlu, SiluGlu, ReluSquared, GeluExact } unit = ClampedGlu;
+    DenseMatrix gate_up /* experts x [2f, W]: gate rows then up rows; ReluSquared: [f (+ W gate logits), W]; GeluExact: [f, W] */, down /* experts x [W, f] */;
     DenseMatrix router;         // RoutedExperts: rows [router logits | sublayer gate]
     Buf table;                  // TableExperts: i32 [vocab, top]
     Buf router_bias;            // RoutedExperts: f32 [experts] (optional)
@@ -429,7 +449,7 @@ struct GatedMlp {               // feed-forward: dense or routed experts; the un
 
 enum MixerKind : uint32_t { MixAttention = 0, MixDeltaNet = 1, MixGeneralDelta = 2, MixLatentAttention = 3, MixSigmoidAttention = 4,
                            MixMinGru = 5, MixWindowAttention = 6, MixRetention = 7, MixSideBySide = 8 /* window attention + retention, summed */,
-                           MixMlstm = 9 };
+                           MixMlstm = 9, MixGatedDelta = 10 };
 
 struct Layer {
     bool is_attention = true;   // the mixer keeps a per-token cache whose length advances with the context (MixAttention, MixLatentAttention)
@@ -453,6 +473,11 @@ struct Layer {
     Norm post_mixer, post_mlp;
     float residual_mult = 1.0f;
     TokenSide side;
+    // Streamed form of a sequential layer: the residual is several copies, every sublayer reads a weighted sum of them and its result is mixed
+    // back into all of them (StreamWeights per sublayer).
+    bool streamed = false;
+    StreamWeights mixer_streams, mlp_streams;
+    GatedDeltaLayer dr;
     bool has_window_attention() const { return kind == MixWindowAttention || kind == MixSideBySide; }
     bool has_retention() const { return kind == MixRetention || kind == MixSideBySide; }
     SublayerGate mix_gate, mlp_gate;
@@ -539,6 +564,8 @@ struct uzu_engine {
     bool parallel_block = false;
     uint32_t store_dt = UZU_DT_BF16, norm_groups = 1;
     float norm_eps = 1e-5f;
+    uint32_t streams = 0;       // > 0: the residual is this many copies of a row ([rows, streams, width]), mixed by every sublayer
+    std::vector<uint32_t> runs; // the layer index of every layer run of a pass, in order; state[i] belongs to run i (a layer that runs twice has two)
     DenseMatrix pb_embed, pb_head, pb_side_embed;   // pb_side_embed: [vocab, layers * side dim], the table of the per-layer token inputs
     Buf pb_final_norm;
     Norm pb_out_norm;           // set when the output norm is not the grouped RMS norm (kind 1: Dynamic Tanh)
@@ -547,6 +574,14 @@ struct uzu_engine {
         Buf pair_weight_compact;                         // router weights in the expert-sorted order of the pair list
         Buf route_scratch;                               // the experts a long pass picked, between the router's two launches
         Buf sub_out;                                     // a sublayer's result before its own norm (sandwich layers)
+        // streamed layers: the weighted sum of the streams the next norm reads; short passes leave it there as the epilogue of a sublayer's last
+        // product and norm it inside the next sublayer's first one (`input_norm`), long ones store the normed rows (bf16 when the product
+        // that reads them runs on tcgen05)
+        Buf stream_u;
+        const StreamWeights* fused_streams = nullptr;
+        uint64_t fused_read = 0;
+        const Norm* input_norm = nullptr;
+        bool normed_bf16 = false;
         Buf token_factors;                               // per (token, head) decay, gain, floor and normaliser product of a gated matrix memory
         Buf expand_f32, expand_keys, expand_values;      // a prompt pass's expanded latents: f32 [rows, heads * (dim + vdim)], then bf16 keys and values
         uint32_t expand_rows = 0;                        // rows the three hold
@@ -756,7 +791,7 @@ static RopeCfg parse_rope(const Json& j) {
 static void rope_tables(const RopeCfg& c, uint32_t count, float* cosines, float* sines) {
     const uint32_t head_dim = c.head_dim, half = head_dim / 2;
     if (c.kind == 3) {
-        // Interleaved pairs (2i, 2i+1), frequency f_i = base^(-2i/dims). YaRN: with where(t) = dims * ln(original / (2 pi t)) / (2 ln base),
+        // One entry per pair, frequency f_i = base^(-2i/dims), divided by the scaling factor (1 without scaling). YaRN: with where(t) = dims * ln(original / (2 pi t)) / (2 ln base),
         // lo = max(floor(where(fast)), 0), hi = min(ceil(where(slow)), dims - 1), ramp_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1), the
         // frequency becomes f_i / factor * ramp_i + f_i * (1 - ramp_i) and cos / sin carry the factor 0.1 ln(factor) + 1. Frequencies are
         // formed in double and rounded once; the angle position * frequency is an f32 product.
@@ -774,6 +809,8 @@ static void rope_tables(const RopeCfg& c, uint32_t count, float* cosines, float*
             if (c.yarn) {
                 const double ramp = std::min(std::max(((double)i - lo) / std::max(hi - lo, 0.001), 0.0), 1.0);
                 f = f / (double)c.scaling_factor * ramp + f * (1.0 - ramp);
+            } else {
+                f /= (double)c.scaling_factor;
             }
             const float ff = (float)f;
             for (uint32_t t = 0; t < count; ++t) {
@@ -815,6 +852,7 @@ static void load_parallel_block_model(uzu_engine* e, const Json& cfg, const std:
 static void load_gamanex_model(uzu_engine* e, const Json& cfg, const std::string& dir);
 static void load_vugipel_model(uzu_engine* e, const Json& cfg, const std::string& dir);
 static void load_vakesun_model(uzu_engine* e, const Json& cfg, const std::string& dir);
+static void load_relidra_model(uzu_engine* e, const Json& cfg, const std::string& dir);
 static void load_language_model_config(uzu_engine* e, const Json& cfg, const std::string& dir);
 
 // Model registry: config.json names its family, either by the reference's type tag or by an "architecture" string.
@@ -829,6 +867,7 @@ static const ModelFamily kModelFamilies[] = {
     {"Gamanex", [](const Json& c) { const Json* a = c.get("architecture"); return a && a->str == "Gamanex"; }, load_gamanex_model},
     {"Vugipel", [](const Json& c) { const Json* a = c.get("architecture"); return a && a->str == "Vugipel"; }, load_vugipel_model},
     {"Vakesun", [](const Json& c) { const Json* a = c.get("architecture"); return a && a->str == "Vakesun"; }, load_vakesun_model},
+    {"Relidra", [](const Json& c) { const Json* a = c.get("architecture"); return a && a->str == "Relidra"; }, load_relidra_model},
 };
 
 static void load_model(uzu_engine* e, const std::string& dir) {
@@ -836,6 +875,9 @@ static void load_model(uzu_engine* e, const std::string& dir) {
     for (const ModelFamily& f : kModelFamilies)
         if (f.matches(cfg)) {
             f.load(e, cfg, dir);
+            if (e->runs.empty())
+                for (size_t i = 0; i < e->layers.size(); ++i) e->runs.push_back((uint32_t)i);
+            e->info.num_layer_runs = (uint32_t)e->runs.size();
             return;
         }
     throw std::runtime_error("config.json: not a LanguageModelConfig and no known \"architecture\"");
@@ -1064,6 +1106,15 @@ static void alloc_layer_state(uzu_engine* e, const Layer& L, LayerState& S, uint
             S.ssm_snapshot = make_buf(e, S.ssm_bytes, UZU_BUFFER_DEVICE);
             break;
         }
+        case MixGatedDelta: {        // f32 [heads, vdim, dim4], and a ring of the convolution's last inputs f32 [taps, channels]
+            S.ssm_bytes = (size_t)L.dr.heads * L.dr.vdim * L.dr.dim4() * 4;
+            S.conv_bytes = (size_t)L.dr.taps * L.dr.channels() * 4;
+            fixed(S.ssm_state, S.ssm_bytes);
+            fixed(S.conv_state, S.conv_bytes);
+            S.ssm_snapshot = make_buf(e, S.ssm_bytes, UZU_BUFFER_DEVICE);
+            S.conv_snapshot = make_buf(e, S.conv_bytes, UZU_BUFFER_DEVICE);
+            break;
+        }
         case MixWindowAttention:
         case MixRetention:
         case MixSideBySide: {        // a layer may hold both: a per-token cache for the attention and an f32 [heads, dim, vdim] state for the retention
@@ -1093,10 +1144,10 @@ static void create_state_and_scratch(uzu_engine* e) {
     e->max_context = max_ctx;
     const uint32_t rows_total = max_ctx + MAX_ROWS;
     const bool sparse = (uzu_context_device_capabilities(e->ctx) & UZU_CAP_SPARSE_BUFFERS) != 0;
-    e->state.resize(e->layers.size());
+    e->state.resize(e->runs.size());
     uint32_t max_qkv = 0, max_qd = 0, max_f = 0, max_proj = 0, max_vd = 0, max_heads = 0, max_hd = 0;
-    for (size_t i = 0; i < e->layers.size(); ++i) {
-        Layer& L = e->layers[i];
+    for (size_t i = 0; i < e->runs.size(); ++i) {
+        Layer& L = e->layers[e->runs[i]];
         alloc_layer_state(e, L, e->state[i], rows_total, sparse, false);
         max_f = std::max(max_f, L.hidden_dim);
         if (L.kind == MixAttention) {
@@ -1187,8 +1238,8 @@ static void create_state_and_scratch(uzu_engine* e) {
 static void alloc_sequence_state(uzu_engine* e, std::vector<LayerState>& st) {
     const uint32_t rows_total = e->max_context + MAX_ROWS;
     const bool sparse = (uzu_context_device_capabilities(e->ctx) & UZU_CAP_SPARSE_BUFFERS) != 0;
-    st.assign(e->layers.size(), LayerState{});
-    for (size_t i = 0; i < e->layers.size(); ++i) alloc_layer_state(e, e->layers[i], st[i], rows_total, sparse, true);
+    st.assign(e->runs.size(), LayerState{});
+    for (size_t i = 0; i < e->runs.size(); ++i) alloc_layer_state(e, e->layers[e->runs[i]], st[i], rows_total, sparse, true);
 }
 
 // TransformerState::prepare (state.rs:141-172): make sure KV pages for rows [0, rows) are mapped
@@ -2243,8 +2294,8 @@ static bool has_delta(const uzu_engine* e) {
 
 // advance host-side bookkeeping after a pass over m tokens (TransformerState::encode_accept: flat, no copies)
 static void accept(uzu_engine* e, uint32_t m) {
-    for (size_t i = 0; i < e->layers.size(); ++i)
-        if (e->layers[i].is_attention) e->state[i].length += m;
+    for (size_t i = 0; i < e->runs.size(); ++i)
+        if (e->layers[e->runs[i]].is_attention) e->state[i].length += m;
     e->context_length += m;
 }
 
@@ -2492,7 +2543,7 @@ uzu_status uzu_engine_restore(uzu_engine* e) {
                 if (S.conv_state.b) cudaMemcpyAsync((void*)S.conv_state.ptr(), (void*)S.conv_snapshot.ptr(), S.conv_bytes, cudaMemcpyDeviceToDevice, s);
                 cudaMemcpyAsync((void*)S.ssm_state.ptr(), (void*)S.ssm_snapshot.ptr(), S.ssm_bytes, cudaMemcpyDeviceToDevice, s);
             }
-            if (e->layers[i].is_attention) S.length = e->snapshot_context;   // KV rows beyond the snapshot are simply overwritten (a layer may hold both)
+            if (e->layers[e->runs[i]].is_attention) S.length = e->snapshot_context;   // KV rows beyond the snapshot are simply overwritten (a layer may hold both)
         }
         cudaMemcpyAsync((void*)e->token_ids.ptr(), (void*)e->snapshot_token.ptr(), 4, cudaMemcpyDeviceToDevice, s);
         e->context_length = e->snapshot_context;
@@ -3037,14 +3088,14 @@ uzu_status uzu_engine_debug_layer_outputs(uzu_engine* e, uint32_t enable, float*
         if (!e->parallel_block) throw std::runtime_error("debug_layer_outputs: only the parallel-block family keeps an f32 residual stream");
         auto& P = e->pb;
         P.dump = enable != 0;
-        if (P.dump && !P.layer_dump.b) P.layer_dump = make_buf(e, (size_t)e->layers.size() * MAX_ROWS * e->model_dim * 4, UZU_BUFFER_DEVICE);
+        if (P.dump && !P.layer_dump.b) P.layer_dump = make_buf(e, (size_t)e->runs.size() * MAX_ROWS * e->model_dim * 4, UZU_BUFFER_DEVICE);
         const uint32_t W = e->model_dim, rows = P.dump_rows;
-        const size_t total = (size_t)e->layers.size() * rows * W;
+        const size_t total = (size_t)e->runs.size() * rows * W;
         if (out_count) *out_count = (uint32_t)total;
         if (out && total) {
             if (capacity_floats < total) throw std::runtime_error("debug_layer_outputs: output too small");
             cudaStreamSynchronize(e->ctx->stream);
-            for (size_t i = 0; i < e->layers.size(); ++i)
+            for (size_t i = 0; i < e->runs.size(); ++i)
                 cudaMemcpy(out + i * rows * W, (void*)(P.layer_dump.ptr() + (uint64_t)i * MAX_ROWS * W * 4), (size_t)rows * W * 4, cudaMemcpyDeviceToHost);
         }
     });

@@ -1,4 +1,4 @@
-// Parallel-block families (Punilix, Gamanex) and the sequential-sublayer families (Vugipel, Vakesun) inside the host engine: configuration, weights, scratch and the encoding of one pass.
+// Parallel-block families (Punilix, Gamanex) and the sequential-sublayer families (Vugipel, Vakesun, Relidra) inside the host engine: configuration, weights, scratch and the encoding of one pass.
 // Included by engine.cu; the pass driver, the state / cache manager, sampling, CUDA-graph decode and the sequence slots are the engine's own.
 //
 //   x = embed[token]                                                      (f32 residual stream)
@@ -6,6 +6,7 @@
 //   Gamanex layer:  h1 = rms(x) n1, h2 = rms(x) n2;  x <- x + ls1 sigmoid(G1 h1 + b1) mixer(h1) + ls2 sigmoid(G2 h2 + b2) mlp(h2)
 //   Vugipel layer:  x <- x + mixer(rms(x) (1 + n1));  x <- x + mlp(rms(x) (1 + n2))     (Layer::sequential)
 //   Vakesun layer:  x <- x + m post1(mixer(pre1(x)));  x <- x + m post2(mlp(pre2(x)));  x <- x + m rms(token input(x))    (Layer::sandwich)
+//   Relidra layer:  u = sum_s in_s x_s;  x_t <- sum_s mix_st x_s + out_t sublayer(norm(u)), for the mixer and then the feed-forward (Layer::streamed)
 //   logits = cap * tanh(head . group_rms(x) / cap)   |   logit_scale * head . rms(x)
 //
 // Both are described by the same Layer fields (a second norm, sublayer gates and a logit scale are optional parts) and encoded by the same
@@ -845,6 +846,191 @@ static void load_vakesun_model(uzu_engine* e, const Json& cfg, const std::string
     e->info.state_bytes_per_token = stb;
 }
 
+// Relidra: sequential pre-norm layers (layer norm, weight only) over a residual of several streams (hyper-connections): every sublayer reads
+// a weighted sum of the streams, and its result is added to all of them while they mix. Mixers: gated delta rule behind short causal
+// convolutions ("delta"); chunked softmax attention whose values are the unrotated keys, with biases, a half-split rotation with linearly
+// scaled frequencies, unit-RMS queries and keys and a sink per head ("attention"). Feed-forward: exact gelu, or none. A range of layers may
+// run several times with the same weights, each run with a state of its own. The readout shares the embedding table.
+// config.json: "width", "vocab", "norm": {"eps"}, "streams", "loop": null | {"start", "stop", "times"}, "layers": [{"type": "delta", "mixer":
+// {"heads", "kv_heads", "dim", "vdim", "conv"}} | {"type": "attention", "mixer": {"heads", "kv_heads", "dim", "vdim", "scale", "mask":
+// {"size"}, "rot": {"base", "dims", "scaling": {"factor"}}}}, each with "mlp": null | {"kind": "dense", "ff"}].
+// Tensors: embed, final.norm, l<i>.norm1 / norm2, l<i>.hc1.{in,out,mix} / hc2.*, l<i>.mix.{q,k,v (+ .conv),a,b,g,o,A_log,dt_bias,norm} |
+// l<i>.mix.{q,q.b,k,k.b,sink,o}, l<i>.mlp.{up,down}.
+static void load_relidra_model(uzu_engine* e, const Json& cfg, const std::string& dir) {
+    if (e->opts.tp_size > 1) throw std::runtime_error("tensor parallelism is not built for the parallel-block families");
+    e->parallel_block = true;
+    e->store_dt = e->opts.storage_f32 ? UZU_DT_F32 : UZU_DT_BF16;
+    const uint32_t W = e->model_dim = cfg_u32(cfg, "width");
+    const uint32_t V = e->vocab = cfg_u32(cfg, "vocab");
+    e->norm_eps = (float)cfg.at("norm").at("eps").number();
+    e->norm_groups = 1;
+    const uint32_t NS = e->streams = cfg_u32(cfg, "streams");
+    if (NS == 0 || NS > 16) throw std::runtime_error("config: streams must be in 1..16");
+    const auto& lcs = cfg.at("layers").arr;
+    uint32_t loop_start = 0, loop_stop = 0, loop_times = 1;
+    if (const Json* lp = cfg.get("loop")) {
+        if (!lp->is_null()) {
+            loop_start = cfg_u32(*lp, "start"); loop_stop = cfg_u32(*lp, "stop"); loop_times = cfg_u32(*lp, "times");
+            if (loop_start > loop_stop || loop_stop > lcs.size() || loop_times == 0 || loop_times > 256) throw std::runtime_error("config: loop must name a range of the layers and a positive number of runs");
+        }
+    }
+    for (uint32_t i = 0; i < loop_start; ++i) e->runs.push_back(i);
+    for (uint32_t t = 0; t < loop_times; ++t)
+        for (uint32_t i = loop_start; i < loop_stop; ++i) e->runs.push_back(i);
+    for (uint32_t i = loop_stop; i < lcs.size(); ++i) e->runs.push_back(i);
+    ParameterLoader pl(dir + "/model.safetensors");
+    auto layer_norm = [&](const std::string& name) {
+        Norm n;
+        n.present = true;
+        n.kind = 2;
+        n.n = W;
+        n.cfg.epsilon = e->norm_eps;
+        n.scales = upload_f32(e, read_floats(pl, name, {W}).v);
+        return n;
+    };
+    auto stream_weights = [&](const std::string& p) {
+        StreamWeights s;
+        s.read = upload_f32(e, read_floats(pl, p + "in", {NS}).v);
+        s.mix = upload_f32(e, read_floats(pl, p + "mix", {NS, NS}).v);
+        s.out = upload_f32(e, read_floats(pl, p + "out", {NS}).v);
+        return s;
+    };
+    e->pb_embed = upload_matrix(e, read_floats(pl, "embed", {V, W}).v, V, W);
+    e->pb_head = e->pb_embed;        // the readout multiplies with the embedding table itself
+    e->pb_out_norm = layer_norm("final.norm");
+    std::vector<uint64_t> wbytes(lcs.size(), 0), kvb(lcs.size(), 0), stb(lcs.size(), 0);
+    e->layers.resize(lcs.size());
+    for (size_t i = 0; i < lcs.size(); ++i) {
+        const Json& lc = lcs[i];
+        Layer& L = e->layers[i];
+        const std::string p = "l" + std::to_string(i) + ".";
+        L.sequential = true;
+        L.streamed = true;
+        L.pre_mixer = layer_norm(p + "norm1");
+        L.mixer_streams = stream_weights(p + "hc1.");
+        const std::string type = lc.at("type").str;
+        const Json& mc = lc.at("mixer");
+        if (type == "attention") {
+            L.kind = MixWindowAttention;
+            L.is_attention = true;
+            WindowAttentionLayer& A = L.wa;
+            A.heads = cfg_u32(mc, "heads");
+            A.kv_heads = cfg_u32(mc, "kv_heads");
+            A.dim = cfg_u32(mc, "dim");
+            A.vdim = cfg_u32(mc, "vdim");
+            A.scale = (float)mc.at("scale").number();
+            A.unit_rms = true;
+            if (A.heads == 0 || A.kv_heads == 0 || A.heads % A.kv_heads || A.dim == 0 || A.dim > 512) throw std::runtime_error(p + "mix: kv_heads must divide heads, the head size must be in 1..512");
+            if (A.vdim != A.dim) throw std::runtime_error(p + "mix: the values are the keys, vdim must equal dim");
+            if (const Json* mk = mc.get("mask")) {
+                if (!mk->is_null()) {
+                    A.chunk = cfg_u32(*mk, "size");
+                    if (A.chunk == 0) throw std::runtime_error(p + "mix: mask.size must be positive");
+                }
+            }
+            if (const Json* rot = mc.get("rot")) {
+                if (!rot->is_null() && cfg_u32(*rot, "dims")) {
+                    RopeCfg rc;
+                    rc.kind = 3;
+                    rc.base = (float)rot->at("base").number();
+                    rc.head_dim = cfg_u32(*rot, "dims");
+                    rc.max_sequence_length = 0xFFFFFFFFu;
+                    if (rc.head_dim % 2 || rc.head_dim > A.dim) throw std::runtime_error(p + "mix: rot.dims must be even and at most dim");
+                    const Json* sc = rot->get("scaling");
+                    if (sc && !sc->is_null()) rc.scaling_factor = (float)sc->at("factor").number();
+                    if (!(rc.scaling_factor > 0.0f)) throw std::runtime_error(p + "mix: rot.scaling.factor must be positive");
+                    int idx = -1;
+                    for (size_t r = 0; r < e->ropes.size(); ++r)
+                        if (e->ropes[r] == rc) idx = (int)r;
+                    if (idx < 0) { e->ropes.push_back(rc); idx = (int)e->ropes.size() - 1; }
+                    A.rope_index = idx;
+                    A.rot_halves = true;
+                }
+            }
+            const uint32_t qn = A.heads * A.dim, kn = A.kv_heads * A.dim;
+            std::vector<float> in, bias;
+            append(in, read_floats(pl, p + "mix.q", {qn, W}));
+            append(in, read_floats(pl, p + "mix.k", {kn, W}));
+            append(bias, read_floats(pl, p + "mix.q.b", {qn}));
+            append(bias, read_floats(pl, p + "mix.k.b", {kn}));
+            A.q_offset = 0; A.k_offset = qn; A.v_offset = qn;       // the values are the key projection itself, before norm and rotation
+            L.side_in = upload_matrix(e, in, qn + kn, W);
+            L.side_in_bias = upload_f32(e, bias);
+            A.sink = upload_f32(e, read_floats(pl, p + "mix.sink", {A.heads}).v);
+            A.out = upload_matrix(e, read_floats(pl, p + "mix.o", {W, A.heads * A.vdim}).v, W, A.heads * A.vdim);
+            wbytes[i] += L.side_in.bytes + A.out.bytes;
+            // rows a decode step reads: the whole context, or half a chunk on average
+            if (A.chunk) stb[i] += (uint64_t)(A.chunk + 1) / 2 * 2 * kn * storage_size(e->store_dt);
+            else kvb[i] += (uint64_t)2 * kn * storage_size(e->store_dt);
+        } else if (type == "delta") {
+            L.kind = MixGatedDelta;
+            L.is_attention = false;
+            GatedDeltaLayer& D = L.dr;
+            D.heads = cfg_u32(mc, "heads");
+            D.kv_heads = cfg_u32(mc, "kv_heads");
+            D.dim = cfg_u32(mc, "dim");
+            D.vdim = cfg_u32(mc, "vdim");
+            D.taps = cfg_u32(mc, "conv");
+            if (D.heads == 0 || D.kv_heads == 0 || D.heads % D.kv_heads || D.dim == 0 || D.dim > 1024 || D.vdim == 0 || D.vdim > 4096 || D.taps == 0)
+                throw std::runtime_error(p + "mix: kv_heads must divide heads, dim must be in 1..1024, vdim in 1..4096, conv positive");
+            const uint32_t kd = D.kv_heads * D.dim, vn = D.heads * D.vdim;
+            std::vector<float> in, conv;
+            append(in, read_floats(pl, p + "mix.q", {kd, W}));
+            append(in, read_floats(pl, p + "mix.k", {kd, W}));
+            append(in, read_floats(pl, p + "mix.v", {vn, W}));
+            append(in, read_floats(pl, p + "mix.g", {vn, W}));
+            append(in, read_floats(pl, p + "mix.a", {D.heads, W}));
+            append(in, read_floats(pl, p + "mix.b", {D.heads, W}));
+            D.gate_offset = 2 * kd + vn; D.a_offset = D.gate_offset + vn; D.b_offset = D.a_offset + D.heads;
+            D.in = upload_matrix(e, in, D.b_offset + D.heads, W);
+            append(conv, read_floats(pl, p + "mix.q.conv", {kd, D.taps}));
+            append(conv, read_floats(pl, p + "mix.k.conv", {kd, D.taps}));
+            append(conv, read_floats(pl, p + "mix.v.conv", {vn, D.taps}));
+            D.conv = upload_f32(e, conv);
+            D.a_log = upload_f32(e, read_floats(pl, p + "mix.A_log", {D.heads}).v);
+            D.dt_bias = upload_f32(e, read_floats(pl, p + "mix.dt_bias", {D.heads}).v);
+            {
+                const HostTensor nw = read_floats(pl, p + "mix.norm", {D.vdim});
+                std::vector<float> rep;
+                for (uint32_t h = 0; h < D.heads; ++h) append(rep, nw);
+                D.norm_weight = upload_f32(e, rep);
+            }
+            D.out = upload_matrix(e, read_floats(pl, p + "mix.o", {W, vn}).v, W, vn);
+            wbytes[i] += D.in.bytes + D.out.bytes;
+            stb[i] += 2ull * D.heads * D.vdim * D.dim4() * 4 + (uint64_t)D.taps * D.channels() * 4;
+        } else {
+            throw std::runtime_error("layer type '" + type + "' is not known to the Relidra family");
+        }
+        GatedMlp& M = L.gmlp;
+        const Json* ml = lc.get("mlp");
+        if (!ml || ml->is_null()) continue;
+        L.pre_mlp = layer_norm(p + "norm2");
+        L.mlp_streams = stream_weights(p + "hc2.");
+        const std::string kind = ml->at("kind").str;
+        if (kind != "dense") throw std::runtime_error("mlp kind '" + kind + "' is not known to the Relidra family");
+        M.kind = GatedMlp::Dense;
+        M.unit = GatedMlp::GeluExact;
+        M.f = cfg_u32(*ml, "ff");
+        if (M.f == 0) throw std::runtime_error(p + "mlp: ff must be positive");
+        M.gate_up = upload_matrix(e, read_floats(pl, p + "mlp.up", {M.f, W}).v, M.f, W);
+        M.down = upload_matrix(e, read_floats(pl, p + "mlp.down", {W, M.f}).v, W, M.f);
+        wbytes[i] += M.gate_up.bytes + M.down.bytes;
+    }
+    pl.assert_all_validated();
+    e->info.model_dim = W;
+    e->info.hidden_dim = 0;
+    e->info.vocab_size = V;
+    e->info.num_layers = (uint32_t)e->layers.size();
+    e->info.weight_bytes_per_token = e->pb_head.bytes;
+    for (uint32_t i : e->runs) {       // a layer that runs several times is read and keeps a state several times
+        if (e->layers[i].is_attention) e->info.num_attention_layers++;
+        else e->info.num_delta_net_layers++;
+        e->info.weight_bytes_per_token += wbytes[i];
+        e->info.kv_bytes_per_token_per_ctx += kvb[i];
+        e->info.state_bytes_per_token += stb[i];
+    }
+}
+
 constexpr uint32_t kPromptChunks = 8;  // most key chunks of a row tile of a sigmoid-attention prompt pass
 constexpr uint32_t kSplitRows = 256;   // query rows x key splits of one latent-attention launch that leaves partial softmax states
 
@@ -874,6 +1060,16 @@ static void create_parallel_block_scratch(uzu_engine* e) {
             gated = std::max(gated, L.ml.heads * L.ml.vdim);
             kmax = std::max(kmax, L.ml.heads * L.ml.vdim);
             factor_heads = std::max(factor_heads, L.ml.heads);
+        } else if (L.kind == MixGatedDelta) {
+            const GatedDeltaLayer& D = L.dr;
+            const uint32_t kd4 = D.kv_heads * D.dim4(), vn = D.heads * D.vdim;
+            proj = std::max(proj, D.in.rows);
+            query = std::max(query, kd4);
+            wide = std::max({wide, kd4, vn});
+            mixed = std::max(mixed, vn);
+            gated = std::max(gated, vn);
+            kmax = std::max(kmax, vn);
+            factor_heads = std::max(factor_heads, D.heads);
         } else if (L.kind == MixMinGru) {
             proj = std::max(proj, L.mg.in.rows);
             gated = std::max(gated, L.mg.width);
@@ -929,10 +1125,11 @@ static void create_parallel_block_scratch(uzu_engine* e) {
     auto dev = [&](size_t bytes) { return make_buf(e, std::max<size_t>(bytes, 256), UZU_BUFFER_DEVICE); };
     const size_t R = MAX_ROWS;
     auto& P = e->pb;
-    P.resid = dev(R * W * 4);
+    P.resid = dev(R * W * 4 * std::max(1u, e->streams));
+    if (e->streams) P.stream_u = dev(R * W * 4);
     P.normed = dev(R * W * 4);
     if (second_norm) P.normed2 = dev(R * W * 4);
-    if (sandwich) P.sub_out = dev(R * W * 4);
+    if (sandwich || e->streams) P.sub_out = dev(R * W * 4);
     if (factor_heads) P.token_factors = dev(4 * R * factor_heads * 4);
     if (expand_cols) {
         P.expand_rows = std::min(expand_rows, 16384u);      // longer ranges take the kernel that reads the latents directly
@@ -982,14 +1179,46 @@ static void encode_dense(uzu_engine* e, uzu_command_buffer* cmd, const DenseMatr
 
 // A sandwich layer's short pass: the output projection's epilogue norms the product, adds it into the residual stream and norms the
 // updated stream for the next reader (both norms are Dynamic Tanh, elementwise), instead of a launch of its own after the projection.
+// A streamed layer's short pass: the epilogue mixes the streams with the product and leaves the weighted sum the next norm reads.
 static void sublayer_epilogue(uzu_engine* e, uzu_dense_linear_args& x) {
     auto& P = e->pb;
+    if (const StreamWeights* s = P.fused_streams) {
+        x.d = P.sub_out.ptr(); x.accumulate = 0;       // (not written)
+        x.streams = e->streams;
+        x.stream_x = P.resid.ptr(); x.stream_mix = s->mix.ptr(); x.stream_out = s->out.ptr(); x.stream_in = P.fused_read; x.stream_u = P.stream_u.ptr();
+        return;
+    }
     if (!P.fused_post) return;
     x.d = P.resid.ptr(); x.accumulate = 0;
     x.post_weight = P.fused_post->scales.ptr(); x.post_bias = P.fused_post->bias.ptr(); x.post_alpha = P.fused_post->alpha; x.post_mult = P.fused_mult;
     if (P.fused_reader) {
         x.next_out = P.normed.ptr(); x.next_weight = P.fused_reader->scales.ptr(); x.next_bias = P.fused_reader->bias.ptr(); x.next_alpha = P.fused_reader->alpha;
     }
+}
+
+static void set_norm(uzu_norm_add_args& a, const Norm& n, bool next) {
+    if (next) { a.next_kind = n.kind; a.next_weight = n.scales.ptr(); a.next_bias = n.bias.ptr(); a.next_alpha = n.alpha; }
+    else { a.kind = n.kind; a.weight = n.scales.ptr(); a.bias = n.bias.ptr(); a.alpha = n.alpha; }
+}
+
+// A sublayer's first product: its A rows are the normed input. A streamed layer's short pass norms them inside the product where that can be
+// done (and in a launch of its own otherwise); its long pass may have left them as bf16.
+static void sublayer_input(uzu_engine* e, uzu_command_buffer* cmd, uzu_dense_linear_args& x) {
+    auto& P = e->pb;
+    const uint32_t W = e->model_dim;
+    x.a = P.normed.ptr(); x.lda = W;
+    if (P.normed_bf16) { x.a_bf16 = 1; return; }
+    if (!P.input_norm) return;
+    x.a = P.stream_u.ptr();
+    if (dense_rows_takes_norm(x)) {
+        x.a_norm_weight = P.input_norm->scales.ptr(); x.a_norm_epsilon = e->norm_eps;
+        return;
+    }
+    uzu_norm_add_args a{};
+    a.input = P.stream_u.ptr(); a.output = P.normed.ptr(); a.rows = x.m; a.n = W; a.in_stride = W; a.epsilon = e->norm_eps;
+    set_norm(a, *P.input_norm, false);
+    uzu_norm_add_encode(cmd, &a);
+    x.a = P.normed.ptr();
 }
 
 // x += A . W^T: the sublayers' output projections add straight into the residual stream. With a sublayer gate the product is first
@@ -1073,7 +1302,7 @@ static void encode_side_by_side(uzu_engine* e, uzu_command_buffer* cmd, const La
     const uint64_t dyn = pc.dynamic ? e->decode_state.ptr() : 0;
     {
         uzu_dense_linear_args x = dense_args(e, L.side_in, P.normed.ptr(), m, P.proj.ptr());
-        x.lda = e->model_dim;
+        sublayer_input(e, cmd, x);
         if (L.side_in_bias.b) x.bias = L.side_in_bias.ptr();
         uzu_dense_linear_encode(cmd, &x);
     }
@@ -1091,17 +1320,18 @@ static void encode_side_by_side(uzu_engine* e, uzu_command_buffer* cmd, const La
         pa.v_cosines = vcos; pa.v_sines = vsin; pa.v_pairs = v_pairs; pa.dynamic_position = dyn;
         pa.rows = m; pa.heads = A.heads; pa.kv_heads = A.kv_heads; pa.dim = A.dim; pa.vdim = A.vdim;
         pa.q_stride = pa.k_stride = pa.v_stride = ld; pa.prefix = S.length; pa.cache_dt = e->store_dt; pa.epsilon = e->norm_eps;
-        pa.rot_halves = A.rot_halves ? 1 : 0;
+        pa.rot_halves = A.rot_halves ? 1 : 0; pa.unit_rms = A.unit_rms ? 1 : 0;
         uzu_window_attention_prepare_encode(cmd, &pa);
         uzu_window_attention_args aa{};
         aa.query = P.query.ptr(); aa.keys = S.keys; aa.values = S.values; aa.out = P.mixed.ptr(); aa.dynamic_position = dyn;
         aa.head_temp = A.head_temp.ptr(); aa.v_cosines = vcos; aa.v_sines = vsin; aa.v_pairs = v_pairs;
         aa.rows = m; aa.heads = A.heads; aa.kv_heads = A.kv_heads; aa.dim = A.dim; aa.vdim = A.vdim; aa.prefix = S.length; aa.cache_dt = e->store_dt;
-        aa.window = A.window; aa.keep_first = A.keep_first; aa.scale = A.scale; aa.softcap = A.softcap;
+        aa.window = A.window; aa.keep_first = A.keep_first; aa.chunk = A.chunk; aa.scale = A.scale; aa.softcap = A.softcap; aa.sinks = A.sink.ptr();
         {   // few query rows: cut the visible keys (in tiles of 16) so that about eight small CTAs per SM run (the captured step sizes the
             // cut for the largest context its graph serves; a window bounds it)
             uint32_t bound = pc.dynamic ? attention_bucket(S.length + m) : S.length + m;
             if (A.window) bound = std::min(bound, A.window + A.keep_first);
+            if (A.chunk) bound = std::min(bound, A.chunk + A.keep_first);
             const uint32_t tiles = (bound + 15) / 16;
             const uint32_t want = std::max(1u, 8u * (uint32_t)e->ctx->sm_count / std::max(1u, m * A.heads));
             aa.splits = std::min({tiles, want, kSplitRows / std::max(1u, m), 128u});
@@ -1134,6 +1364,43 @@ static void encode_side_by_side(uzu_engine* e, uzu_command_buffer* cmd, const La
         if (!L.has_window_attention()) sublayer_epilogue(e, x);
         uzu_dense_linear_encode(cmd, &x);
     }
+}
+
+// h [m, W] -> gated delta rule: one stacked projection [q | k | v | output gate | decay | step size], then one launch for a single token, or
+// the convolutions and gates of all tokens, the recurrence, and the per-head norm with its silu gate; the output projection follows
+static void encode_gated_delta(uzu_engine* e, uzu_command_buffer* cmd, const Layer& L, LayerState& S, const PassCtx& pc) {
+    const GatedDeltaLayer& D = L.dr;
+    auto& P = e->pb;
+    const uint32_t m = pc.m, ld = D.in.rows, vn = D.heads * D.vdim;
+    {
+        uzu_dense_linear_args x = dense_args(e, D.in, P.normed.ptr(), m, P.proj.ptr());
+        sublayer_input(e, cmd, x);
+        uzu_dense_linear_encode(cmd, &x);
+    }
+    uzu_delta_prepare_args pa{};
+    pa.proj = P.proj.ptr(); pa.conv = D.conv.ptr(); pa.ring = S.conv_state.ptr(); pa.a_log = D.a_log.ptr(); pa.dt_bias = D.dt_bias.ptr();
+    pa.dynamic_position = pc.dynamic ? e->decode_state.ptr() : 0;
+    pa.rows = m; pa.heads = D.heads; pa.kv_heads = D.kv_heads; pa.dim = D.dim; pa.vdim = D.vdim; pa.taps = D.taps; pa.stride = ld;
+    pa.a_offset = D.a_offset; pa.b_offset = D.b_offset; pa.prefix = e->context_length;
+    if (m == 1) {
+        uzu_gated_delta_step_args sa{};
+        sa.prep = pa; sa.state = S.ssm_state.ptr(); sa.norm = D.norm_weight.ptr(); sa.out = P.gated_mix.ptr();
+        sa.gate_offset = D.gate_offset; sa.epsilon = e->norm_eps;
+        uzu_gated_delta_step_encode(cmd, &sa);
+    } else {
+        pa.q = P.query.ptr(); pa.k = P.lat_wide.ptr(); pa.v = P.mixed.ptr();
+        pa.decay = P.token_factors.ptr(); pa.beta = P.token_factors.ptr() + (uint64_t)MAX_ROWS * D.heads * 4;
+        uzu_delta_prepare_encode(cmd, &pa);
+        uzu_gated_delta_args ga{};
+        ga.prep = pa; ga.state = S.ssm_state.ptr(); ga.out = P.wide.ptr();
+        uzu_gated_delta_encode(cmd, &ga);
+        uzu_head_norm_gate_args na{};
+        na.x = P.wide.ptr(); na.scales = D.norm_weight.ptr(); na.gate = P.proj.ptr() + (uint64_t)D.gate_offset * 4; na.out = P.gated_mix.ptr();
+        na.rows = m; na.heads = D.heads; na.dim = D.vdim; na.x_stride = vn; na.gate_stride = ld; na.out_stride = vn; na.normalize = 1;
+        na.epsilon = e->norm_eps; na.gate_op = 1;
+        uzu_head_norm_gate_encode(cmd, &na);
+    }
+    encode_into_residual(e, cmd, D.out, P.gated_mix.ptr(), vn, m);
 }
 
 // h [m, W] -> the mixer's output is added to the residual stream
@@ -1315,6 +1582,23 @@ static void encode_gated_mlp(uzu_engine* e, uzu_command_buffer* cmd, const Layer
         encode_into_residual(e, cmd, M.down, P.proj2.ptr(), ld, m, &L.mlp_gate, P.proj2.ptr(), ld, 2);
         return;
     }
+    if (M.kind == GatedMlp::Dense && M.unit == GatedMlp::GeluExact) {
+        uzu_dense_linear_args up = dense_args(e, M.gate_up, h, m, P.act.ptr());
+        up.d_op = 1;
+        sublayer_input(e, cmd, up);
+        // long passes keep the unit's rows in bf16, as the down projection's A rows (the precision its operand has anyway)
+        uzu_dense_linear_args dn = dense_args(e, M.down, P.act.ptr(), m, P.sub_out.ptr());
+        dn.lda = M.f;
+        up.d_bf16 = P.redirect && dense_umma_applicable(up) && dense_umma_applicable(dn) ? 1 : 0;
+        uzu_dense_linear_encode(cmd, &up);
+        if (up.d_bf16) {
+            dn.a_bf16 = 1;
+            uzu_dense_linear_encode(cmd, &dn);
+        } else {
+            encode_into_residual(e, cmd, M.down, P.act.ptr(), M.f, m);
+        }
+        return;
+    }
     if (M.kind == GatedMlp::Dense) {
         uzu_dense_linear_args up = gate_up_args();
         uzu_dense_linear_encode(cmd, &up);
@@ -1375,13 +1659,9 @@ static void encode_mixer(uzu_engine* e, uzu_command_buffer* cmd, const Layer& L,
     else if (L.kind == MixSigmoidAttention) encode_sigmoid_attention(e, cmd, L, S, pc);
     else if (L.kind == MixMinGru) encode_min_gru(e, cmd, L, S, pc);
     else if (L.kind == MixMlstm) encode_mlstm(e, cmd, L, S, pc);
+    else if (L.kind == MixGatedDelta) encode_gated_delta(e, cmd, L, S, pc);
     else if (L.has_window_attention() || L.has_retention()) encode_side_by_side(e, cmd, L, S, pc);
     else encode_latent_attention(e, cmd, L, S, pc);
-}
-
-static void set_norm(uzu_norm_add_args& a, const Norm& n, bool next) {
-    if (next) { a.next_kind = n.kind; a.next_weight = n.scales.ptr(); a.next_bias = n.bias.ptr(); a.next_alpha = n.alpha; }
-    else { a.kind = n.kind; a.weight = n.scales.ptr(); a.bias = n.bias.ptr(); a.alpha = n.alpha; }
 }
 
 // A sandwich layer: x <- x + mult * post(sublayer(pre(x))) for the mixer, the feed-forward (if any) and the token input (if any). A
@@ -1443,6 +1723,75 @@ static void encode_sandwich_layer(uzu_engine* e, uzu_command_buffer* cmd, const 
     }
 }
 
+// A pass over streamed layers. Between two sublayers the residual's copies take the first one's result and the second one's input is formed:
+//   short passes (< 128 rows, at most 4 streams): the first sublayer's last product does it as its epilogue (leaving the weighted sum of the
+//   copies), the second's first product norms its rows as it stages them: no launch between the two;
+//   long passes: the products run on tcgen05, and one launch (stream_mix) mixes, sums and norms, a row per CTA.
+// Without a reader (the last layer) the sum of the streams stays in P.stream_u for the readout.
+static void encode_streamed_layers(uzu_engine* e, uzu_command_buffer* cmd, const PassCtx& pc, bool dump) {
+    auto& P = e->pb;
+    const uint32_t m = pc.m, W = e->model_dim;
+    const bool fuse = m < 128 && e->streams <= 4;
+    struct Sublayer { const Layer* L; const StreamWeights* streams; const Norm* norm; const DenseMatrix* first; };
+    auto mixer_of = [&](size_t run) -> Sublayer {
+        const Layer& L = e->layers[e->runs[run]];
+        return {&L, &L.mixer_streams, &L.pre_mixer, L.kind == MixGatedDelta ? &L.dr.in : &L.side_in};
+    };
+    auto mlp_of = [&](size_t run) -> Sublayer {
+        const Layer& L = e->layers[e->runs[run]];
+        return {&L, &L.mlp_streams, &L.pre_mlp, &L.gmlp.gate_up};
+    };
+    // one launch: begin (from the embedding) or take `done`'s result in, then what `next` reads
+    auto mix = [&](const StreamWeights* done, const Sublayer* next) {
+        uzu_stream_mix_args a{};
+        a.x = P.resid.ptr(); a.rows = m; a.n = W; a.streams = e->streams; a.epsilon = e->norm_eps;
+        if (done) { a.y = P.sub_out.ptr(); a.mix = done->mix.ptr(); a.out = done->out.ptr(); }
+        else { a.token_ids = e->token_ids.ptr(); a.table = e->pb_embed.w.ptr(); a.table_dt = e->store_dt; a.vocab = e->vocab; }
+        if (next) a.read = next->streams->read.ptr();
+        if (fuse || !next) {
+            a.u = P.stream_u.ptr();
+        } else {
+            P.normed_bf16 = dense_umma_applicable(dense_args(e, *next->first, P.normed.ptr(), m, P.proj.ptr()));
+            a.weight = next->norm->scales.ptr(); a.output = P.normed.ptr(); a.output_bf16 = P.normed_bf16 ? 1 : 0;
+        }
+        uzu_stream_mix_encode(cmd, &a);
+    };
+    auto sublayer = [&](const Sublayer& s, const Sublayer* next, auto&& encode) {
+        if (fuse) { P.input_norm = s.norm; P.fused_streams = s.streams; P.fused_read = next ? next->streams->read.ptr() : 0; }
+        else P.redirect = true;
+        encode();
+        P.input_norm = nullptr; P.fused_streams = nullptr; P.fused_read = 0; P.redirect = false; P.normed_bf16 = false;
+        if (!fuse) mix(s.streams, next);
+    };
+    if (e->runs.empty()) {
+        mix(nullptr, nullptr);
+        return;
+    }
+    {
+        const Sublayer first = mixer_of(0);
+        mix(nullptr, &first);
+    }
+    for (size_t i = 0; i < e->runs.size(); ++i) {
+        const Layer& L = e->layers[e->runs[i]];
+        const bool has_mlp = L.gmlp.kind != GatedMlp::None, last = i + 1 == e->runs.size();
+        Sublayer following{};
+        if (!last) following = mixer_of(i + 1);
+        const Sublayer* next = last ? nullptr : &following;
+        if (has_mlp) {
+            const Sublayer ff = mlp_of(i);
+            sublayer(mixer_of(i), &ff, [&] { encode_mixer(e, cmd, L, e->state[i], pc); });
+            sublayer(ff, next, [&] { encode_gated_mlp(e, cmd, L, pc, P.normed.ptr()); });
+        } else {
+            sublayer(mixer_of(i), next, [&] { encode_mixer(e, cmd, L, e->state[i], pc); });
+        }
+        if (dump) {
+            uzu_stream_mix_args a{};
+            a.x = P.resid.ptr(); a.rows = m; a.n = W; a.streams = e->streams; a.u = P.layer_dump.ptr() + (uint64_t)i * MAX_ROWS * W * 4;
+            uzu_stream_mix_encode(cmd, &a);
+        }
+    }
+}
+
 static void encode_parallel_block_decoder(uzu_engine* e, uzu_command_buffer* cmd, const PassCtx& pc, uint32_t row_begin, uint32_t row_end) {
     const uint32_t m = pc.m, W = e->model_dim;
     auto& P = e->pb;
@@ -1450,8 +1799,14 @@ static void encode_parallel_block_decoder(uzu_engine* e, uzu_command_buffer* cmd
         cmd->record_error(UZU_ERROR_UNSUPPORTED, "speculation passes are not built for the parallel-block families");
         return;
     }
-    uzu_embedding_f32_scaled_encode(cmd, e->token_ids.ptr(), e->pb_embed.w.ptr(), e->store_dt, P.resid.ptr(), m, e->vocab, W, e->input_scale);
     const bool dump = P.dump && !pc.dynamic && P.layer_dump.b;
+    if (e->streams) {
+        encode_streamed_layers(e, cmd, pc, dump);
+        if (dump) P.dump_rows = m;
+        encode_parallel_block_readout(e, cmd, row_begin, row_end);
+        return;
+    }
+    uzu_embedding_f32_scaled_encode(cmd, e->token_ids.ptr(), e->pb_embed.w.ptr(), e->store_dt, P.resid.ptr(), m, e->vocab, W, e->input_scale);
     bool normed_ready = false;
     for (size_t i = 0; i < e->layers.size(); ++i) {
         Layer& L = e->layers[i];
@@ -1486,22 +1841,25 @@ static void encode_parallel_block_readout(uzu_engine* e, uzu_command_buffer* cmd
     if (row_end <= row_begin) return;
     const uint32_t rows = row_end - row_begin, W = e->model_dim;
     auto& P = e->pb;
-    if (e->pb_out_norm.present) {
+    const uint64_t rows_in = (e->streams ? P.stream_u : P.resid).ptr() + (uint64_t)row_begin * W * 4;
+    uzu_dense_linear_args x = dense_args(e, e->pb_head, P.normed_rows.ptr(), rows, P.logits_f32.ptr());
+    x.lda = W;
+    if (e->has_logit_scale) x.scale = e->logit_scale;
+    uzu_dense_linear_args direct = x;
+    direct.a = rows_in;
+    if (e->pb_out_norm.present && e->pb_out_norm.kind == 2 && dense_rows_takes_norm(direct)) {      // few rows: normed inside the readout product
+        x.a = rows_in; x.a_norm_weight = e->pb_out_norm.scales.ptr(); x.a_norm_epsilon = e->norm_eps;
+    } else if (e->pb_out_norm.present) {
         uzu_norm_add_args a{};
-        a.input = P.resid.ptr() + (uint64_t)row_begin * W * 4; a.output = P.normed_rows.ptr(); a.rows = rows; a.n = W; a.in_stride = W; a.epsilon = e->norm_eps;
+        a.input = rows_in; a.output = P.normed_rows.ptr(); a.rows = rows; a.n = W; a.in_stride = W; a.epsilon = e->norm_eps;
         set_norm(a, e->pb_out_norm, false);
         uzu_norm_add_encode(cmd, &a);
     } else {
         uzu_group_rms_norm_args na{};
-        na.input = P.resid.ptr() + (uint64_t)row_begin * W * 4; na.scales = e->pb_final_norm.ptr(); na.output = P.normed_rows.ptr();
+        na.input = rows_in; na.scales = e->pb_final_norm.ptr(); na.output = P.normed_rows.ptr();
         na.rows = rows; na.n = W; na.groups = e->norm_groups; na.in_stride = W; na.out_stride = W; na.epsilon = e->norm_eps;
         uzu_group_rms_norm_encode(cmd, &na);
     }
-    {
-        uzu_dense_linear_args x = dense_args(e, e->pb_head, P.normed_rows.ptr(), rows, P.logits_f32.ptr());
-        x.lda = W;
-        if (e->has_logit_scale) x.scale = e->logit_scale;
-        uzu_dense_linear_encode(cmd, &x);
-    }
+    uzu_dense_linear_encode(cmd, &x);
     uzu_logit_cap_f32_encode(cmd, P.logits_f32.ptr(), e->logits.ptr(), rows * e->vocab, e->logit_soft_cap, e->has_logit_soft_cap);
 }

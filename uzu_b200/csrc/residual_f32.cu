@@ -1,5 +1,5 @@
-// Glue kernels of the parallel-block family (f32 residual stream): grouped RMS norm, norm (RMS or Dynamic Tanh) with residual add and
-// the next norm, embedding rows into f32, the token-gated gelu unit, the clamped gated unit, tanh, residual add, logit cap, and the routers (by table or by the largest logits: expert-sorted pair lists + weighted, optionally
+// Glue kernels of the parallel-block family (f32 residual stream): grouped RMS norm, norm (RMS, Dynamic Tanh or layer norm) with residual add and
+// the next norm, a residual kept as several mixed streams with the next layer norm, embedding rows into f32, the token-gated gelu unit, the clamped gated unit, tanh, residual add, logit cap, and the routers (by table or by the largest logits: expert-sorted pair lists + weighted, optionally
 // gated combine). Everything is f32 arithmetic.
 #include "common.cuh"
 
@@ -47,8 +47,8 @@ __global__ void __launch_bounds__(256) group_rms_norm_kernel(const uzu_group_rms
 
 // One CTA per row. RMS norm: the row's sum of squares first; Dynamic Tanh is elementwise. With a residual the normed row is added into
 // it (times mult) and the updated row can be normed again for the next sublayer; a second RMS norm takes a second sum over the row.
-__device__ __forceinline__ float norm_add_value(uint32_t kind, float x, float inv, float alpha, const float* w, const float* b, uint32_t i) {
-    float v = kind == 1 ? tanhf(alpha * x) : x * inv;
+__device__ __forceinline__ float norm_add_value(uint32_t kind, float x, float mean, float inv, float alpha, const float* w, const float* b, uint32_t i) {
+    float v = kind == 1 ? tanhf(alpha * x) : (x - mean) * inv;
     if (w) v *= w[i];
     if (b) v += b[i];
     return v;
@@ -62,13 +62,13 @@ __global__ void __launch_bounds__(256) norm_add_elementwise_kernel(const uzu_nor
     if (i >= a.n) return;
     const float* w = reinterpret_cast<const float*>(a.weight);
     const float* b = reinterpret_cast<const float*>(a.bias);
-    const float v = norm_add_value(1, reinterpret_cast<const float*>(a.input)[(size_t)row * a.in_stride + i], 1.0f, a.alpha, w, b, i);
+    const float v = norm_add_value(1, reinterpret_cast<const float*>(a.input)[(size_t)row * a.in_stride + i], 0.0f, 1.0f, a.alpha, w, b, i);
     float* out = a.output ? reinterpret_cast<float*>(a.output) + (size_t)row * a.n : nullptr;
     if (!a.residual) { out[i] = v; return; }
     float* res = reinterpret_cast<float*>(a.residual) + (size_t)row * a.n;
     const float x = fmaf(a.mult, v, res[i]);
     res[i] = x;
-    if (out) out[i] = norm_add_value(1, x, 1.0f, a.next_alpha, reinterpret_cast<const float*>(a.next_weight), reinterpret_cast<const float*>(a.next_bias), i);
+    if (out) out[i] = norm_add_value(1, x, 0.0f, 1.0f, a.next_alpha, reinterpret_cast<const float*>(a.next_weight), reinterpret_cast<const float*>(a.next_bias), i);
 }
 
 // One CTA per row; a thread keeps up to KEEP of the row's elements (input, weights, residual) in registers, all requested before the
@@ -98,47 +98,159 @@ __global__ void __launch_bounds__(256) norm_add_kernel(const uzu_norm_add_args a
         nwv[j] = (ok && nw) ? nw[i] : 1.0f;
         nbv[j] = (ok && nb) ? nb[i] : 0.0f;
     }
-    float inv = 1.0f;
-    if (a.kind == 0) {
+    float inv = 1.0f, mean = 0.0f;
+    if (a.kind == 2) {
+        float s = 0.0f;
+#pragma unroll
+        for (int j = 0; j < KEEP; ++j) s += x[j];
+        for (uint32_t i = threadIdx.x + KEEP * blockDim.x; i < a.n; i += blockDim.x) s += in[i];
+        mean = block_sum(s, red) / (float)a.n;
+    }
+    if (a.kind != 1) {
         float ss = 0.0f;
 #pragma unroll
-        for (int j = 0; j < KEEP; ++j) ss = fmaf(x[j], x[j], ss);
-        for (uint32_t i = threadIdx.x + KEEP * blockDim.x; i < a.n; i += blockDim.x) ss = fmaf(in[i], in[i], ss);
+        for (int j = 0; j < KEEP; ++j) {
+            const float d = threadIdx.x + j * blockDim.x < a.n ? x[j] - mean : 0.0f;
+            ss = fmaf(d, d, ss);
+        }
+        for (uint32_t i = threadIdx.x + KEEP * blockDim.x; i < a.n; i += blockDim.x) { const float d = in[i] - mean; ss = fmaf(d, d, ss); }
         ss = block_sum(ss, red);
         inv = 1.0f / sqrtf(ss / (float)a.n + a.epsilon);
     }
     // first norm, and the residual add
-    float ss2 = 0.0f;
+    float s2 = 0.0f, ss2 = 0.0f;
 #pragma unroll
     for (int j = 0; j < KEEP; ++j) {
         const uint32_t i = threadIdx.x + j * blockDim.x;
-        float v = (a.kind == 1 ? tanhf(a.alpha * x[j]) : x[j] * inv) * wv[j] + bv[j];
+        float v = (a.kind == 1 ? tanhf(a.alpha * x[j]) : (x[j] - mean) * inv) * wv[j] + bv[j];
         if (res) v = fmaf(a.mult, v, rv[j]);
         x[j] = v;
         if (i < a.n) {
             ss2 = fmaf(v, v, ss2);
+            s2 += v;
             if (res) res[i] = v;
             else out[i] = v;
         }
     }
     for (uint32_t i = threadIdx.x + KEEP * blockDim.x; i < a.n; i += blockDim.x) {
-        float v = norm_add_value(a.kind, in[i], inv, a.alpha, w, b, i);
+        float v = norm_add_value(a.kind, in[i], mean, inv, a.alpha, w, b, i);
         if (res) { v = fmaf(a.mult, v, res[i]); res[i] = v; }          // read back below by the thread that wrote it
         else out[i] = v;
         ss2 = fmaf(v, v, ss2);
+        s2 += v;
     }
     if (!res || !out) return;
-    float inv2 = 1.0f;
-    if (a.next_kind == 0) {
+    float inv2 = 1.0f, mean2 = 0.0f;
+    if (a.next_kind == 2) {         // the deviations need the mean: a second sum over the row
+        mean2 = block_sum(s2, red) / (float)a.n;
+        ss2 = 0.0f;
+#pragma unroll
+        for (int j = 0; j < KEEP; ++j) {
+            const float d = threadIdx.x + j * blockDim.x < a.n ? x[j] - mean2 : 0.0f;
+            ss2 = fmaf(d, d, ss2);
+        }
+        for (uint32_t i = threadIdx.x + KEEP * blockDim.x; i < a.n; i += blockDim.x) { const float d = res[i] - mean2; ss2 = fmaf(d, d, ss2); }
+    }
+    if (a.next_kind != 1) {
         ss2 = block_sum(ss2, red);
         inv2 = 1.0f / sqrtf(ss2 / (float)a.n + a.epsilon);
     }
 #pragma unroll
     for (int j = 0; j < KEEP; ++j) {
         const uint32_t i = threadIdx.x + j * blockDim.x;
-        if (i < a.n) out[i] = (a.next_kind == 1 ? tanhf(a.next_alpha * x[j]) : x[j] * inv2) * nwv[j] + nbv[j];
+        if (i < a.n) out[i] = (a.next_kind == 1 ? tanhf(a.next_alpha * x[j]) : (x[j] - mean2) * inv2) * nwv[j] + nbv[j];
     }
-    for (uint32_t i = threadIdx.x + KEEP * blockDim.x; i < a.n; i += blockDim.x) out[i] = norm_add_value(a.next_kind, res[i], inv2, a.next_alpha, nw, nb, i);
+    for (uint32_t i = threadIdx.x + KEEP * blockDim.x; i < a.n; i += blockDim.x) out[i] = norm_add_value(a.next_kind, res[i], mean2, inv2, a.next_alpha, nw, nb, i);
+}
+
+// One CTA per row of a residual kept as several streams: begin from the embedding, or take a sublayer's result in; then the next reader's
+// weighted sum of the streams and its layer norm. A thread keeps up to KEEP elements of that sum in registers between the passes over it.
+template <int MAXS>
+__global__ void __launch_bounds__(MAXS > 4 ? 256 : 1024) stream_mix_kernel(const uzu_stream_mix_args a) {
+    pdl_launch_dependents();
+    __shared__ float red[32], cmix[MAXS * MAXS], cout[MAXS], cread[MAXS];
+    const uint32_t row = blockIdx.x, S = a.streams;
+    for (uint32_t i = threadIdx.x; i < MAXS * MAXS; i += blockDim.x) {          // coefficients (weights: not written by the launch before)
+        const uint32_t s = i / MAXS, t = i % MAXS;
+        cmix[i] = (a.y && s < S && t < S) ? reinterpret_cast<const float*>(a.mix)[s * S + t] : 0.0f;
+        if (i < MAXS) {
+            cout[i] = (a.y && i < S) ? reinterpret_cast<const float*>(a.out)[i] : 0.0f;
+            cread[i] = i < S ? (a.read ? reinterpret_cast<const float*>(a.read)[i] : 1.0f) : 0.0f;
+        }
+    }
+    pdl_wait();
+    __syncthreads();
+    float* x = reinterpret_cast<float*>(a.x) + (size_t)row * S * a.n;
+    const float* y = a.y ? reinterpret_cast<const float*>(a.y) + (size_t)row * a.n : nullptr;
+    float* u_out = a.u ? reinterpret_cast<float*>(a.u) + (size_t)row * a.n : nullptr;
+    const uint32_t tok = a.token_ids ? reinterpret_cast<const uint32_t*>(a.token_ids)[row] : 0u;
+    auto element = [&](uint32_t i) {
+        float xs[MAXS], u = 0.0f;
+        if (a.token_ids) {
+            float e = 0.0f;
+            if (tok < a.vocab) {
+                const size_t at = (size_t)tok * a.n + i;
+                e = a.table_dt == UZU_DT_F32 ? reinterpret_cast<const float*>(a.table)[at] : __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(a.table)[at]);
+            }
+#pragma unroll
+            for (int s = 0; s < MAXS; ++s) xs[s] = e;
+        } else {
+#pragma unroll
+            for (int s = 0; s < MAXS; ++s) xs[s] = (uint32_t)s < S ? x[(size_t)s * a.n + i] : 0.0f;
+        }
+        const float yy = y ? y[i] : 0.0f;
+#pragma unroll
+        for (int t = 0; t < MAXS; ++t) {
+            if ((uint32_t)t < S) {
+                float v = xs[t];
+                if (y) {
+                    v = cout[t] * yy;
+#pragma unroll
+                    for (int s = 0; s < MAXS; ++s) v = fmaf(cmix[s * MAXS + t], xs[s], v);
+                }
+                if (y || a.token_ids) x[(size_t)t * a.n + i] = v;
+                u = fmaf(cread[t], v, u);
+            }
+        }
+        if (u_out) u_out[i] = u;
+        return u;
+    };
+    auto again = [&](uint32_t i) {          // the same sum from the streams this thread has just stored (or that nobody changed)
+        float u = 0.0f;
+        for (uint32_t t = 0; t < S; ++t) u = fmaf(cread[t], x[(size_t)t * a.n + i], u);
+        return u;
+    };
+    constexpr int KEEP = 8;
+    float u[KEEP], sum = 0.0f;
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+        const uint32_t i = threadIdx.x + j * blockDim.x;
+        u[j] = i < a.n ? element(i) : 0.0f;
+        sum += u[j];
+    }
+    for (uint32_t i = threadIdx.x + KEEP * blockDim.x; i < a.n; i += blockDim.x) sum += element(i);
+    if (!a.output) return;
+    const float mean = block_sum(sum, red) / (float)a.n;
+    float ss = 0.0f;
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+        const float d = threadIdx.x + j * blockDim.x < a.n ? u[j] - mean : 0.0f;
+        ss = fmaf(d, d, ss);
+    }
+    for (uint32_t i = threadIdx.x + KEEP * blockDim.x; i < a.n; i += blockDim.x) { const float d = again(i) - mean; ss = fmaf(d, d, ss); }
+    const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)a.n + a.epsilon);
+    const float* w = reinterpret_cast<const float*>(a.weight);
+    auto store = [&](uint32_t i, float v) {
+        v = (v - mean) * inv * w[i];
+        if (a.output_bf16) reinterpret_cast<__nv_bfloat16*>(a.output)[(size_t)row * a.n + i] = __float2bfloat16_rn(v);
+        else reinterpret_cast<float*>(a.output)[(size_t)row * a.n + i] = v;
+    };
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+        const uint32_t i = threadIdx.x + j * blockDim.x;
+        if (i < a.n) store(i, u[j]);
+    }
+    for (uint32_t i = threadIdx.x + KEEP * blockDim.x; i < a.n; i += blockDim.x) store(i, again(i));
 }
 
 template <typename TW>
@@ -477,7 +589,7 @@ void uzu_embedding_f32_encode(uzu_command_buffer* cmd, uint64_t token_ids, uint6
 
 void uzu_norm_add_encode(uzu_command_buffer* cmd, const uzu_norm_add_args* a) {
     if (!encodable(cmd, "norm_add")) return;
-    if (!a->input || (!a->residual && !a->output) || a->kind > 1 || a->next_kind > 1) {
+    if (!a->input || (!a->residual && !a->output) || a->kind > 2 || a->next_kind > 2) {
         cmd->record_error(UZU_ERROR_INVALID_ARGUMENT, "norm_add: null operand or unknown norm kind");
         return;
     }
@@ -488,6 +600,21 @@ void uzu_norm_add_encode(uzu_command_buffer* cmd, const uzu_norm_add_args* a) {
         launch(cmd, "norm_add_elementwise_kernel", norm_add_elementwise_kernel, dim3((b.n + 255) / 256, b.rows), dim3(256), 0, b);
     else
         launch(cmd, "norm_add_kernel", norm_add_kernel, dim3(b.rows), dim3(256), 0, b);
+}
+
+void uzu_stream_mix_encode(uzu_command_buffer* cmd, const uzu_stream_mix_args* a) {
+    if (!encodable(cmd, "stream_mix")) return;
+    if (!a->x || a->streams == 0 || a->streams > 16 || (a->y && (!a->mix || !a->out)) || (a->output && !a->weight) || (a->token_ids && (!a->table || a->y)) ||
+        (a->token_ids && a->table_dt != UZU_DT_BF16 && a->table_dt != UZU_DT_F32)) {
+        cmd->record_error(UZU_ERROR_INVALID_ARGUMENT, "stream_mix: null operand, more than 16 streams, or a beginning that also takes a result in");
+        return;
+    }
+    if (a->rows == 0 || a->n == 0) return;
+    const uint32_t threads = (a->n <= 2048 || a->streams > 4) ? 256 : (a->n <= 4096 ? 512 : 1024);
+    auto go = [&](auto kernel) { launch(cmd, "stream_mix_kernel", kernel, dim3(a->rows), dim3(threads), 0, *a); };
+    if (a->streams <= 2) go(stream_mix_kernel<2>);
+    else if (a->streams <= 4) go(stream_mix_kernel<4>);
+    else go(stream_mix_kernel<16>);
 }
 
 void uzu_rows_to_bf16_encode(uzu_command_buffer* cmd, uint64_t src, uint32_t src_stride, uint64_t dst, uint32_t rows, uint32_t n) {

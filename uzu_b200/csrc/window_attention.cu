@@ -1,5 +1,6 @@
 // Windowed softmax attention with kept first tokens, rotated keys AND rotated values.
-//   visibility:  key j is seen from position p when j <= p and (p - j < window or j < keep_first); kept tokens keep their true positions
+//   visibility:  key j is seen from position p when j <= p and (p - j < window or j < keep_first); kept tokens keep their true positions;
+//                with a chunk size also only from inside its own chunk, floor(j / chunk) = floor(p / chunk), counted from position 0
 //   score:       s = scale * temp[h] * q . k, then softcap * tanh(s / softcap); ordinary softmax over the visible keys
 //   rotation:    q and k turn by their position over the first 2 * rot_pairs channels (pairs (2i, 2i+1), or (i, i + rot_pairs) with
 //                rot_halves); the value of position j turns
@@ -12,7 +13,7 @@
 //                splits in a scratch: the last split to finish (a ticket per query and head) merges them in split order;
 //   attend, tensor pipe (window_attention_mma_kernel): bf16 caches and passes of >= 64 rows (described at the kernel).
 // The cache holds bf16 or f32 rows; scores, weights and sums are f32. Only the visible keys are read: a long context costs a decode
-// step window + keep_first keys.
+// step window + keep_first keys, or at most a chunk.
 #include <type_traits>
 
 #include "common.cuh"
@@ -88,9 +89,10 @@ struct Visible {
     __device__ __forceinline__ uint32_t key(uint32_t idx) const { return idx < first ? idx : lo + (idx - first); }
 };
 
-__device__ __forceinline__ Visible wa_visible(uint32_t p, uint32_t window, uint32_t keep_first) {
+__device__ __forceinline__ Visible wa_visible(uint32_t p, uint32_t window, uint32_t keep_first, uint32_t chunk) {
     Visible v;
     v.lo = (window && p + 1 > window) ? p + 1 - window : 0u;
+    if (chunk) v.lo = max(v.lo, p - p % chunk);
     v.first = min(keep_first, v.lo);
     v.total = v.first + (p + 1 - v.lo);
     return v;
@@ -115,7 +117,7 @@ __global__ void __launch_bounds__(128) window_attention_prepare_kernel(const uzu
     if (unit < a.heads) {
         const float* src = reinterpret_cast<const float*>(a.q) + (size_t)t * a.q_stride + (size_t)unit * a.dim;
         const float* sc = reinterpret_cast<const float*>(a.q_scales);
-        const float inv = sc ? wa_head_inv_rms(src, a.dim, a.epsilon, lane) : 1.0f;
+        const float inv = sc || a.unit_rms ? wa_head_inv_rms(src, a.dim, a.epsilon, lane) : 1.0f;
         float* dst = reinterpret_cast<float*>(a.query) + ((size_t)t * a.heads + unit) * a.dim;
         if (a.rot_halves) wa_rotate_row_halves<float>(src, inv, sc, dst, a.dim, a.rot_pairs, cs, sn, lane);
         else wa_rotate_row<float>(src, inv, sc, dst, a.dim, a.rot_pairs, cs, sn, lane);
@@ -123,7 +125,7 @@ __global__ void __launch_bounds__(128) window_attention_prepare_kernel(const uzu
         const uint32_t g = unit - a.heads;
         const float* src = reinterpret_cast<const float*>(a.k) + (size_t)t * a.k_stride + (size_t)g * a.dim;
         const float* sc = reinterpret_cast<const float*>(a.k_scales);
-        const float inv = sc ? wa_head_inv_rms(src, a.dim, a.epsilon, lane) : 1.0f;
+        const float inv = sc || a.unit_rms ? wa_head_inv_rms(src, a.dim, a.epsilon, lane) : 1.0f;
         T* dst = reinterpret_cast<T*>(a.keys) + ((size_t)pos * a.kv_heads + g) * a.dim;
         if (a.rot_halves) wa_rotate_row_halves<T>(src, inv, sc, dst, a.dim, a.rot_pairs, cs, sn, lane);
         else wa_rotate_row<T>(src, inv, sc, dst, a.dim, a.rot_pairs, cs, sn, lane);
@@ -151,7 +153,7 @@ __global__ void __launch_bounds__(WA_WARPS * 32) window_attention_kernel(const u
     const uint32_t tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const uint32_t prefix = a.dynamic_position ? *reinterpret_cast<const uint32_t*>(a.dynamic_position) : a.prefix;
     const uint32_t p = prefix + t;
-    const Visible vis = wa_visible(p, a.window, a.keep_first);
+    const Visible vis = wa_visible(p, a.window, a.keep_first, a.chunk);
     const uint32_t tiles = (vis.total + WA_TILE - 1) / WA_TILE, per = (tiles + splits - 1) / splits;
     const uint32_t i_begin = min(vis.total, split * per * WA_TILE), i_end = min(vis.total, (split + 1) * per * WA_TILE);
     const uint32_t g = h / (a.heads / a.kv_heads);

@@ -3,7 +3,7 @@
 // first the tiles of the kept first tokens that lie before the window, then the tiles from the window's start of the CTA's first row up
 // to its last row; the next tile's keys and values arrive by cp.async while the current one is used. mma.sync.m16n8k16 (bf16 x bf16 -> f32):
 //   S = (q * scale * temp) . K^T   with q = q_hi + q_lo, two bf16 numbers per f32 query entry (two MMAs per tile of S);
-//   soft cap, mask (j <= i and (i - j < window or j < keep_first)) and the running (max, sum) of the softmax in f32 on the accumulator
+//   soft cap, mask (j <= i and (inside the window and chunk of i, or j < keep_first)) and the running (max, sum) of the softmax in f32 on the accumulator
 //   fragment, in units of ln 2; the accumulators of O are rescaled when a row's maximum moves;
 //   O += p . V                     with p = p_hi + p_lo again, the fragment of S re-used as the A fragment, V by ldmatrix.trans.
 // The split keeps the error of the query and of the weights below 2^-16 relative, so only the cache's own bf16 rounding remains.
@@ -61,9 +61,14 @@ __global__ void __launch_bounds__(128) window_attention_mma_kernel(const uzu_win
     const uint32_t m0 = mt * WM_BM;
     const uint32_t rows_here = min((uint32_t)WM_BM, a.rows - m0);
     const uint32_t i_first = prefix + m0, i_last = i_first + rows_here - 1, nkeys = i_last + 1;
-    const uint32_t window = a.window ? a.window : 0xFFFFFFFFu, keep = a.keep_first;
+    const uint32_t window = a.window ? a.window : 0xFFFFFFFFu, keep = a.keep_first, chunk = a.chunk;
+    // first key the window (and the chunk) of position i covers; it never decreases with i
+    auto first_seen = [&](uint32_t i) {
+        const uint32_t lo = i >= window ? i + 1 - window : 0u;
+        return chunk ? max(lo, i - i % chunk) : lo;
+    };
     // tiles: [0, keep_tiles) hold kept tokens before the window, then [t_lo, t_hi]
-    const uint32_t j_lo = i_first + 1 > window ? i_first + 1 - window : 0u;
+    const uint32_t j_lo = first_seen(i_first);
     const uint32_t t_lo = j_lo / WM_BN, t_hi = i_last / WM_BN;
     const uint32_t keep_tiles = min((keep + WM_BN - 1) / WM_BN, t_lo);
     const uint32_t ntiles = keep_tiles + (t_hi - t_lo + 1);
@@ -104,6 +109,8 @@ __global__ void __launch_bounds__(128) window_attention_mma_kernel(const uzu_win
     const uint32_t row_lo = warp * 16 + g;                     // this thread's rows of the tile: row_lo and row_lo + 8
     const uint32_t i_lo = i_first + row_lo;
     const uint32_t i_warp_first = i_first + warp * 16, i_warp_last = i_warp_first + 15;
+    const uint32_t lo_row[2] = {first_seen(i_lo), first_seen(i_lo + 8)};                         // of this thread's two rows
+    const uint32_t lo_warp_first = first_seen(i_warp_first), lo_warp_last = first_seen(i_warp_last);
     load_tile(0);
     {   // the query tile, scaled, as hi + lo; sixteen loads of a thread in flight, behind the first tile's requests
         const float* q = reinterpret_cast<const float*>(a.query) + (size_t)m0 * a.heads * dim + (size_t)h * dim;
@@ -135,8 +142,7 @@ __global__ void __launch_bounds__(128) window_attention_mma_kernel(const uzu_win
         const uint32_t j0 = tile_of(idx) * WM_BN, j_end = j0 + WM_BN - 1;
         // nothing of this tile is visible to the warp's rows: it lies after them, or before their windows and holds no kept token
         if (j0 > i_warp_last) continue;
-        const bool before_window = i_warp_first - min(i_warp_first, j_end) >= window;
-        if (before_window && j0 >= keep) continue;
+        if (j_end < lo_warp_first && j0 >= keep) continue;
         const __nv_bfloat16* kt = k_s + (idx & 1) * WM_BN * ldk;
         const __nv_bfloat16* vt = v_s + (idx & 1) * WM_BN * ldv;
         float s[8][4];
@@ -173,7 +179,7 @@ __global__ void __launch_bounds__(128) window_attention_mma_kernel(const uzu_win
         }
         // Scores on the fragment: element c of tile n is row row_lo + 8 * (c >> 1), key j0 + n * 8 + t4 * 2 + (c & 1). Only tiles that
         // touch the diagonal, a window's start or the end of the kept tokens need the mask.
-        const bool all_visible = j_end <= i_warp_first && (i_warp_last - j0 < window || j_end < keep);
+        const bool all_visible = j_end <= i_warp_first && (j0 >= lo_warp_last || j_end < keep);
         float tile_m[2] = {-INFINITY, -INFINITY};
 #pragma unroll
         for (int n = 0; n < 8; ++n)
@@ -184,7 +190,7 @@ __global__ void __launch_bounds__(128) window_attention_mma_kernel(const uzu_win
                 else x *= kLog2e;
                 if (!all_visible) {
                     const uint32_t i = i_lo + 8 * (c >> 1), j = j0 + n * 8 + t4 * 2 + (c & 1);
-                    if (!(j <= i && (i - j < window || j < keep))) x = -INFINITY;
+                    if (!(j <= i && (j >= lo_row[c >> 1] || j < keep))) x = -INFINITY;
                 }
                 s[n][c] = x;
                 tile_m[c >> 1] = fmaxf(tile_m[c >> 1], x);
