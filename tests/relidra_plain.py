@@ -242,3 +242,66 @@ def forward(cfg, weights, tokens):
     m = Model(cfg, weights)
     logits = m.feed(tokens)
     return logits, m.runs_out
+
+
+# ---- configurations and random weights of the tests -------------------------------------------------------------------------------------
+
+def dense(ff):
+    return {"kind": "dense", "ff": ff} if ff else None
+
+
+def delta_layer(heads, kv_heads, dim, vdim, conv, ff=None):
+    return {"type": "delta", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "conv": conv}, "mlp": dense(ff)}
+
+
+def attention_layer(heads, kv_heads, dim, size, ff=None, rot_dims=None, base=1000.0, factor=2.0, scale=None):
+    rot_dims = dim if rot_dims is None else rot_dims
+    return {"type": "attention", "mlp": dense(ff), "mixer": {
+        "heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "mask": {"size": size} if size else None,
+        "rot": {"base": base, "dims": rot_dims, "scaling": {"factor": factor}}, "scale": dim ** -0.5 if scale is None else scale}}
+
+
+def make_config(width, vocab, layers, streams=2, loop=None, eps=1e-5):
+    cfg = {"architecture": "Relidra", "width": width, "vocab": vocab, "norm": {"eps": eps}, "streams": streams, "layers": layers}
+    if loop:
+        cfg["loop"] = dict(zip(("start", "stop", "times"), loop))
+    return cfg
+
+
+def random_weights(cfg, seed):
+    """bf16 tensors of a configuration; decays spread from quick to slow, step sizes and sinks of either sign"""
+    g = torch.Generator().manual_seed(seed)
+    W, V, S = cfg["width"], cfg["vocab"], cfg["streams"]
+
+    def rnd(*shape, mean=0.0, spread=1.0):
+        return (mean + spread * torch.randn(*shape, generator=g)).to(torch.bfloat16)
+
+    def mat(o, i, gain=1.0):
+        return rnd(o, i, spread=gain / math.sqrt(i))
+
+    w = {"embed": rnd(V, W), "final.norm": rnd(W, mean=1.0, spread=0.2)}
+    for i, L in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", L["mixer"]
+        for q in (1, 2) if L.get("mlp") else (1,):
+            w[p + f"norm{q}"] = rnd(W, mean=1.0, spread=0.2)
+            w[p + f"hc{q}.in"] = rnd(S, mean=1.0 / S, spread=0.3)
+            w[p + f"hc{q}.out"] = rnd(S, mean=0.7, spread=0.3)
+            w[p + f"hc{q}.mix"] = (torch.eye(S) * 0.8 + 0.2 * torch.randn(S, S, generator=g)).to(torch.bfloat16)
+        if L["type"] == "attention":
+            H, G, d = m["heads"], m["kv_heads"], m["dim"]
+            w[p + "mix.q"], w[p + "mix.q.b"] = mat(H * d, W, 1.5), rnd(H * d, spread=0.5)
+            w[p + "mix.k"], w[p + "mix.k.b"] = mat(G * d, W, 1.5), rnd(G * d, spread=0.5)
+            w[p + "mix.sink"], w[p + "mix.o"] = rnd(H, mean=0.5), mat(W, H * d)
+        else:
+            H, G, d, dv, taps = m["heads"], m["kv_heads"], m["dim"], m["vdim"], m["conv"]
+            for name, c in (("q", G * d), ("k", G * d), ("v", H * dv)):
+                w[p + "mix." + name] = mat(c, W, 1.5)
+                w[p + f"mix.{name}.conv"] = rnd(c, taps, spread=taps ** -0.5)
+            w[p + "mix.g"], w[p + "mix.o"] = mat(H * dv, W, 1.5), mat(W, H * dv)
+            w[p + "mix.a"], w[p + "mix.b"] = mat(H, W, 1.5), mat(H, W, 2.0)
+            w[p + "mix.A_log"], w[p + "mix.dt_bias"] = rnd(H, mean=-1.0, spread=1.0), rnd(H, mean=-1.0, spread=1.0)
+            w[p + "mix.norm"] = rnd(dv, mean=1.0, spread=0.2)
+        if L.get("mlp"):
+            f = L["mlp"]["ff"]
+            w[p + "mlp.up"], w[p + "mlp.down"] = mat(f, W, 1.5), mat(W, f)
+    return w

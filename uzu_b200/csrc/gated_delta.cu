@@ -8,7 +8,7 @@
 // contiguous bytes at L = 8: no bank conflict, the columns of a warp share the read).
 //   gated_delta_kernel       the tokens of a pass in order, 4 warps per CTA, grid (column blocks, heads). The prepared q / k / v / decay / beta
 //                            rows arrive by cp.async one batch ahead. An element's arithmetic does not depend on how a prompt is cut.
-//   delta_prepare_kernel     convolution, silu, unit vectors and gates of all tokens of a pass at once, a warp per (token, head part).
+//   delta_prepare_kernel     convolution, silu, unit vectors and gates of all tokens of a pass at once, a warp per (a few tokens, head).
 //   gated_delta_step_kernel  one token with everything between the projections in one launch: a cluster of CL CTAs per head, each CTA owning
 //                            vdim / CL columns; the state is requested before the previous kernel's results are waited for; the head's sum
 //                            of squares meets through distributed shared memory in rank order; norm weight and silu gate applied on the way out.
@@ -51,6 +51,18 @@ __device__ __forceinline__ float gd_conv(const uzu_delta_prepare_args& a, uint32
     return gd_silu(y);
 }
 
+// the convolution of channel c at position `prefix` without its last tap (all inputs come from the ring), and that tap's weight
+__device__ __forceinline__ void gd_conv_past(const uzu_delta_prepare_args& a, uint32_t channels, uint32_t prefix, uint32_t c, float& past, float& tap) {
+    const float* w = reinterpret_cast<const float*>(a.conv) + (size_t)c * a.taps;
+    const float* ring = reinterpret_cast<const float*>(a.ring) + c;
+    past = 0.0f;
+    for (uint32_t j = 0; j + 1 < a.taps; ++j) {
+        const uint32_t back = a.taps - 1 - j;
+        if (back <= prefix) past = fmaf(w[j], ring[(size_t)((prefix - back) % a.taps) * channels], past);
+    }
+    tap = w[a.taps - 1];
+}
+
 __device__ __forceinline__ void gd_cp_async16(void* smem_ptr, const void* gmem_ptr) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(smem_ptr)), "l"(gmem_ptr) : "memory");
 }
@@ -63,6 +75,28 @@ __device__ __forceinline__ float gd_lane_sum(float v) {
 #pragma unroll
     for (int o = L / 2; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
     return v;
+}
+
+// v[0] of lane part p <- the sum over the L lanes of a column of v[p / (L / U)]  (U values, U <= L, both powers of two)
+template <int U, int L>
+__device__ __forceinline__ void gd_transpose_sum(float (&v)[U], uint32_t part) {
+    int n = U;
+#pragma unroll
+    for (int o = L / 2; o > 0; o >>= 1) {
+        if (n > 1) {
+            n >>= 1;
+            const bool up = (part & o) != 0;
+#pragma unroll
+            for (int i = 0; i < U / 2; ++i) {
+                if (i < n) {
+                    const float keep = up ? v[i + n] : v[i], send = up ? v[i] : v[i + n];
+                    v[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+                }
+            }
+        } else {
+            v[0] += __shfl_xor_sync(0xffffffffu, v[0], o);
+        }
+    }
 }
 
 template <int NV>
@@ -92,7 +126,88 @@ __device__ __forceinline__ void gd_update(float4 (&s)[NV], const float4 (&k)[NV]
 
 }  // namespace
 
-// a warp per (row, unit): units [0, kv_heads) queries, [kv_heads, 2 kv_heads) keys, then the value heads, then one unit for the row's gates
+// A warp per (block of GP_ROWS tokens, unit): units [0, kv_heads) queries, [kv_heads, 2 kv_heads) keys, then the value heads, then one unit for
+// the gates. NC = channels of a head per lane; the convolution's window of a channel slides through registers, so an input is read once.
+constexpr int GP_ROWS = 8;
+
+template <int TAPS, int NC>
+__global__ void __launch_bounds__(128) delta_prepare_window_kernel(const uzu_delta_prepare_args a) {
+    pdl_launch_dependents();
+    const uint32_t lane = threadIdx.x & 31;
+    const uint32_t units = 2 * a.kv_heads + a.heads + 1, blocks = (a.rows + GP_ROWS - 1) / GP_ROWS;
+    const uint32_t item = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (item >= blocks * units) return;
+    const uint32_t t0 = item / units * GP_ROWS, unit = item % units, nr = min((uint32_t)GP_ROWS, a.rows - t0);
+    const uint32_t kd = a.kv_heads * a.dim, channels = 2 * kd + a.heads * a.vdim, dim4 = (a.dim + 3) & ~3u;
+    if (unit == units - 1) {
+        pdl_wait();
+        for (uint32_t i = lane; i < nr * a.heads; i += 32) {
+            const uint32_t t = t0 + i / a.heads, h = i % a.heads;
+            const float* row = reinterpret_cast<const float*>(a.proj) + (size_t)t * a.stride;
+            reinterpret_cast<float*>(a.decay)[(size_t)t * a.heads + h] =
+                gd_decay(reinterpret_cast<const float*>(a.a_log)[h], row[a.a_offset + h] + reinterpret_cast<const float*>(a.dt_bias)[h]);
+            reinterpret_cast<float*>(a.beta)[(size_t)t * a.heads + h] = gd_sigmoid(row[a.b_offset + h]);
+        }
+        return;
+    }
+    const bool is_q = unit < a.kv_heads, is_v = unit >= 2 * a.kv_heads;
+    const uint32_t head = is_q ? unit : (is_v ? unit - 2 * a.kv_heads : unit - a.kv_heads), n = is_v ? a.vdim : a.dim;
+    const uint32_t c0 = is_q ? head * a.dim : (is_v ? 2 * kd + head * a.vdim : kd + head * a.dim);
+    const uint32_t pad = is_v ? n : dim4;                        // q / k rows are padded to whole float4
+    float* out = reinterpret_cast<float*>(is_q ? a.q : (is_v ? a.v : a.k)) + ((size_t)t0 * (is_v ? a.heads : a.kv_heads) + head) * pad;
+    const size_t out_stride = (size_t)(is_v ? a.heads : a.kv_heads) * pad;
+    const float* proj = reinterpret_cast<const float*>(a.proj) + (size_t)t0 * a.stride + c0;
+    float w[NC][TAPS], x[NC][TAPS + GP_ROWS - 1];
+#pragma unroll
+    for (int i = 0; i < NC; ++i) {
+        const uint32_t c = lane + 32u * i;
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) w[i][j] = c < n ? reinterpret_cast<const float*>(a.conv)[(size_t)(c0 + c) * TAPS + j] : 0.0f;
+    }
+    pdl_wait();
+    const uint32_t prefix = gd_prefix(a);
+#pragma unroll
+    for (int i = 0; i < NC; ++i) {
+        const uint32_t c = lane + 32u * i;
+#pragma unroll
+        for (int j = 0; j < TAPS + GP_ROWS - 1; ++j) {
+            const int t = j - (TAPS - 1);                        // row relative to the block's first
+            float v = 0.0f;
+            if (c < n) {
+                if (t >= 0 || (uint32_t)(-t) <= t0) { if (t < (int)nr) v = proj[(ptrdiff_t)t * a.stride + c]; }
+                else if ((uint32_t)(-t) <= prefix + t0)
+                    v = reinterpret_cast<const float*>(a.ring)[(size_t)((prefix + t0 + t) % TAPS) * channels + c0 + c];
+            }
+            x[i][j] = v;
+        }
+    }
+#pragma unroll
+    for (int r = 0; r < GP_ROWS; ++r) {
+        if ((uint32_t)r >= nr) break;
+        float y[NC], f = 1.0f;
+#pragma unroll
+        for (int i = 0; i < NC; ++i) {
+            float s = 0.0f;
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) s = fmaf(w[i][j], x[i][r + j], s);
+            y[i] = gd_silu(s);
+        }
+        if (!is_v) {
+            float ss = 0.0f;
+#pragma unroll
+            for (int i = 0; i < NC; ++i) ss = fmaf(y[i], y[i], ss);      // (channels past the head hold zero)
+            f = 1.0f / sqrtf(warp_sum(ss) + kUnitEps);
+            if (is_q) f *= 1.0f / sqrtf((float)a.dim);
+        }
+#pragma unroll
+        for (int i = 0; i < NC; ++i) {
+            const uint32_t c = lane + 32u * i;
+            if (c < pad) out[(size_t)r * out_stride + c] = y[i] * f;
+        }
+    }
+}
+
+// the same for any number of taps and any head size: a warp per (token, unit), every input read once per tap
 __global__ void __launch_bounds__(128) delta_prepare_kernel(const uzu_delta_prepare_args a) {
     pdl_launch_dependents();
     pdl_wait();
@@ -150,7 +265,7 @@ constexpr int gd_batch() { return L * NV * 4 <= 256 ? 16 : (L * NV * 4 <= 512 ? 
 
 template <int L, int NV>
 __global__ void __launch_bounds__(GD_WARPS * 32) gated_delta_kernel(const uzu_gated_delta_args ga) {
-    constexpr int ROWF = L * NV * 4, BATCH = gd_batch<L, NV>(), CC = GD_WARPS * (32 / L);
+    constexpr int ROWF = L * NV * 4, BATCH = gd_batch<L, NV>(), CC = GD_WARPS * (32 / L), U = BATCH < 8 ? BATCH : 8;
     pdl_launch_dependents();
     pdl_wait();
     extern __shared__ __align__(16) float gd_smem[];
@@ -227,19 +342,50 @@ __global__ void __launch_bounds__(GD_WARPS * 32) gated_delta_kernel(const uzu_ga
         const float* v = vs + buf * BATCH * CC + cl;
         const float* g = gs + buf * BATCH;
         const float* b = bs + buf * BATCH;
-#pragma unroll 2
-        for (uint32_t r = 0; r < nb; ++r) {
+        auto load_row = [&](float4 (&x)[NV], const float* row) {
+#pragma unroll
+            for (int i = 0; i < NV; ++i) x[i] = *reinterpret_cast<const float4*>(row + i * L * 4);
+        };
+        uint32_t r0 = 0;
+        for (; r0 + U <= nb; r0 += U) {              // U tokens in straight-line code: the next token's rows are read during this token's reduction
+            float gr[U], bg[U], bv[U], o[U];
+            float4 kc[NV], qc[NV], kn[NV], qn[NV];
+            load_row(kc, k + r0 * ROWF);
+            load_row(qc, q + r0 * ROWF);
+#pragma unroll
+            for (int j = 0; j < U; ++j) {
+                const float beta = b[r0 + j];
+                gr[j] = g[r0 + j];
+                bg[j] = -beta * gr[j];
+                bv[j] = beta * v[(r0 + j) * CC];
+            }
+#pragma unroll
+            for (int j = 0; j < U; ++j) {
+                if (j + 1 < U) {
+                    load_row(kn, k + (r0 + j + 1) * ROWF);
+                    load_row(qn, q + (r0 + j + 1) * ROWF);
+                }
+                const float z = gd_lane_sum<L>(gd_dot<NV>(S, kc));
+                gd_update<NV>(S, kc, gr[j], fmaf(bg[j], z, bv[j]));
+                o[j] = gd_dot<NV>(S, qc);
+                if (j + 1 < U) {
+#pragma unroll
+                    for (int i = 0; i < NV; ++i) { kc[i] = kn[i]; qc[i] = qn[i]; }
+                }
+            }
+            // the U read-outs meet over the lanes of a column all at once: at every level a lane keeps half of the values
+            gd_transpose_sum<U, L>(o, part);
+            if (col_ok && part % (L / U) == 0) out[(size_t)(tb + r0 + part / (L / U)) * v_stride] = o[0];
+        }
+        for (; r0 < nb; ++r0) {
             float4 k4[NV], q4[NV];
-#pragma unroll
-            for (int i = 0; i < NV; ++i) k4[i] = *reinterpret_cast<const float4*>(k + r * ROWF + i * L * 4);
-            const float gr = g[r];
+            load_row(k4, k + r0 * ROWF);
+            load_row(q4, q + r0 * ROWF);
+            const float gr = g[r0], beta = b[r0];
             const float z = gd_lane_sum<L>(gd_dot<NV>(S, k4));
-            const float u = b[r] * (v[r * CC] - gr * z);
-#pragma unroll
-            for (int i = 0; i < NV; ++i) q4[i] = *reinterpret_cast<const float4*>(q + r * ROWF + i * L * 4);
-            gd_update<NV>(S, k4, gr, u);
+            gd_update<NV>(S, k4, gr, fmaf(-beta * gr, z, beta * v[r0 * CC]));
             const float o = gd_lane_sum<L>(gd_dot<NV>(S, q4));
-            if (part == 0 && col_ok) out[(size_t)(tb + r) * v_stride] = o;
+            if (part == 0 && col_ok) out[(size_t)(tb + r0) * v_stride] = o;
         }
         __syncthreads();
     }
@@ -280,30 +426,48 @@ __global__ void __cluster_dims__(CL, 1, 1) __launch_bounds__(GS_THREADS) gated_d
             S[i] = (cl < ncols && c < dim4) ? *reinterpret_cast<const float4*>(state + (size_t)cl * dim4 + c) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
         }
     };
-    load_state(tid / L);             // nothing in front of this kernel writes the state: requested before the wait
+    load_state(tid / L);             // nothing in front of this kernel writes the state or the ring: requested before the wait
+    // ... and so is what the convolution takes from earlier tokens: all but the last tap
+    const uint32_t prefix = gd_prefix(a), v0 = 2 * kd + h * a.vdim + col0;
+    constexpr int QK = (2 * ROWF + GS_THREADS - 1) / GS_THREADS;      // q / k channels of a thread
+    float qk_past[QK], qk_tap[QK], v_past = 0.0f, v_tap = 0.0f;
+    auto qk_channel = [&](uint32_t i) { return (i < ROWF ? 0u : kd - ROWF) + kvh * a.dim + i; };      // (i counts q channels, then k channels)
+    auto in_head = [&](uint32_t i) { return i < 2 * ROWF && (i < ROWF ? i : i - ROWF) < a.dim; };
+#pragma unroll
+    for (int u = 0; u < QK; ++u) {
+        const uint32_t i = tid + u * GS_THREADS;
+        qk_past[u] = qk_tap[u] = 0.0f;
+        if (in_head(i)) gd_conv_past(a, channels, prefix, qk_channel(i), qk_past[u], qk_tap[u]);
+    }
+    if (tid < ncols) gd_conv_past(a, channels, prefix, v0 + tid, v_past, v_tap);
+    const float a_log = reinterpret_cast<const float*>(a.a_log)[h], dt_bias = reinterpret_cast<const float*>(a.dt_bias)[h];
+    const float norm0 = tid < ncols ? reinterpret_cast<const float*>(sa.norm)[(size_t)h * a.vdim + col0 + tid] : 0.0f;
     pdl_wait();
-    const uint32_t prefix = gd_prefix(a);
     const float* proj = reinterpret_cast<const float*>(a.proj);
+    const float* gate = proj + sa.gate_offset + (size_t)h * a.vdim + col0;
+    const float gate0 = tid < ncols ? gate[tid] : 0.0f;
     float* ring = reinterpret_cast<float*>(a.ring) + (size_t)(prefix % a.taps) * channels;        // the slot of this token: nobody reads it here
     float sq = 0.0f, sk = 0.0f;
-    for (uint32_t i = tid; i < 2 * ROWF; i += GS_THREADS) {
-        const bool is_q = i < ROWF;
-        const uint32_t c = is_q ? i : i - ROWF, ch = (is_q ? 0u : kd) + kvh * a.dim + c;
+#pragma unroll
+    for (int u = 0; u < QK; ++u) {
+        const uint32_t i = tid + u * GS_THREADS;
         float y = 0.0f;
-        if (c < a.dim) {
-            y = gd_conv(a, channels, prefix, 0, ch);
-            if (rank == 0 && h % group == 0 && a.taps > 1) ring[ch] = proj[ch];
+        if (in_head(i)) {
+            const float x = proj[qk_channel(i)];
+            y = gd_silu(fmaf(qk_tap[u], x, qk_past[u]));
+            if (rank == 0 && h % group == 0 && a.taps > 1) ring[qk_channel(i)] = x;
         }
-        (is_q ? qs : ks)[c] = y;
-        if (is_q) sq = fmaf(y, y, sq);
+        if (i < 2 * ROWF) qs[i] = y;                                     // ks follows qs
+        if (i < ROWF) sq = fmaf(y, y, sq);
         else sk = fmaf(y, y, sk);
     }
     for (uint32_t i = tid; i < ncols; i += GS_THREADS) {
-        const uint32_t ch = 2 * kd + h * a.vdim + col0 + i;
-        vs[i] = gd_conv(a, channels, prefix, 0, ch);
-        if (a.taps > 1) ring[ch] = proj[ch];
+        if (i >= GS_THREADS) gd_conv_past(a, channels, prefix, v0 + i, v_past, v_tap);
+        const float x = proj[v0 + i];
+        vs[i] = gd_silu(fmaf(v_tap, x, v_past));
+        if (a.taps > 1) ring[v0 + i] = x;
     }
-    const float g = gd_decay(reinterpret_cast<const float*>(a.a_log)[h], proj[a.a_offset + h] + reinterpret_cast<const float*>(a.dt_bias)[h]);
+    const float g = gd_decay(a_log, proj[a.a_offset + h] + dt_bias);
     const float beta = gd_sigmoid(proj[a.b_offset + h]);
     sq = warp_sum(sq);
     sk = warp_sum(sk);
@@ -354,10 +518,10 @@ __global__ void __cluster_dims__(CL, 1, 1) __launch_bounds__(GS_THREADS) gated_d
         for (int c = 0; c < CL; ++c) ss += ss_parts[c];
     }
     const float inv = 1.0f / sqrtf(ss / (float)a.vdim + sa.epsilon);
-    const float* gate = proj + sa.gate_offset + (size_t)h * a.vdim + col0;
-    const float* norm = reinterpret_cast<const float*>(sa.norm) + col0;
     float* out = reinterpret_cast<float*>(sa.out) + (size_t)h * a.vdim + col0;
-    for (uint32_t i = tid; i < ncols; i += GS_THREADS) out[i] = os[i] * inv * norm[i] * gd_silu(gate[i]);
+    if (tid < ncols) out[tid] = os[tid] * inv * norm0 * gd_silu(gate0);
+    const float* norm = reinterpret_cast<const float*>(sa.norm) + (size_t)h * a.vdim + col0;
+    for (uint32_t i = tid + GS_THREADS; i < ncols; i += GS_THREADS) out[i] = os[i] * inv * norm[i] * gd_silu(gate[i]);
 }
 
 static const char* delta_prepare_check(const uzu_delta_prepare_args& a, bool scratch) {
@@ -393,7 +557,23 @@ void uzu_delta_prepare_encode(uzu_command_buffer* cmd, const uzu_delta_prepare_a
         return;
     }
     if (a->rows == 0) return;
-    const uint32_t items = a->rows * (2 * a->kv_heads + a->heads + 1);
+    const uint32_t units = 2 * a->kv_heads + a->heads + 1, widest = std::max(a->dim, a->vdim);
+    if (a->rows >= 4 && a->taps >= 2 && a->taps <= 4 && widest <= 256) {
+        const uint32_t blocks = (a->rows + GP_ROWS - 1) / GP_ROWS;
+        auto go = [&](auto kernel) { launch(cmd, "delta_prepare_kernel", kernel, dim3((blocks * units + 3) / 4), dim3(128), 0, *a); };
+        auto by_width = [&](auto taps_c) {
+            constexpr int T = decltype(taps_c)::value;
+            if (widest <= 32) go(delta_prepare_window_kernel<T, 1>);
+            else if (widest <= 64) go(delta_prepare_window_kernel<T, 2>);
+            else if (widest <= 128) go(delta_prepare_window_kernel<T, 4>);
+            else go(delta_prepare_window_kernel<T, 8>);
+        };
+        if (a->taps == 2) by_width(std::integral_constant<int, 2>{});
+        else if (a->taps == 3) by_width(std::integral_constant<int, 3>{});
+        else by_width(std::integral_constant<int, 4>{});
+        return;
+    }
+    const uint32_t items = a->rows * units;
     launch(cmd, "delta_prepare_kernel", delta_prepare_kernel, dim3((items + 3) / 4), dim3(128), 0, *a);
 }
 

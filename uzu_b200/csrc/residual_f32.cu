@@ -253,6 +253,112 @@ __global__ void __launch_bounds__(MAXS > 4 ? 256 : 1024) stream_mix_kernel(const
     for (uint32_t i = threadIdx.x + KEEP * blockDim.x; i < a.n; i += blockDim.x) store(i, again(i));
 }
 
+// The same for rows of whole float4 that a CTA holds in registers (n <= 8 * threads): 16-byte requests, all of a thread's in flight at once.
+template <int MAXS>
+__global__ void __launch_bounds__(512) stream_mix_vec_kernel(const uzu_stream_mix_args a) {
+    pdl_launch_dependents();
+    __shared__ float red[32], cmix[MAXS * MAXS], cout[MAXS], cread[MAXS];
+    const uint32_t row = blockIdx.x, S = a.streams, n4 = a.n / 4;
+    if (threadIdx.x < MAXS * MAXS) {
+        const uint32_t s = threadIdx.x / MAXS, t = threadIdx.x % MAXS;
+        cmix[threadIdx.x] = (a.y && s < S && t < S) ? reinterpret_cast<const float*>(a.mix)[s * S + t] : 0.0f;
+        if (s == 0) {
+            cout[t] = (a.y && t < S) ? reinterpret_cast<const float*>(a.out)[t] : 0.0f;
+            cread[t] = t < S ? (a.read ? reinterpret_cast<const float*>(a.read)[t] : 1.0f) : 0.0f;
+        }
+    }
+    constexpr int KEEP = 2;
+    const float4 zero = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    float4 w[KEEP];
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+        const uint32_t i = threadIdx.x + j * blockDim.x;
+        w[j] = (a.output && i < n4) ? reinterpret_cast<const float4*>(a.weight)[i] : zero;
+    }
+    pdl_wait();
+    float4* x = reinterpret_cast<float4*>(a.x) + (size_t)row * S * n4;
+    const float4* y = a.y ? reinterpret_cast<const float4*>(a.y) + (size_t)row * n4 : nullptr;
+    float4 xs[KEEP][MAXS], yy[KEEP], u[KEEP];
+    if (a.token_ids) {
+        const uint32_t tok = reinterpret_cast<const uint32_t*>(a.token_ids)[row];
+#pragma unroll
+        for (int j = 0; j < KEEP; ++j) {
+            const uint32_t i = threadIdx.x + j * blockDim.x;
+            float4 e = zero;
+            if (tok < a.vocab && i < n4) {
+                const size_t at = (size_t)tok * n4 + i;
+                if (a.table_dt == UZU_DT_F32) {
+                    e = reinterpret_cast<const float4*>(a.table)[at];
+                } else {
+                    const uint2 b = reinterpret_cast<const uint2*>(a.table)[at];
+                    e = make_float4(__uint_as_float(b.x << 16), __uint_as_float(b.x & 0xffff0000u), __uint_as_float(b.y << 16), __uint_as_float(b.y & 0xffff0000u));
+                }
+            }
+#pragma unroll
+            for (int s = 0; s < MAXS; ++s) xs[j][s] = e;
+            yy[j] = zero;
+        }
+    } else {
+#pragma unroll
+        for (int j = 0; j < KEEP; ++j) {
+            const uint32_t i = threadIdx.x + j * blockDim.x;
+#pragma unroll
+            for (int s = 0; s < MAXS; ++s) xs[j][s] = ((uint32_t)s < S && i < n4) ? x[(size_t)s * n4 + i] : zero;
+            yy[j] = (y && i < n4) ? y[i] : zero;
+        }
+    }
+    __syncthreads();
+    float sum = 0.0f;
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+        const uint32_t i = threadIdx.x + j * blockDim.x;
+        u[j] = zero;
+#pragma unroll
+        for (int t = 0; t < MAXS; ++t) {
+            if ((uint32_t)t < S) {
+                float4 v = xs[j][t];
+                if (y) {
+                    const float co = cout[t];
+                    v = make_float4(co * yy[j].x, co * yy[j].y, co * yy[j].z, co * yy[j].w);
+#pragma unroll
+                    for (int s = 0; s < MAXS; ++s) {
+                        const float m = cmix[s * MAXS + t];
+                        v.x = fmaf(m, xs[j][s].x, v.x); v.y = fmaf(m, xs[j][s].y, v.y); v.z = fmaf(m, xs[j][s].z, v.z); v.w = fmaf(m, xs[j][s].w, v.w);
+                    }
+                }
+                if ((y || a.token_ids) && i < n4) x[(size_t)t * n4 + i] = v;
+                const float cr = cread[t];
+                u[j].x = fmaf(cr, v.x, u[j].x); u[j].y = fmaf(cr, v.y, u[j].y); u[j].z = fmaf(cr, v.z, u[j].z); u[j].w = fmaf(cr, v.w, u[j].w);
+            }
+        }
+        if (a.u && i < n4) reinterpret_cast<float4*>(a.u)[(size_t)row * n4 + i] = u[j];
+        sum += (u[j].x + u[j].y) + (u[j].z + u[j].w);              // (zero past the row)
+    }
+    if (!a.output) return;
+    const float mean = block_sum(sum, red) / (float)a.n;
+    float ss = 0.0f;
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+        if (threadIdx.x + j * blockDim.x < n4) {
+            u[j].x -= mean; u[j].y -= mean; u[j].z -= mean; u[j].w -= mean;
+            ss += (u[j].x * u[j].x + u[j].y * u[j].y) + (u[j].z * u[j].z + u[j].w * u[j].w);
+        }
+    }
+    const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)a.n + a.epsilon);
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+        const uint32_t i = threadIdx.x + j * blockDim.x;
+        if (i >= n4) continue;
+        const float4 v = make_float4(u[j].x * inv * w[j].x, u[j].y * inv * w[j].y, u[j].z * inv * w[j].z, u[j].w * inv * w[j].w);
+        if (a.output_bf16) {
+            const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+            reinterpret_cast<uint2*>(a.output)[(size_t)row * n4 + i] = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+        } else {
+            reinterpret_cast<float4*>(a.output)[(size_t)row * n4 + i] = v;
+        }
+    }
+}
+
 template <typename TW>
 __global__ void token_gate_kernel(const uzu_token_gate_args a) {
     pdl_launch_dependents();
@@ -610,6 +716,14 @@ void uzu_stream_mix_encode(uzu_command_buffer* cmd, const uzu_stream_mix_args* a
         return;
     }
     if (a->rows == 0 || a->n == 0) return;
+    // rows of whole float4 up to 4096 elements, all row blocks 16-byte aligned
+    const uint64_t blocks = a->x | a->y | a->u | a->weight | a->output | a->table;
+    if (a->n % 4 == 0 && a->n <= 4096 && a->streams <= 4 && (blocks & 15) == 0) {
+        const uint32_t t = a->n <= 1024 ? 128 : (a->n <= 2048 ? 256 : 512);
+        if (a->streams <= 2) launch(cmd, "stream_mix_kernel", stream_mix_vec_kernel<2>, dim3(a->rows), dim3(t), 0, *a);
+        else launch(cmd, "stream_mix_kernel", stream_mix_vec_kernel<4>, dim3(a->rows), dim3(t), 0, *a);
+        return;
+    }
     const uint32_t threads = (a->n <= 2048 || a->streams > 4) ? 256 : (a->n <= 4096 ? 512 : 1024);
     auto go = [&](auto kernel) { launch(cmd, "stream_mix_kernel", kernel, dim3(a->rows), dim3(threads), 0, *a); };
     if (a->streams <= 2) go(stream_mix_kernel<2>);

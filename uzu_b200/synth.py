@@ -749,3 +749,84 @@ def vakesun_preset(width=2048, vocab=32768, layers=8, ff=None, window=512, side_
         else:
             out.append(vakesun_latent_layer(heads, 128, 128, 512, min(1536, width), window, vakesun_dense_mlp(ff), kv_from=i - 3))
     return vakesun_config(width, vocab, out, eps=1e-6, residual_mult=0.3, embedding_scale=1.0, side_dim=side_dim)
+
+
+# ---- Relidra: gated delta rule and chunked attention over a residual of mixed streams, looped layers ---------------------------------------
+
+def relidra_dense_mlp(ff: int) -> dict:
+    return {"kind": "dense", "ff": ff}
+
+
+def relidra_delta_layer(heads: int, kv_heads: int, dim: int, vdim: int, conv: int, mlp: dict | None) -> dict:
+    return {"type": "delta", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "conv": conv}, "mlp": mlp}
+
+
+def relidra_attention_layer(heads: int, kv_heads: int, dim: int, chunk: int, mlp: dict | None, scale: float | None = None, rot_dims: int | None = None,
+                            rot_base: float = 10000.0, factor: float = 1.0) -> dict:
+    return {"type": "attention", "mlp": mlp, "mixer": {
+        "heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "mask": {"size": chunk}, "scale": dim ** -0.5 if scale is None else scale,
+        "rot": {"base": rot_base, "dims": dim if rot_dims is None else rot_dims, "scaling": {"factor": factor}}}}
+
+
+def relidra_config(width: int, vocab: int, layers: list, streams: int = 2, loop: dict | None = None, eps: float = 1e-6) -> dict:
+    """loop: {"start", "stop", "times"} or None (every layer once)"""
+    cfg = {"architecture": "Relidra", "width": width, "vocab": vocab, "norm": {"eps": eps}, "streams": streams, "layers": layers}
+    if loop:
+        cfg["loop"] = loop
+    return cfg
+
+
+def relidra_tensors(config: dict, seed: int = 0) -> dict:
+    """Seeded random tensors of a Relidra config: f32 values that bf16 holds exactly."""
+    rng = np.random.default_rng(seed)
+    W, V, S = config["width"], config["vocab"], config["streams"]
+
+    def bf(x):
+        return st_bits_to_f32(f32_to_bf16_bits(np.asarray(x, np.float32)))
+
+    def mat(rows, cols, gain=1.0):
+        return bf(rng.standard_normal((rows, cols), dtype=np.float32) * (gain / np.sqrt(cols)))
+
+    def vec(n, mean=0.0, spread=0.1):
+        return bf(mean + spread * rng.standard_normal(n, dtype=np.float32))
+
+    t = {"embed": mat(V, W, np.sqrt(W)), "final.norm": vec(W, 1.0, 0.2)}
+    for i, L in enumerate(config["layers"]):
+        p, m = f"l{i}.", L["mixer"]
+        for q in (1, 2) if L.get("mlp") else (1,):
+            t[p + f"norm{q}"] = vec(W, 1.0, 0.2)
+            t[p + f"hc{q}.in"], t[p + f"hc{q}.out"] = vec(S, 1.0 / S, 0.1), vec(S, 0.7, 0.2)
+            t[p + f"hc{q}.mix"] = bf(0.9 * np.eye(S, dtype=np.float32) + 0.1 * rng.standard_normal((S, S), dtype=np.float32))
+        if L["type"] == "attention":
+            H, G, D = m["heads"], m["kv_heads"], m["dim"]
+            t[p + "mix.q"], t[p + "mix.q.b"], t[p + "mix.k"], t[p + "mix.k.b"] = mat(H * D, W, 1.5), vec(H * D, 0.0, 0.2), mat(G * D, W, 1.5), vec(G * D, 0.0, 0.2)
+            t[p + "mix.sink"], t[p + "mix.o"] = vec(H, 0.5, 1.0), mat(W, H * D)
+        else:
+            H, G, D, Dv, taps = m["heads"], m["kv_heads"], m["dim"], m["vdim"], m["conv"]
+            for name, c in (("q", G * D), ("k", G * D), ("v", H * Dv)):
+                t[p + "mix." + name], t[p + f"mix.{name}.conv"] = mat(c, W, 1.5), mat(c, taps)
+            t[p + "mix.g"], t[p + "mix.o"], t[p + "mix.norm"] = mat(H * Dv, W, 1.5), mat(W, H * Dv), vec(Dv, 1.0, 0.2)
+            t[p + "mix.a"], t[p + "mix.b"] = mat(H, W), mat(H, W, 2.0)
+            t[p + "mix.A_log"], t[p + "mix.dt_bias"] = vec(H, -1.0, 1.0), vec(H, -1.0, 1.0)
+        if L.get("mlp"):
+            f = L["mlp"]["ff"]
+            t[p + "mlp.up"], t[p + "mlp.down"] = mat(f, W, 1.5), mat(W, f)
+    return t
+
+
+def write_relidra_model(config: dict, path, seed: int = 0, tensors: dict | None = None) -> Path:
+    """config.json + model.safetensors (bf16). `tensors` overrides the seeded random ones (values are rounded to bf16)."""
+    return write_punilix_model(config, path, seed, tensors if tensors is not None else relidra_tensors(config, seed))
+
+
+def relidra_preset(width=2048, vocab=32768, layers=6, ff=None, chunk=512, streams=2, loop: dict | None = None) -> dict:
+    """A layer stack of realistic sizes for benchmarks: delta layers and attention layers in turn, each with a feed-forward."""
+    ff = ff or 4 * width
+    heads = max(width // 128, 1)
+    out = []
+    for i in range(layers):
+        if i % 2 == 0:
+            out.append(relidra_delta_layer(heads, heads, 128, 128, 4, relidra_dense_mlp(ff)))
+        else:
+            out.append(relidra_attention_layer(heads, max(heads // 4, 1), 128, chunk, relidra_dense_mlp(ff), rot_dims=64, rot_base=1e6, factor=4.0))
+    return relidra_config(width, vocab, out, streams=streams, loop=loop)
