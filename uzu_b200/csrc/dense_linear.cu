@@ -1,11 +1,12 @@
 // Dense (unquantised) linear: D (+)= scale * A . W^T, f32 activations, bf16 or f32 weights [n, k], f32 accumulation.
-// Three kernels behind one entry point (uzu_dense_linear_encode):
+// Four kernels behind one entry point (uzu_dense_linear_encode):
+//   one-row kernel (a single row, one plain product): the same weight pass with CTAs that stay for many output features;
 //   rows kernel   (<= 8 rows per group): one warp per output feature, the weight row streamed once with 128-bit loads and multiplied
 //                 with every activation row in f32 -- the decode step's weight pass, bound by the weight bytes;
 //   tensor kernels (bf16 weights, >= 32 rows): 64 x 64 output tiles (128 x 128 with ldmatrix fragments from 96 rows on) on
 //                 mma.sync.m16n8k16 (bf16 x bf16 -> f32), A rounded to bf16 while it is staged, double-buffered shared-memory tiles;
 //   tile kernel   (everything else, and every f32-weight product of more than 8 rows): 64 x 64 tiles of f32 multiply-adds.
-// All three share the operand addressing: z-batches (per-head weights: operand z starts z*stride further in A, W and D) and row groups
+// All share the operand addressing: z-batches (per-head weights: operand z starts z*stride further in A, W and D) and row groups
 // (per-expert weights: compact rows [off[z], off[z+1]) use weight z, an optional map names the activation row a compact row reads).
 #include <mma.h>
 
@@ -327,6 +328,114 @@ __global__ void __launch_bounds__(256, RMAX == 1 ? 4 : 2) dense_rows_kernel(cons
     }
 }
 
+// ---- one activation row, one plain product: the decode step's usual shape --------------------------------------------------------------
+// CTAs stay for several groups of output features: the activation row is staged (and, with a_norm_weight, layer-normed) once per CTA, and the
+// weights of a warp's next batch -- of the next feature, too -- are requested before the current batch is used, so the weight stream does
+// not stop between features. KS warps share a feature as in the rows kernel. bf16 weights: the row is kept as two planes (the first and the
+// second float4 of every eight elements), so that a warp's 16-byte reads fall into different banks.
+constexpr uint32_t DG_MAX_K = 16384;
+
+template <typename TW, int KS>
+__global__ void __launch_bounds__(256, 4) dense_gemv_kernel(const uzu_dense_linear_args a) {
+    extern __shared__ __align__(16) float dg_row[];      // [k]
+    __shared__ float part[2][8], red[32];
+    constexpr uint32_t VEC = 16 / sizeof(TW), STEP = 32 * VEC, BATCH = 4, CPG = 8 / KS;
+    const uint32_t lane = threadIdx.x & 31, warp = threadIdx.x >> 5, slice = warp % KS;
+    const uint32_t groups = (a.n + CPG - 1) / CPG, sweeps = (a.k + STEP - 1) / STEP, per = (sweeps + KS - 1) / KS;
+    const uint32_t k_lo = min(a.k, slice * per * STEP), k_hi = min(a.k, (slice + 1) * per * STEP), k_first = k_lo + lane * VEC;
+    const TW* W = reinterpret_cast<const TW*>(a.w);
+    pdl_launch_dependents();
+    uint4 cur[BATCH], nxt[BATCH];
+    auto request = [&](uint4 (&r)[BATCH], uint32_t g, uint32_t kb) {
+        const uint32_t col = g * CPG + warp / KS;
+        if (g < groups && col < a.n) {
+            const TW* w = W + (size_t)col * a.k;
+#pragma unroll
+            for (uint32_t u = 0; u < BATCH; ++u)
+                if (kb + u * STEP < k_hi) r[u] = ldg_stream_u4(w + kb + u * STEP);
+        }
+    };
+    request(cur, blockIdx.x, k_first);                   // weights do not depend on the kernel before
+    pdl_wait();
+    const float4* src = reinterpret_cast<const float4*>(a.a);
+    const uint32_t k4 = a.k / 4;
+    auto at = [&](uint32_t c) { return VEC == 8 ? (c & 1) * (a.k / 2) + (c >> 1) * 4 : c * 4; };      // where float4 c of the row lies
+    float sum = 0.0f;
+    for (uint32_t c = threadIdx.x; c < k4; c += 256) {
+        float4 x = src[c];
+        if (a.a_op) { x.x = dense_a(a, x.x); x.y = dense_a(a, x.y); x.z = dense_a(a, x.z); x.w = dense_a(a, x.w); }
+        sum += (x.x + x.y) + (x.z + x.w);
+        *reinterpret_cast<float4*>(dg_row + at(c)) = x;
+    }
+    if (a.a_norm_weight) {                               // (a thread norms the elements it staged)
+        const float mean = block_sum(sum, red) / (float)a.k;
+        float ss = 0.0f;
+        for (uint32_t c = threadIdx.x; c < k4; c += 256) {
+            const float4 x = *reinterpret_cast<const float4*>(dg_row + at(c));
+            const float d0 = x.x - mean, d1 = x.y - mean, d2 = x.z - mean, d3 = x.w - mean;
+            ss += (d0 * d0 + d1 * d1) + (d2 * d2 + d3 * d3);
+        }
+        const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)a.k + a.a_norm_epsilon);
+        const float4* nw = reinterpret_cast<const float4*>(a.a_norm_weight);
+        for (uint32_t c = threadIdx.x; c < k4; c += 256) {
+            float4 x = *reinterpret_cast<const float4*>(dg_row + at(c));
+            const float4 w = nw[c];
+            x = make_float4((x.x - mean) * inv * w.x, (x.y - mean) * inv * w.y, (x.z - mean) * inv * w.z, (x.w - mean) * inv * w.w);
+            *reinterpret_cast<float4*>(dg_row + at(c)) = x;
+        }
+    }
+    __syncthreads();
+    uint32_t turn = 0;
+    for (uint32_t g = blockIdx.x; g < groups; g += gridDim.x, turn ^= 1) {
+        const uint32_t col = g * CPG + warp / KS;
+        float acc = 0.0f;
+        for (uint32_t kb = k_first; ; kb += BATCH * STEP) {
+            const bool last = kb - lane * VEC + BATCH * STEP >= k_hi;      // uniform over the warp
+            if (last) request(nxt, g + gridDim.x, k_first);
+            else request(nxt, g, kb + BATCH * STEP);
+#pragma unroll
+            for (uint32_t u = 0; u < BATCH; ++u) {
+                const uint32_t k0 = kb + u * STEP;
+                if (k0 < k_hi) {
+                    float wf[VEC];
+                    unpack_weights<VEC, TW>(cur[u], wf);
+#pragma unroll
+                    for (uint32_t i = 0; i < VEC; i += 4) {
+                        const float4 x = *reinterpret_cast<const float4*>(dg_row + at((k0 + i) / 4));
+                        acc = fmaf(x.x, wf[i], acc);
+                        acc = fmaf(x.y, wf[i + 1], acc);
+                        acc = fmaf(x.z, wf[i + 2], acc);
+                        acc = fmaf(x.w, wf[i + 3], acc);
+                    }
+                }
+            }
+#pragma unroll
+            for (uint32_t u = 0; u < BATCH; ++u) cur[u] = nxt[u];
+            if (last) break;
+        }
+        const float s = warp_sum(acc);
+        if constexpr (KS == 1) {
+            if (lane == 0 && col < a.n) dense_store(a, reinterpret_cast<float*>(a.d) + col, 0, 0, col, s);
+        } else {
+            if (lane == 0) part[turn][warp] = s;         // (two buffers: the readers of one group are past it when the next but one writes)
+            __syncthreads();
+            if (slice == 0 && lane == 0 && col < a.n) {
+                float t = 0.0f;
+#pragma unroll
+                for (int q = 0; q < KS; ++q) t += part[turn][warp + q];
+                dense_store(a, reinterpret_cast<float*>(a.d) + col, 0, 0, col, t);
+            }
+        }
+    }
+}
+
+// the shapes it takes (the caller's addresses included)
+static bool dense_gemv_applicable(const uzu_dense_linear_args& a) {
+    const uint32_t vec = a.weights_dt == UZU_DT_BF16 ? 8 : 4;
+    return a.m == 1 && a.batch == 1 && !a.group_offsets && !a.rows_map && !a.pair_rows && !a.a_bf16 && a.k % vec == 0 && a.k > 0 && a.k <= DG_MAX_K &&
+           (a.w & 15) == 0 && (a.a & 15) == 0 && (a.a_norm_weight & 15) == 0;
+}
+
 // ---- tile kernel (f32 multiply-adds) ------------------------------------------------------------------------------------------------
 constexpr int DT_BM = 64, DT_BN = 64, DT_BK = 16;
 
@@ -630,8 +739,9 @@ __global__ void __launch_bounds__(256) dense_tensor128_kernel(const uzu_dense_li
             }
 }
 
-// the rows kernel stages its activation rows under exactly these conditions (its own test of them includes the device addresses)
+// the one-row kernel always stages its row; the rows kernel stages its activation rows under exactly these conditions (its own test of them includes the device addresses)
 bool dense_rows_takes_norm(const uzu_dense_linear_args& a) {
+    if (dense_gemv_applicable(a) && !a.a_op) return true;
     const uint32_t vec = a.weights_dt == UZU_DT_BF16 ? 8 : 4, lda = a.lda ? a.lda : a.k;
     return a.m <= (uint32_t)DL_MAX_ROWS && (size_t)a.m * a.k <= DL_STAGE_FLOATS && a.k % vec == 0 && lda % 4 == 0 && (a.w & 15) == 0 && (a.a & 15) == 0 &&
            a.batch == 1 && !a.group_offsets && !a.rows_map && !a.a_op && !a.a_bf16 && (!a.pair_rows || ((uint64_t)a.pair_rows * a.k) % vec == 0);
@@ -691,6 +801,29 @@ extern "C" void uzu_dense_linear_encode(uzu_command_buffer* cmd, const uzu_dense
         const uint32_t sweep = bf16 ? 256 : 128;
         const uint64_t features = (uint64_t)a.n * a.batch;
         const int ks = (features >= 4096 || a.k < 2 * sweep) ? 1 : (features >= 2048 || a.k < 4 * sweep) ? 2 : 4;
+        static const bool no_gemv = getenv("UZU_DENSE_NO_GEMV") != nullptr;      // A/B runs
+        // (rows longer than the staging size leave room for three CTAs per SM only: the rows kernel reads those from memory and is faster)
+        if (dense_gemv_applicable(a) && ((!no_gemv && a.k <= DL_STAGE_FLOATS) || a.a_norm_weight)) {
+            // at most four CTAs per SM, all with the same number of groups (give or take one)
+            const uint32_t groups = (a.n * ks + 7) / 8, most = 4u * (uint32_t)cmd->ctx->sm_count, rounds = (groups + most - 1) / most;
+            const dim3 g((groups + rounds - 1) / rounds);
+            const size_t smem = (size_t)a.k * sizeof(float);
+            auto gemv = [&](auto kernel, std::atomic<uint64_t>& done) {
+                opt_in_dynamic_smem(cmd, kernel, (int)(DG_MAX_K * sizeof(float)), done);
+                launch(cmd, "dense_gemv_kernel", kernel, g, dim3(256), smem, a);
+            };
+            static std::atomic<uint64_t> done[6];
+            if (bf16) {
+                if (ks == 1) gemv(dense_gemv_kernel<__nv_bfloat16, 1>, done[0]);
+                else if (ks == 2) gemv(dense_gemv_kernel<__nv_bfloat16, 2>, done[1]);
+                else gemv(dense_gemv_kernel<__nv_bfloat16, 4>, done[2]);
+            } else {
+                if (ks == 1) gemv(dense_gemv_kernel<float, 1>, done[3]);
+                else if (ks == 2) gemv(dense_gemv_kernel<float, 2>, done[4]);
+                else gemv(dense_gemv_kernel<float, 4>, done[5]);
+            }
+            return;
+        }
         dim3 grid((a.n * ks + 7) / 8, a.batch);
         auto go = [&](auto kernel) { launch(cmd, "dense_rows_kernel", kernel, grid, dim3(256), 0, a); };
         auto pick = [&](auto tw, auto ks_c, auto pair_c) {
