@@ -3,13 +3,14 @@
 // tile shapes, shared-memory layout and barrier protocol, but the producers have nothing to dequantise -- both operand tiles travel by
 // cp.async straight into their swizzled stage, several K blocks ahead, and no thread touches the data.
 //
-//   CTA = 128 tokens x 128 features, K in blocks of 64, 4 stages of (16 KB activation tile + 16 KB weight tile).
+//   CTA = 128 tokens x 128 features, K in blocks of 64, 3 stages of (16 KB activation tile + 16 KB weight tile): two CTAs share an SM, so one
+//   CTA's epilogue runs beside the other's products (measured: 1024 x 8192 x 2048 in 47 us, 63 us with four stages and one CTA per SM).
 //   warps 0..3 (128 threads): PRODUCERS. Per K block each thread copies 8 + 8 16-byte pieces (8 consecutive lanes per row: whole
 //     128-byte lines) into the K-major SWIZZLE_128B layout (8-row x 128-byte atoms, piece index XOR row-in-atom), waits for its copies
 //     of the block two iterations back, fences them to the async proxy and arrives on the stage's `full` barrier.
 //   warp 4, one lane: MMA ISSUER. Per K block 4 x tcgen05.mma.cta_group::1.kind::f16 (128 x 128 x 16) into 128 TMEM columns, then
 //     tcgen05.commit on the stage's `empty` barrier; after the last block a commit on the accumulator barrier.
-//   warps 0..3 again: EPILOGUE. tcgen05.ld 32 lanes x 32 columns, scale / sigmoid gate / accumulate, f32 stores.
+//   warps 0..3 again: EPILOGUE. tcgen05.ld 32 lanes x 32 columns, scale / factors / bias / gelu / accumulate, 16-byte stores (f32 or bf16).
 // Every barrier wait is bounded (about a second): a wait that runs out sets an error word, the CTA stops working, still meets at the
 // final barrier, frees its tensor memory and returns.
 #include "common.cuh"
@@ -34,7 +35,7 @@ struct DenseUmmaParams {
 __device__ unsigned int g_dense_umma_error = 0;
 
 constexpr uint32_t DU_TILE_BYTES = 128 * 64 * 2;
-constexpr int DU_STAGES = 4;
+constexpr int DU_STAGES = 3;
 constexpr int DU_NP = 128;
 constexpr uint32_t DU_STAGE_BYTES = 2 * DU_TILE_BYTES;
 
@@ -73,6 +74,9 @@ __device__ __forceinline__ void du_cp_async16(uint32_t dst_smem, const void* src
 }
 __device__ __forceinline__ uint32_t du_tile_off(uint32_t row, uint32_t ch) { return row * 128u + ((ch ^ (row & 7u)) << 4); }
 
+enum DuEpilogue : int { DuPlain = 0 /* scale, bias, accumulate */, DuGelu = 1 /* the exact gelu besides */, DuGeneral = 2 /* gate, row and column factors besides */ };
+
+template <int EPI>
 __global__ void __launch_bounds__(DU_NP + 32, 1) dense_umma_kernel(const DenseUmmaParams p) {
     extern __shared__ uint8_t du_smem_raw[];
     __shared__ __align__(8) uint64_t bars[2 * DU_STAGES + 1];
@@ -171,19 +175,73 @@ __global__ void __launch_bounds__(DU_NP + 32, 1) dense_umma_kernel(const DenseUm
                 __nv_bfloat16* out16 = reinterpret_cast<__nv_bfloat16*>(p.d) + (size_t)row * p.ldd + col0;
                 const float* gate = p.gate ? p.gate + (size_t)row * p.gate_ld + col0 : nullptr;
                 const float rs = p.row_scale ? p.row_scale[row] : 1.0f;
+                // A thread holds 32 consecutive elements of one row: whole column blocks of aligned rows move as 16-byte pieces. The kinds of epilogue
+                // are kernels of their own: one loop that could do everything is 32 copies of an exponential and an error function.
+                const bool whole = col0 + 32u <= p.n, vec = whole && p.ldd % 8u == 0;
 #pragma unroll
                 for (int j = 0; j < 32; ++j) {
-                    if (col0 + (uint32_t)j < p.n) {
-                        float val = __uint_as_float(v[j]) * p.scale;
-                        if (p.row_scale) val *= rs;
-                        if (gate) val *= 1.0f / (1.0f + expf(-(gate[j] + (p.gate_bias ? p.gate_bias[col0 + j] : 0.0f))));
-                        if (p.col_scale) val *= p.col_scale[col0 + j];
-                        if (p.bias) val += p.bias[col0 + j];
-                        if (p.d_op == 1) val = 0.5f * val * (1.0f + erff(val * 0.70710678118654752f));
-                        if (p.d_bf16) { out16[j] = __float2bfloat16_rn(val); continue; }
-                        if (p.accumulate) val += out[j];
-                        out[j] = val;
+                    float val = __uint_as_float(v[j]) * p.scale;
+                    if constexpr (EPI == DuGeneral) {
+                        if (whole || col0 + (uint32_t)j < p.n) {
+                            if (p.row_scale) val *= rs;
+                            if (gate) val *= 1.0f / (1.0f + expf(-(gate[j] + (p.gate_bias ? p.gate_bias[col0 + j] : 0.0f))));
+                            if (p.col_scale) val *= p.col_scale[col0 + j];
+                        }
                     }
+                    v[j] = __float_as_uint(val);
+                }
+                if (p.bias) {
+#pragma unroll
+                    for (int j = 0; j < 32; ++j)
+                        if (whole || col0 + (uint32_t)j < p.n) v[j] = __float_as_uint(__uint_as_float(v[j]) + p.bias[col0 + j]);
+                }
+                if constexpr (EPI == DuGelu) {
+#pragma unroll
+                    for (int j = 0; j < 32; ++j) {
+                        const float z = __uint_as_float(v[j]);
+                        v[j] = __float_as_uint(0.5f * z * (1.0f + erff(z * 0.70710678118654752f)));
+                    }
+                }
+                if (p.accumulate) {
+#pragma unroll
+                    for (int j = 0; j < 32; j += 4) {
+                        if (vec) {
+                            const float4 o4 = *reinterpret_cast<const float4*>(out + j);
+                            v[j] = __float_as_uint(__uint_as_float(v[j]) + o4.x);
+                            v[j + 1] = __float_as_uint(__uint_as_float(v[j + 1]) + o4.y);
+                            v[j + 2] = __float_as_uint(__uint_as_float(v[j + 2]) + o4.z);
+                            v[j + 3] = __float_as_uint(__uint_as_float(v[j + 3]) + o4.w);
+                        } else {
+#pragma unroll
+                            for (int i = j; i < j + 4; ++i)
+                                if (col0 + (uint32_t)i < p.n) v[i] = __float_as_uint(__uint_as_float(v[i]) + out[i]);
+                        }
+                    }
+                }
+                if (p.d_bf16) {
+#pragma unroll
+                    for (int j = 0; j < 32; j += 8) {
+                        uint32_t w[4];
+#pragma unroll
+                        for (int i = 0; i < 4; ++i) {
+                            const __nv_bfloat162 h = __floats2bfloat162_rn(__uint_as_float(v[j + 2 * i]), __uint_as_float(v[j + 2 * i + 1]));
+                            w[i] = *reinterpret_cast<const uint32_t*>(&h);
+                        }
+                        if (vec) {
+                            *reinterpret_cast<uint4*>(out16 + j) = make_uint4(w[0], w[1], w[2], w[3]);
+                        } else {
+#pragma unroll
+                            for (int i = 0; i < 8; ++i)
+                                if (col0 + (uint32_t)(j + i) < p.n) out16[j + i] = __float2bfloat16_rn(__uint_as_float(v[j + i]));
+                        }
+                    }
+                } else if (vec) {
+#pragma unroll
+                    for (int j = 0; j < 32; j += 4) *reinterpret_cast<uint4*>(out + j) = make_uint4(v[j], v[j + 1], v[j + 2], v[j + 3]);
+                } else {
+#pragma unroll
+                    for (int j = 0; j < 32; ++j)
+                        if (col0 + (uint32_t)j < p.n) out[j] = __uint_as_float(v[j]);
                 }
             }
         }
@@ -247,6 +305,8 @@ bool dense_umma_applicable(const uzu_dense_linear_args& a) {
     static const bool off = getenv("UZU_DENSE_NO_UMMA") != nullptr;      // A/B runs
     if (off || !a.workspace || a.weights_dt != UZU_DT_BF16 || a.batch != 1 || a.group_offsets || a.rows_map || a.pair_rows) return false;
     if (a.m < 128 || a.k % 64u != 0 || a.n < 64) return false;
+    if ((a.d & 15u) && (a.ldd ? a.ldd : a.n) % 8u == 0) return false;      // rows of whole 16-byte pieces are stored as such
+    if (a.d_op && (a.gate || a.row_scale || a.col_scale)) return false;
     if ((a.a & 15u) || (a.w & 15u) || (a.workspace & 15u) || a.lda % 4u != 0) return false;
     return true;
 }
@@ -279,9 +339,14 @@ void encode_dense_umma(uzu_command_buffer* cmd, const uzu_dense_linear_args& a) 
     cudaGetSymbolAddress(&err, g_dense_umma_error);
     p.error = (unsigned int*)err;
     constexpr size_t smem = (size_t)DU_STAGES * DU_STAGE_BYTES + 1024;
-    static std::atomic<uint64_t> opt_in{0};
-    opt_in_dynamic_smem(cmd, dense_umma_kernel, (int)smem, opt_in);
-    launch(cmd, "dense_umma_kernel", dense_umma_kernel, dim3((a.n + 127u) / 128u, (a.m + 127u) / 128u), dim3(DU_NP + 32), smem, p);
+    auto go = [&](auto kernel, std::atomic<uint64_t>& opt_in) {
+        opt_in_dynamic_smem(cmd, kernel, (int)smem, opt_in);
+        launch(cmd, "dense_umma_kernel", kernel, dim3((a.n + 127u) / 128u, (a.m + 127u) / 128u), dim3(DU_NP + 32), smem, p);
+    };
+    static std::atomic<uint64_t> opt_in[3];
+    if (a.gate || a.row_scale || a.col_scale) go(dense_umma_kernel<DuGeneral>, opt_in[2]);
+    else if (a.d_op == 1) go(dense_umma_kernel<DuGelu>, opt_in[1]);
+    else go(dense_umma_kernel<DuPlain>, opt_in[0]);
 }
 
 }  // namespace uzu
