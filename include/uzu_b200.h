@@ -480,7 +480,7 @@ typedef struct uzu_dense_linear_args {
                                       g = A.W[col], u = A.W[col + pair_rows] and stores the clamped gated unit
                                       min(g, limit) * sigmoid(alpha * min(g, limit)) * (clamp(u, -limit, limit) + 1) */
     float glu_limit, glu_alpha;
-    uint32_t glu_kind;             /* paired epilogue: 0 the clamped unit above, 1 g * sigmoid(g) * u */
+    uint32_t glu_kind;             /* paired epilogue: 0 the clamped unit above, 1 g * sigmoid(g) * u, 2 gelu_tanh(g) * u */
     uint32_t d_op;                 /* applied to the finished element (after scale, gate and bias): 0 none, 1 the exact gelu z * Phi(z) */
     uint64_t gate_bias;            /* optional f32 [n] (with gate): sigmoid(gate[row, col] + gate_bias[col]) */
     uint64_t col_scale;            /* optional f32 [n]: the product is multiplied by col_scale[col] (a per-channel layer scale) */
@@ -509,7 +509,14 @@ typedef struct uzu_dense_linear_args {
     float a_norm_epsilon;
     uint32_t streams;
     uint32_t d_bf16;               /* 1: D is bf16 [m, ldd] (tcgen05 form only, no accumulate): the next product's A rows */
-    uint32_t reserved1;
+    /* Residual prologue (a_residual != 0, with a_norm_weight; a single row, one plain or paired product): A is a sublayer's raw result y, and the
+     * product reads the residual stream after it took y in,
+     *   x = a_residual[k] + a_residual_mult * (y - mean(y)) / sqrt(variance(y) + a_norm_epsilon) * a_norm_weight[k],
+     * which is also stored to a_residual_out (f32 [k], not the same rows as a_residual: other CTAs still read those). */
+    float a_residual_mult;
+    uint64_t a_residual, a_residual_out;
+    float glu_limit_last;          /* paired epilogue with row groups: the limit of the groups from index glu_last_group on (0: all take glu_limit) */
+    uint32_t glu_last_group;
 } uzu_dense_linear_args;
 UZU_API void uzu_dense_linear_encode(uzu_command_buffer* cmd, const uzu_dense_linear_args* args);
 /* 0, or the code of the first bounded barrier wait that ran out inside a tensor-memory dense product (the kernel gives up and returns) */
@@ -539,7 +546,7 @@ typedef struct uzu_norm_add_args {
     uint64_t input, weight, bias, residual, output, next_weight, next_bias;
     uint32_t rows, n, in_stride, kind, next_kind;
     float alpha, epsilon, mult, next_alpha;
-    uint32_t reserved;
+    uint32_t residual_bf16;        /* 1 (with a residual): `output` is the updated residual itself as bf16 rows (no next norm), A rows of a product */
 } uzu_norm_add_args;
 UZU_API void uzu_norm_add_encode(uzu_command_buffer* cmd, const uzu_norm_add_args* args);
 
@@ -579,6 +586,25 @@ UZU_API void uzu_embedding_f32_encode(uzu_command_buffer* cmd, uint64_t token_id
 /*   embedding_f32_scaled: the same rows times `scale` */
 UZU_API void uzu_embedding_f32_scaled_encode(uzu_command_buffer* cmd, uint64_t token_ids, uint64_t table, uint32_t weights_dt, uint64_t output,
                                              uint32_t rows, uint32_t vocab, uint32_t n, float scale);
+/* Embedding rows into the f32 residual stream, out[r, :] = scale * table[token[r], :] (ids >= vocab read 0), with position_turns != 0 plus the
+ * sinusoidal vector of the row's position p = prefix + r (prefix read from dynamic_position when non-zero): channel 2i gets sin(2 pi p
+ * position_turns[i]), channel 2i + 1 the cosine. position_turns f64 [(n + 1) / 2] holds turns per token, so that only the fraction of p * turns
+ * reaches the sine. rows_bf16 (optional, bf16 [rows, n]): a second copy, A rows of a product. */
+typedef struct uzu_embedding_f32_args {
+    uint64_t token_ids, table, output, position_turns, dynamic_position, rows_bf16;
+    uint32_t rows, vocab, n, weights_dt, prefix;
+    float scale;
+} uzu_embedding_f32_args;
+UZU_API void uzu_embedding_f32_position_encode(uzu_command_buffer* cmd, const uzu_embedding_f32_args* args);
+/* The gated unit of a product's [gate | up] rows: f32 [rows, 2f] -> f32 or (output_bf16) bf16 [rows, f].
+ *   kind 0: min(g, limit) * sigmoid(alpha min(g, limit)) * (clamp(u, -limit, limit) + 1);  1: g * sigmoid(g) * u;  2: gelu_tanh(g) * u
+ * Rows from group_offsets[last_group] on (a u32 list on the device, optional) take limit_last instead of limit. */
+typedef struct uzu_glu_args {
+    uint64_t gate_up, output, group_offsets;
+    uint32_t rows, f, kind, output_bf16, last_group;
+    float limit, limit_last, alpha;
+} uzu_glu_args;
+UZU_API void uzu_glu_encode(uzu_command_buffer* cmd, const uzu_glu_args* args);
 UZU_API void uzu_clamped_glu_encode(uzu_command_buffer* cmd, uint64_t gate_up, uint64_t output, uint32_t rows, uint32_t f, float limit, float alpha);
 /*   silu_glu:        out = g * sigmoid(g) * u, same operand layout as clamped_glu */
 UZU_API void uzu_silu_glu_encode(uzu_command_buffer* cmd, uint64_t gate_up, uint64_t output, uint32_t rows, uint32_t f);
@@ -604,10 +630,19 @@ UZU_API void uzu_routed_combine_encode(uzu_command_buffer* cmd, uint64_t pairs, 
 typedef struct uzu_topk_route_args {
     uint64_t logits /* f32 [rows, logits_stride] */, bias /* optional f32 [experts] */, group_offsets, rows_map, pair_pos, pair_weight;
     uint32_t rows, top, experts, logits_stride;
-    uint32_t weight_kind;          /* 0: softmax over the chosen logits; 1: sigmoid of each chosen logit on its own (not renormalised) */
-    uint32_t reserved;
+    uint32_t weight_kind;          /* 0: softmax over the chosen logits; 1: sigmoid of each chosen logit on its own (not renormalised);
+                                      2: corrected choice, see below */
+    uint32_t always;               /* experts [experts, experts + always) are used by every row with weight 1: they take the row's last `always` slots,
+                                      a row then has top + always pairs (all pair arrays are sized and indexed so) */
     uint64_t compact_weight;       /* optional f32 [rows*top]: the same weights in the compact (expert-sorted) order of rows_map */
     uint64_t scratch;              /* optional u16 [rows*top]: with it, passes of >= 64 rows make the choice over many CTAs (a second launch sorts) */
+    /* weight_kind 2: s = sigmoid(logit + bias), choice score c = s + correction. The experts form choice_groups equal groups of neighbours (0 / 1: one);
+     * a group's score is the sum of its two largest c (of its only one), and the experts of the choice_keep best groups can be chosen. The `top`
+     * largest c are taken; weights are their s over the sum of the chosen s (+ 1e-20), times weight_scale. */
+    uint64_t correction;           /* optional f32 [experts] */
+    uint32_t choice_groups, choice_keep;
+    float weight_scale;
+    uint32_t reserved;
 } uzu_topk_route_args;
 UZU_API void uzu_topk_route_encode(uzu_command_buffer* cmd, const uzu_topk_route_args* args);
 
@@ -676,7 +711,7 @@ typedef struct uzu_head_norm_gate_args {
     uint32_t gate_op, reserved;
     uint64_t denom, denom_floor;
     float denom_epsilon;
-    uint32_t reserved1;
+    float out_scale;               /* the result is multiplied by this factor (0 = 1) */
 } uzu_head_norm_gate_args;
 UZU_API void uzu_head_norm_gate_encode(uzu_command_buffer* cmd, const uzu_head_norm_gate_args* args);
 
@@ -732,7 +767,7 @@ typedef struct uzu_retention_args {
     uint64_t q, k, v, decay /* f32 [heads] */, state, out;
     uint32_t rows, heads, dim, vdim, q_stride, k_stride, v_stride, out_stride;
     float key_scale;
-    uint32_t reserved;
+    uint32_t input_op;             /* applied to every q, k and v element as it is read: 0 none, 1 silu (not with the gated form) */
     /* Gated form (token_decay != 0; `decay` is then unused): the factors change from token to token,
      *   S_t = token_decay[t, h] * S_(t-1) + token_gain[t, h] * (key_scale * k_t) v_t^T,   out[t, h, :] = S_t^T (query_scale * q_t)
      * and, with norm_out, a normaliser n_t = token_decay n_(t-1) + token_gain * key_scale * k_t is kept as one more state column:
@@ -818,7 +853,8 @@ UZU_API void uzu_window_attention_prepare_encode(uzu_command_buffer* cmd, const 
  * first tokens: key j is visible when j <= p and (p - j < window or j < keep_first); window = 0 means no window; a chunk bounds the
  * window's keys to the query's own chunk. Query head h reads
  * key / value head h / (heads / kv_heads).
- *   s = scale * head_temp[h] * query . key;  softcap > 0: s <- softcap * tanh(s / softcap);  weights = softmax over the visible keys
+ *   s = scale * head_temp[h] * query . key;  softcap > 0: s <- softcap * tanh(s / softcap);  s <- s - dist_slope[h] * (p - j);
+ *   weights = softmax over the visible keys
  *   out[t, h, :] = rotate_(-p)(sum_j weight_j * values[j, g, :])   (the rotation back over 2 * v_pairs channels only when v_pairs > 0)
  * Scores, weights and sums are f32. bf16 caches with rows >= 64 and dim, vdim multiples of 16 up to 128 run on the tensor pipe with the
  * query and the weights each as a sum of two bf16 numbers (hi + lo). Few rows: the visible keys of a query are cut into `splits` parts,
@@ -835,6 +871,9 @@ typedef struct uzu_window_attention_args {
     uint64_t sinks;                /* optional f32 [heads]: the softmax denominator also holds exp(sinks[h]) (no key, no value, not scaled) */
     uint64_t head_gate;            /* optional f32 [rows, head_gate_stride]: head h's output is multiplied by sigmoid(head_gate[t, h]) */
     uint32_t chunk;                /* > 0: only keys of the query's own chunk are visible, floor(j / chunk) = floor(p / chunk), counted from position 0 */
+    uint32_t out_stride;           /* f32 elements between output rows (0 = heads * vdim) */
+    uint64_t dist_slope;           /* optional f32 [heads]: the score loses dist_slope[h] per position of distance */
+    float out_scale;               /* the output is multiplied by this factor (0 = 1) */
     uint32_t reserved;
 } uzu_window_attention_args;
 UZU_API void uzu_window_attention_encode(uzu_command_buffer* cmd, const uzu_window_attention_args* args);

@@ -141,7 +141,15 @@ DenseLinearArgs = _struct("uzu_dense_linear_args", [
     ("post_alpha", f32), ("post_mult", f32), ("next_alpha", f32), ("token_gate_dt", u32), ("token_ids", u64), ("token_table", u64),
     ("token_table_stride", u32), ("token_column", u32), ("token_vocab", u32), ("a_bf16", u32),
     ("stream_x", u64), ("stream_mix", u64), ("stream_out", u64), ("stream_in", u64), ("stream_u", u64), ("a_norm_weight", u64), ("a_norm_epsilon", f32),
-    ("streams", u32), ("d_bf16", u32), ("reserved1", u32)])
+    ("streams", u32), ("d_bf16", u32), ("a_residual_mult", f32), ("a_residual", u64), ("a_residual_out", u64), ("glu_limit_last", f32), ("glu_last_group", u32)])
+
+EmbeddingF32Args = _struct("uzu_embedding_f32_args", [
+    ("token_ids", u64), ("table", u64), ("output", u64), ("position_turns", u64), ("dynamic_position", u64), ("rows_bf16", u64),
+    ("rows", u32), ("vocab", u32), ("n", u32), ("weights_dt", u32), ("prefix", u32), ("scale", f32)])
+
+GluArgs = _struct("uzu_glu_args", [
+    ("gate_up", u64), ("output", u64), ("group_offsets", u64), ("rows", u32), ("f", u32), ("kind", u32), ("output_bf16", u32), ("last_group", u32),
+    ("limit", f32), ("limit_last", f32), ("alpha", f32)])
 
 GroupRmsNormArgs = _struct("uzu_group_rms_norm_args", [
     ("input", u64), ("scales", u64), ("output", u64), ("row_indices", u64),
@@ -160,7 +168,7 @@ GeneralDeltaArgs = _struct("uzu_general_delta_args", [
 HeadNormGateArgs = _struct("uzu_head_norm_gate_args", [
     ("x", u64), ("scales", u64), ("gate", u64), ("out", u64),
     ("rows", u32), ("heads", u32), ("dim", u32), ("x_stride", u32), ("gate_stride", u32), ("out_stride", u32), ("normalize", u32),
-    ("epsilon", f32), ("gate_op", u32), ("reserved", u32), ("denom", u64), ("denom_floor", u64), ("denom_epsilon", f32), ("reserved1", u32)])
+    ("epsilon", f32), ("gate_op", u32), ("reserved", u32), ("denom", u64), ("denom_floor", u64), ("denom_epsilon", f32), ("out_scale", f32)])
 
 LatentPrepareArgs = _struct("uzu_latent_prepare_args", [
     ("kv", u64), ("q", u64), ("query", u64), ("cache", u64), ("latent_scales", u64), ("cosines", u64), ("sines", u64),
@@ -176,7 +184,8 @@ LatentAttentionArgs = _struct("uzu_latent_attention_args", [
 
 TopkRouteArgs = _struct("uzu_topk_route_args", [
     ("logits", u64), ("bias", u64), ("group_offsets", u64), ("rows_map", u64), ("pair_pos", u64), ("pair_weight", u64),
-    ("rows", u32), ("top", u32), ("experts", u32), ("logits_stride", u32), ("weight_kind", u32), ("reserved", u32), ("compact_weight", u64), ("scratch", u64)])
+    ("rows", u32), ("top", u32), ("experts", u32), ("logits_stride", u32), ("weight_kind", u32), ("always", u32), ("compact_weight", u64), ("scratch", u64),
+    ("correction", u64), ("choice_groups", u32), ("choice_keep", u32), ("weight_scale", f32), ("reserved", u32)])
 
 RoutedCombineArgs = _struct("uzu_routed_combine_args", [
     ("pairs", u64), ("pair_pos", u64), ("pair_weight", u64), ("gate", u64), ("gate_bias", u64), ("col_scale", u64), ("output", u64),
@@ -201,7 +210,7 @@ MinGruArgs = _struct("uzu_min_gru_args", [
 RetentionArgs = _struct("uzu_retention_args", [
     ("q", u64), ("k", u64), ("v", u64), ("decay", u64), ("state", u64), ("out", u64),
     ("rows", u32), ("heads", u32), ("dim", u32), ("vdim", u32), ("q_stride", u32), ("k_stride", u32), ("v_stride", u32), ("out_stride", u32),
-    ("key_scale", f32), ("reserved", u32), ("token_decay", u64), ("token_gain", u64), ("norm_out", u64), ("query_scale", f32), ("reserved1", u32)])
+    ("key_scale", f32), ("input_op", u32), ("token_decay", u64), ("token_gain", u64), ("norm_out", u64), ("query_scale", f32), ("reserved1", u32)])
 
 ExpGatesArgs = _struct("uzu_exp_gates_args", [
     ("i_pre", u64), ("f_pre", u64), ("state", u64), ("token_decay", u64), ("token_gain", u64), ("floor", u64),
@@ -210,7 +219,7 @@ ExpGatesArgs = _struct("uzu_exp_gates_args", [
 NormAddArgs = _struct("uzu_norm_add_args", [
     ("input", u64), ("weight", u64), ("bias", u64), ("residual", u64), ("output", u64), ("next_weight", u64), ("next_bias", u64),
     ("rows", u32), ("n", u32), ("in_stride", u32), ("kind", u32), ("next_kind", u32),
-    ("alpha", f32), ("epsilon", f32), ("mult", f32), ("next_alpha", f32), ("reserved", u32)])
+    ("alpha", f32), ("epsilon", f32), ("mult", f32), ("next_alpha", f32), ("residual_bf16", u32)])
 
 TokenGateArgs = _struct("uzu_token_gate_args", [
     ("z", u64), ("token_ids", u64), ("table", u64), ("out", u64),
@@ -227,7 +236,7 @@ WindowAttentionArgs = _struct("uzu_window_attention_args", [
     ("v_cosines", u64), ("v_sines", u64), ("partials", u64), ("tickets", u64),
     ("rows", u32), ("heads", u32), ("kv_heads", u32), ("dim", u32), ("vdim", u32), ("prefix", u32), ("cache_dt", u32), ("window", u32),
     ("keep_first", u32), ("v_pairs", u32), ("scale", f32), ("softcap", f32), ("splits", u32), ("head_gate_stride", u32), ("sinks", u64), ("head_gate", u64),
-    ("chunk", u32), ("reserved", u32)])
+    ("chunk", u32), ("out_stride", u32), ("dist_slope", u64), ("out_scale", f32), ("reserved", u32)])
 
 StreamMixArgs = _struct("uzu_stream_mix_args", [
     ("x", u64), ("y", u64), ("mix", u64), ("out", u64), ("read", u64), ("u", u64), ("weight", u64), ("output", u64), ("token_ids", u64), ("table", u64),
@@ -246,7 +255,7 @@ GatedDeltaStepArgs = _struct("uzu_gated_delta_step_args", [
 
 MAIN_SLOT = 0xFFFFFFFF
 
-ABI_STRUCTS = [StreamMixArgs, DeltaPrepareArgs, GatedDeltaArgs, GatedDeltaStepArgs, ExpGatesArgs, NormAddArgs, TokenGateArgs, MinGruArgs, RetentionArgs, WindowAttentionPrepareArgs, WindowAttentionArgs, TopkRouteArgs, RoutedCombineArgs, SigmoidAttentionPrepareArgs, SigmoidAttentionArgs, DenseLinearArgs, GroupRmsNormArgs, TableRouteArgs, GeneralDeltaArgs, HeadNormGateArgs, LatentPrepareArgs, LatentAttentionArgs,
+ABI_STRUCTS = [EmbeddingF32Args, GluArgs, StreamMixArgs, DeltaPrepareArgs, GatedDeltaArgs, GatedDeltaStepArgs, ExpGatesArgs, NormAddArgs, TokenGateArgs, MinGruArgs, RetentionArgs, WindowAttentionPrepareArgs, WindowAttentionArgs, TopkRouteArgs, RoutedCombineArgs, SigmoidAttentionPrepareArgs, SigmoidAttentionArgs, DenseLinearArgs, GroupRmsNormArgs, TableRouteArgs, GeneralDeltaArgs, HeadNormGateArgs, LatentPrepareArgs, LatentAttentionArgs,
                DeltaNetFusedUpdateArgs, QkNormConfig, AttentionPrepareNormArgs, FusedLinearArgs, RingParams, TrieNode, KvCopy, MatmulArgs, NormalizationArgs, QkvNormArgs, AttentionPrepareArgs, AttentionArgs,
                AttentionTwoPass2Args, KvCacheUpdateArgs, GatedActMulArgs, QuantizedEmbeddingLookupArgs, UnifiedSamplingArgs,
                DeltaNetConvUpdateArgs, DeltaNetUpdateArgs, EngineOptions, SamplingMethod, ModelInfo, TpAllGatherArgs]
@@ -281,7 +290,7 @@ uzu_silu_glu_encode uzu_topk_route_encode uzu_routed_combine_gated_encode uzu_si
 uzu_engine_slot_acquire uzu_engine_slot_release uzu_engine_forward_rows uzu_engine_debug_layer_outputs uzu_debug_dense_umma_error
 uzu_min_gru_encode uzu_retention_encode uzu_window_attention_prepare_encode uzu_window_attention_encode
 uzu_exp_gates_encode uzu_norm_add_encode uzu_token_gate_encode uzu_embedding_f32_scaled_encode uzu_rows_to_bf16_encode
-uzu_stream_mix_encode uzu_delta_prepare_encode uzu_gated_delta_encode uzu_gated_delta_step_encode""".split()
+uzu_embedding_f32_position_encode uzu_glu_encode uzu_stream_mix_encode uzu_delta_prepare_encode uzu_gated_delta_encode uzu_gated_delta_step_encode""".split()
 
 _lib = None
 
@@ -445,6 +454,8 @@ def load() -> C.CDLL:
         "uzu_token_gate_encode": (None, [vp, C.POINTER(TokenGateArgs)]),
         "uzu_rows_to_bf16_encode": (None, [vp, u64, u32, u64, u32, u32]),
         "uzu_embedding_f32_scaled_encode": (None, [vp, u64, u64, u32, u64, u32, u32, u32, f32]),
+        "uzu_embedding_f32_position_encode": (None, [vp, C.POINTER(EmbeddingF32Args)]),
+        "uzu_glu_encode": (None, [vp, C.POINTER(GluArgs)]),
         "uzu_engine_slot_acquire": (C.c_int, [vp, C.POINTER(u32)]),
         "uzu_engine_slot_release": (C.c_int, [vp, u32]),
         "uzu_engine_forward_rows": (C.c_int, [vp, u32, C.POINTER(u32), u32, C.POINTER(u32), u32, C.POINTER(C.c_float)]),

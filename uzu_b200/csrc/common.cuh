@@ -108,6 +108,8 @@ void encode_prefill_gemm(uzu_command_buffer* cmd, const uzu_matmul_args& a);
 
 // whether a dense product runs on the kernel that can norm its A rows as it stages them (dense_linear.cu)
 bool dense_rows_takes_norm(const uzu_dense_linear_args& a);
+// whether a dense product runs on the one-row kernel, which can take a sublayer's result into the residual as it stages its row (dense_linear.cu)
+bool dense_takes_residual(const uzu_dense_linear_args& a);
 // whether a dense product runs on tcgen05 with its operands in tensor memory (dense_umma.cu)
 bool dense_umma_applicable(const uzu_dense_linear_args& a);
 

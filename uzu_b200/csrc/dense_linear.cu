@@ -1,6 +1,7 @@
 // Dense (unquantised) linear: D (+)= scale * A . W^T, f32 activations, bf16 or f32 weights [n, k], f32 accumulation.
 // Four kernels behind one entry point (uzu_dense_linear_encode):
-//   one-row kernel (a single row, one plain product): the same weight pass with CTAs that stay for many output features;
+//   one-row kernel (a single row, one plain or paired product): the same weight pass with CTAs that stay for many output features; it can
+//                 layer-norm the row it stages, and take it into a residual stream first;
 //   rows kernel   (<= 8 rows per group): one warp per output feature, the weight row streamed once with 128-bit loads and multiplied
 //                 with every activation row in f32 -- the decode step's weight pass, bound by the weight bytes;
 //   tensor kernels (bf16 weights, >= 32 rows): 64 x 64 output tiles (128 x 128 with ldmatrix fragments from 96 rows on) on
@@ -137,6 +138,13 @@ __device__ __forceinline__ float clamped_glu_value(float g, float u, float limit
     g = fminf(g, limit);
     u = fminf(fmaxf(u, -limit), limit);
     return g * (1.0f / (1.0f + expf(-alpha * g))) * (u + 1.0f);
+}
+
+// the paired epilogue of weight block z
+__device__ __forceinline__ float pair_value(const uzu_dense_linear_args& a, uint32_t z, float g, float u) {
+    if (a.glu_kind == 1) return g * (1.0f / (1.0f + expf(-g))) * u;
+    if (a.glu_kind == 2) return 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
+    return clamped_glu_value(g, u, a.glu_last_group && z >= a.glu_last_group ? a.glu_limit_last : a.glu_limit, a.glu_alpha);
 }
 
 constexpr uint32_t DL_STAGE_FLOATS = 8192;   // activation rows of a group are staged in shared memory when they fit (32 KB)
@@ -295,7 +303,7 @@ __global__ void __launch_bounds__(256, RMAX == 1 ? 4 : 2) dense_rows_kernel(cons
         if constexpr (PAIR) {
             if (a.row_scale) { const float rs = reinterpret_cast<const float*>(a.row_scale)[R.begin + r]; s *= rs; s2 *= rs; }
         }
-        if constexpr (PAIR) *d = a.glu_kind == 1 ? s * (1.0f / (1.0f + expf(-s))) * s2 : clamped_glu_value(s, s2, a.glu_limit, a.glu_alpha);
+        if constexpr (PAIR) *d = pair_value(a, z, s, s2);
         else dense_store(a, d, z, R.begin + r, col, s);
     };
 #pragma unroll
@@ -328,34 +336,38 @@ __global__ void __launch_bounds__(256, RMAX == 1 ? 4 : 2) dense_rows_kernel(cons
     }
 }
 
-// ---- one activation row, one plain product: the decode step's usual shape --------------------------------------------------------------
+// ---- one activation row, one plain or paired product: the decode step's usual shape --------------------------------------------------------------
 // CTAs stay for several groups of output features: the activation row is staged (and, with a_norm_weight, layer-normed) once per CTA, and the
 // weights of a warp's next batch -- of the next feature, too -- are requested before the current batch is used, so the weight stream does
 // not stop between features. KS warps share a feature as in the rows kernel. bf16 weights: the row is kept as two planes (the first and the
-// second float4 of every eight elements), so that a warp's 16-byte reads fall into different banks.
+// second float4 of every eight elements), so that a warp's 16-byte reads fall into different banks. PAIR: a warp streams two weight rows.
+// With a_residual the staged row is a sublayer's raw result: every CTA forms x = residual + mult * norm(row) for itself, the first one stores it.
 constexpr uint32_t DG_MAX_K = 16384;
 
-template <typename TW, int KS>
+template <typename TW, int KS, bool PAIR>
 __global__ void __launch_bounds__(256, 4) dense_gemv_kernel(const uzu_dense_linear_args a) {
     extern __shared__ __align__(16) float dg_row[];      // [k]
-    __shared__ float part[2][8], red[32];
-    constexpr uint32_t VEC = 16 / sizeof(TW), STEP = 32 * VEC, BATCH = 4, CPG = 8 / KS;
+    __shared__ float part[2][PAIR ? 2 : 1][8], red[32];
+    constexpr uint32_t VEC = 16 / sizeof(TW), STEP = 32 * VEC, BATCH = PAIR ? 2 : 4, CPG = 8 / KS;
     const uint32_t lane = threadIdx.x & 31, warp = threadIdx.x >> 5, slice = warp % KS;
     const uint32_t groups = (a.n + CPG - 1) / CPG, sweeps = (a.k + STEP - 1) / STEP, per = (sweeps + KS - 1) / KS;
     const uint32_t k_lo = min(a.k, slice * per * STEP), k_hi = min(a.k, (slice + 1) * per * STEP), k_first = k_lo + lane * VEC;
     const TW* W = reinterpret_cast<const TW*>(a.w);
     pdl_launch_dependents();
-    uint4 cur[BATCH], nxt[BATCH];
-    auto request = [&](uint4 (&r)[BATCH], uint32_t g, uint32_t kb) {
+    uint4 cur[BATCH], nxt[BATCH], cur2[PAIR ? BATCH : 1], nxt2[PAIR ? BATCH : 1];
+    auto request = [&](uint4 (&r)[BATCH], uint4 (&r2)[PAIR ? BATCH : 1], uint32_t g, uint32_t kb) {
         const uint32_t col = g * CPG + warp / KS;
         if (g < groups && col < a.n) {
             const TW* w = W + (size_t)col * a.k;
 #pragma unroll
             for (uint32_t u = 0; u < BATCH; ++u)
-                if (kb + u * STEP < k_hi) r[u] = ldg_stream_u4(w + kb + u * STEP);
+                if (kb + u * STEP < k_hi) {
+                    r[u] = ldg_stream_u4(w + kb + u * STEP);
+                    if constexpr (PAIR) r2[u] = ldg_stream_u4(w + (size_t)a.pair_rows * a.k + kb + u * STEP);
+                }
         }
     };
-    request(cur, blockIdx.x, k_first);                   // weights do not depend on the kernel before
+    request(cur, cur2, blockIdx.x, k_first);             // weights do not depend on the kernel before
     pdl_wait();
     const float4* src = reinterpret_cast<const float4*>(a.a);
     const uint32_t k4 = a.k / 4;
@@ -377,10 +389,17 @@ __global__ void __launch_bounds__(256, 4) dense_gemv_kernel(const uzu_dense_line
         }
         const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)a.k + a.a_norm_epsilon);
         const float4* nw = reinterpret_cast<const float4*>(a.a_norm_weight);
+        const float4* res = reinterpret_cast<const float4*>(a.a_residual);
         for (uint32_t c = threadIdx.x; c < k4; c += 256) {
             float4 x = *reinterpret_cast<const float4*>(dg_row + at(c));
             const float4 w = nw[c];
             x = make_float4((x.x - mean) * inv * w.x, (x.y - mean) * inv * w.y, (x.z - mean) * inv * w.z, (x.w - mean) * inv * w.w);
+            if (res) {
+                const float4 r = res[c];
+                const float m = a.a_residual_mult;
+                x = make_float4(fmaf(m, x.x, r.x), fmaf(m, x.y, r.y), fmaf(m, x.z, r.z), fmaf(m, x.w, r.w));
+                if (blockIdx.x == 0) reinterpret_cast<float4*>(a.a_residual_out)[c] = x;
+            }
             *reinterpret_cast<float4*>(dg_row + at(c)) = x;
         }
     }
@@ -388,17 +407,18 @@ __global__ void __launch_bounds__(256, 4) dense_gemv_kernel(const uzu_dense_line
     uint32_t turn = 0;
     for (uint32_t g = blockIdx.x; g < groups; g += gridDim.x, turn ^= 1) {
         const uint32_t col = g * CPG + warp / KS;
-        float acc = 0.0f;
+        float acc = 0.0f, acc2 = 0.0f;
         for (uint32_t kb = k_first; ; kb += BATCH * STEP) {
             const bool last = kb - lane * VEC + BATCH * STEP >= k_hi;      // uniform over the warp
-            if (last) request(nxt, g + gridDim.x, k_first);
-            else request(nxt, g, kb + BATCH * STEP);
+            if (last) request(nxt, nxt2, g + gridDim.x, k_first);
+            else request(nxt, nxt2, g, kb + BATCH * STEP);
 #pragma unroll
             for (uint32_t u = 0; u < BATCH; ++u) {
                 const uint32_t k0 = kb + u * STEP;
                 if (k0 < k_hi) {
-                    float wf[VEC];
+                    float wf[VEC], wf2[PAIR ? VEC : 1];
                     unpack_weights<VEC, TW>(cur[u], wf);
+                    if constexpr (PAIR) unpack_weights<VEC, TW>(cur2[u], wf2);
 #pragma unroll
                     for (uint32_t i = 0; i < VEC; i += 4) {
                         const float4 x = *reinterpret_cast<const float4*>(dg_row + at((k0 + i) / 4));
@@ -406,24 +426,48 @@ __global__ void __launch_bounds__(256, 4) dense_gemv_kernel(const uzu_dense_line
                         acc = fmaf(x.y, wf[i + 1], acc);
                         acc = fmaf(x.z, wf[i + 2], acc);
                         acc = fmaf(x.w, wf[i + 3], acc);
+                        if constexpr (PAIR) {
+                            acc2 = fmaf(x.x, wf2[i], acc2);
+                            acc2 = fmaf(x.y, wf2[i + 1], acc2);
+                            acc2 = fmaf(x.z, wf2[i + 2], acc2);
+                            acc2 = fmaf(x.w, wf2[i + 3], acc2);
+                        }
                     }
                 }
             }
 #pragma unroll
-            for (uint32_t u = 0; u < BATCH; ++u) cur[u] = nxt[u];
+            for (uint32_t u = 0; u < BATCH; ++u) {
+                cur[u] = nxt[u];
+                if constexpr (PAIR) cur2[u] = nxt2[u];
+            }
             if (last) break;
         }
-        const float s = warp_sum(acc);
+        const float s = warp_sum(acc), s2 = PAIR ? warp_sum(acc2) : 0.0f;
+        auto store = [&](float t, float t2) {
+            if constexpr (PAIR) {
+                if (a.row_scale) { const float rs = *reinterpret_cast<const float*>(a.row_scale); t *= rs; t2 *= rs; }
+                reinterpret_cast<float*>(a.d)[col] = pair_value(a, 0, t, t2);
+            } else {
+                dense_store(a, reinterpret_cast<float*>(a.d) + col, 0, 0, col, t);
+            }
+        };
         if constexpr (KS == 1) {
-            if (lane == 0 && col < a.n) dense_store(a, reinterpret_cast<float*>(a.d) + col, 0, 0, col, s);
+            if (lane == 0 && col < a.n) store(s, s2);
         } else {
-            if (lane == 0) part[turn][warp] = s;         // (two buffers: the readers of one group are past it when the next but one writes)
+            if (lane == 0) {
+                part[turn][0][warp] = s;
+                if constexpr (PAIR) part[turn][1][warp] = s2;
+            }
+            // (two buffers: the readers of one group are past it when the next but one writes)
             __syncthreads();
             if (slice == 0 && lane == 0 && col < a.n) {
-                float t = 0.0f;
+                float t = 0.0f, t2 = 0.0f;
 #pragma unroll
-                for (int q = 0; q < KS; ++q) t += part[turn][warp + q];
-                dense_store(a, reinterpret_cast<float*>(a.d) + col, 0, 0, col, t);
+                for (int q = 0; q < KS; ++q) {
+                    t += part[turn][0][warp + q];
+                    if constexpr (PAIR) t2 += part[turn][1][warp + q];
+                }
+                store(t, t2);
             }
         }
     }
@@ -432,7 +476,7 @@ __global__ void __launch_bounds__(256, 4) dense_gemv_kernel(const uzu_dense_line
 // the shapes it takes (the caller's addresses included)
 static bool dense_gemv_applicable(const uzu_dense_linear_args& a) {
     const uint32_t vec = a.weights_dt == UZU_DT_BF16 ? 8 : 4;
-    return a.m == 1 && a.batch == 1 && !a.group_offsets && !a.rows_map && !a.pair_rows && !a.a_bf16 && a.k % vec == 0 && a.k > 0 && a.k <= DG_MAX_K &&
+    return a.m == 1 && a.batch == 1 && !a.group_offsets && !a.rows_map && !a.a_bf16 && a.k % vec == 0 && a.k > 0 && a.k <= DG_MAX_K &&
            (a.w & 15) == 0 && (a.a & 15) == 0 && (a.a_norm_weight & 15) == 0;
 }
 
@@ -739,6 +783,10 @@ __global__ void __launch_bounds__(256) dense_tensor128_kernel(const uzu_dense_li
             }
 }
 
+bool dense_takes_residual(const uzu_dense_linear_args& a) {
+    return dense_gemv_applicable(a) && !a.a_op && ((a.a_residual | a.a_residual_out) & 15) == 0;
+}
+
 // the one-row kernel always stages its row; the rows kernel stages its activation rows under exactly these conditions (its own test of them includes the device addresses)
 bool dense_rows_takes_norm(const uzu_dense_linear_args& a) {
     if (dense_gemv_applicable(a) && !a.a_op) return true;
@@ -757,7 +805,7 @@ extern "C" void uzu_dense_linear_encode(uzu_command_buffer* cmd, const uzu_dense
         cmd->record_error(UZU_ERROR_INVALID_ARGUMENT, "dense_linear: null operand / bad dtype / bad batch");
         return;
     }
-    if (a.a_op > 2 || a.glu_kind > 1 || (a.gate_bias && !a.gate) || (a.pair_rows && (a.gate || a.bias || a.accumulate || a.col_scale))) {
+    if (a.a_op > 2 || a.glu_kind > 2 || (a.gate_bias && !a.gate) || (a.pair_rows && (a.gate || a.bias || a.accumulate || a.col_scale))) {
         cmd->record_error(UZU_ERROR_INVALID_ARGUMENT, "dense_linear: unknown A operation, or a paired epilogue combined with gate / bias / accumulate");
         return;
     }
@@ -776,6 +824,10 @@ extern "C" void uzu_dense_linear_encode(uzu_command_buffer* cmd, const uzu_dense
     if (a.m == 0 || a.n == 0) return;
     if (a.a_norm_weight && !dense_rows_takes_norm(a)) {
         cmd->record_error(UZU_ERROR_UNSUPPORTED, "dense_linear: the layer-norm prologue takes one plain product of at most 8 rows that fit the staging buffer");
+        return;
+    }
+    if (a.a_residual && (!a.a_norm_weight || !a.a_residual_out || a.a_residual == a.a_residual_out || !dense_takes_residual(a))) {
+        cmd->record_error(UZU_ERROR_UNSUPPORTED, "dense_linear: the residual prologue takes a single row, one plain or paired product, a norm weight and a second residual row");
         return;
     }
     if (a.d_bf16 && (a.post_weight || a.token_table || !dense_umma_applicable(a))) {
@@ -812,16 +864,18 @@ extern "C" void uzu_dense_linear_encode(uzu_command_buffer* cmd, const uzu_dense
                 opt_in_dynamic_smem(cmd, kernel, (int)(DG_MAX_K * sizeof(float)), done);
                 launch(cmd, "dense_gemv_kernel", kernel, g, dim3(256), smem, a);
             };
-            static std::atomic<uint64_t> done[6];
-            if (bf16) {
-                if (ks == 1) gemv(dense_gemv_kernel<__nv_bfloat16, 1>, done[0]);
-                else if (ks == 2) gemv(dense_gemv_kernel<__nv_bfloat16, 2>, done[1]);
-                else gemv(dense_gemv_kernel<__nv_bfloat16, 4>, done[2]);
-            } else {
-                if (ks == 1) gemv(dense_gemv_kernel<float, 1>, done[3]);
-                else if (ks == 2) gemv(dense_gemv_kernel<float, 2>, done[4]);
-                else gemv(dense_gemv_kernel<float, 4>, done[5]);
-            }
+            static std::atomic<uint64_t> done[12];
+            auto by_slices = [&](auto tw, auto pair_c, int at) {
+                using TW = decltype(tw);
+                constexpr bool P = decltype(pair_c)::value;
+                if (ks == 1) gemv(dense_gemv_kernel<TW, 1, P>, done[at]);
+                else if (ks == 2) gemv(dense_gemv_kernel<TW, 2, P>, done[at + 1]);
+                else gemv(dense_gemv_kernel<TW, 4, P>, done[at + 2]);
+            };
+            if (bf16 && !a.pair_rows) by_slices(__nv_bfloat16{}, std::false_type{}, 0);
+            else if (bf16) by_slices(__nv_bfloat16{}, std::true_type{}, 3);
+            else if (!a.pair_rows) by_slices(float{}, std::false_type{}, 6);
+            else by_slices(float{}, std::true_type{}, 9);
             return;
         }
         dim3 grid((a.n * ks + 7) / 8, a.batch);

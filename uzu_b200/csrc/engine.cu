@@ -401,12 +401,20 @@ struct WindowAttentionLayer {   // softmax attention with a sliding window that 
     bool rot_halves = false;    // q / k pair channel i with i + rot.dims / 2 instead of (2i, 2i + 1)
     bool unit_rms = false;      // q and k are divided by their root mean square per head (no weight)
     uint32_t chunk = 0;         // > 0: only keys of the query's own chunk of positions are visible
+    Buf dist_slope;             // f32 [heads] (absent: none): what a score loses per position of distance
+    bool head_gate = false;     // head h's output is multiplied by the sigmoid of column gate_offset + h of the stacked projection
+    uint32_t gate_offset = 0;
     Buf sink;                   // f32 [heads] (absent: none): one more term exp(sink) in every softmax denominator
 };
 
-struct RetentionLayer {         // retention: per head S <- decay S + (k / sqrt(dim)) v^T, out = S^T q; per-head unit RMS, silu gate
+struct RetentionLayer {         // retention: per head S <- decay S + (key_scale k) v^T, out = S^T q; unit RMS per head with a silu gate, or (joint_norm) one
+                                // weighted RMS norm over all heads with a sigmoid gate
     DenseMatrix out;
     Buf decay;                  // f32 [heads]
+    Buf norm_weight;            // f32 [heads * vdim] (joint_norm)
+    bool joint_norm = false;
+    bool silu_inputs = false;   // q, k and v pass a silu first
+    float key_scale = 1.0f;
     uint32_t heads = 0, dim = 0, vdim = 0;
     uint32_t q_offset = 0, k_offset = 0, v_offset = 0, gate_offset = 0;
     float share = 1.0f;
@@ -436,7 +444,7 @@ struct SublayerGate {           // y * scale[c] * sigmoid(gate_logit[c] + bias[c
 
 struct GatedMlp {               // feed-forward: dense or routed experts; the unit is a clamped gated one, silu(g) * u, relu(u)^2 or the exact gelu(u) (no gate rows)
     enum Kind { None, Dense, TableExperts, RoutedExperts } kind = None;
-    enum Unit { ClampedGlu, SiluGlu, ReluSquared, GeluExact } unit = ClampedGlu;
+    enum Unit { ClampedGlu, SiluGlu, ReluSquared, GeluExact, GeluTanhGlu } unit = ClampedGlu;
     DenseMatrix gate_up /* experts x [2f, W]: gate rows then up rows; ReluSquared: [f (+ W gate logits), W]; GeluExact: [f, W] */, down /* experts x [W, f] */;
     DenseMatrix router;         // RoutedExperts: rows [router logits | sublayer gate]
     Buf table;                  // TableExperts: i32 [vocab, top]
@@ -445,6 +453,20 @@ struct GatedMlp {               // feed-forward: dense or routed experts; the un
     float limit = 0.0f;
     bool sigmoid_weights = false;   // RoutedExperts: a chosen expert's weight is the sigmoid of its own logit (default: softmax over the chosen)
     bool weight_on_input = false;   // RoutedExperts: the weight multiplies the expert's input, not its output
+    // RoutedExperts with a corrected choice: experts are chosen by sigmoid(logit) + correction among the best groups, weighted by their sigmoids over
+    // the chosen ones' sum, times weight_scale
+    bool corrected_choice = false;
+    Buf correction;             // f32 [experts]
+    uint32_t choice_groups = 1, choice_keep = 1;
+    float weight_scale = 1.0f;
+    // A feed-forward that every token uses besides (a shared expert), cut into `shared` slices of f units (the last one padded with zero rows: such a
+    // unit's result is 0): they lie behind the experts in gate_up and down, so short passes run them as experts of weight 1; long passes run them
+    // as two plain products, the second one on shared_down [W, shared * f].
+    uint32_t shared = 0;
+    bool shared_in_list = false;    // few enough slices for the pair lists
+    float shared_limit = 0.0f;
+    DenseMatrix shared_down;
+    uint32_t slots() const { return top + (shared_in_list ? shared : 0u); }
 };
 
 enum MixerKind : uint32_t { MixAttention = 0, MixDeltaNet = 1, MixGeneralDelta = 2, MixLatentAttention = 3, MixSigmoidAttention = 4,
@@ -464,6 +486,7 @@ struct Layer {
     WindowAttentionLayer wa;
     RetentionLayer rt;
     DenseMatrix side_in;        // MixWindowAttention / MixRetention / MixSideBySide: the stacked input projection of the layer's mixers
+    DenseMatrix side_out;       // MixSideBySide (optional): both output projections side by side along their inputs, one product for the sum
     Buf side_in_bias;           // f32 [side_in.rows] when any part has biases
     MlstmLayer ml;
     bool sequential = false;    // parallel-block engine: the feed-forward reads the residual AFTER the mixer's sum, through its own norm
@@ -472,6 +495,8 @@ struct Layer {
     bool sandwich = false;
     Norm post_mixer, post_mlp;
     float residual_mult = 1.0f;
+    // Output-normed form: only a sublayer's result is normed, the sublayers read the residual itself: x <- x + residual_mult * post(sublayer(x)).
+    bool output_normed = false;
     TokenSide side;
     // Streamed form of a sequential layer: the residual is several copies, every sublayer reads a weighted sum of them and its result is mixed
     // back into all of them (StreamWeights per sublayer).
@@ -566,6 +591,7 @@ struct uzu_engine {
     float norm_eps = 1e-5f;
     uint32_t streams = 0;       // > 0: the residual is this many copies of a row ([rows, streams, width]), mixed by every sublayer
     std::vector<uint32_t> runs; // the layer index of every layer run of a pass, in order; state[i] belongs to run i (a layer that runs twice has two)
+    Buf pb_position_turns;      // f64 [(width + 1) / 2]: turns per token of a sinusoidal position vector that is added to the embedding rows
     DenseMatrix pb_embed, pb_head, pb_side_embed;   // pb_side_embed: [vocab, layers * side dim], the table of the per-layer token inputs
     Buf pb_final_norm;
     Norm pb_out_norm;           // set when the output norm is not the grouped RMS norm (kind 1: Dynamic Tanh)
@@ -582,6 +608,14 @@ struct uzu_engine {
         uint64_t fused_read = 0;
         const Norm* input_norm = nullptr;
         bool normed_bf16 = false;
+        // Output-normed layers: the last sublayer's result waits in sub_out; whoever reads the residual next takes it in with its first launch
+        // (a decode step's first product does it itself, from the rows at resid_at into the other of resid / resid2).
+        Buf resid2;
+        uint64_t resid_at = 0;                           // where the residual's rows are (0: resid)
+        const Norm* pending = nullptr;                   // the norm of the waiting result
+        float pending_mult = 1.0f;
+        bool reads_residual = false;                     // the sublayer being encoded reads the residual itself
+        uint64_t residual() const { return resid_at ? resid_at : resid.ptr(); }
         Buf token_factors;                               // per (token, head) decay, gain, floor and normaliser product of a gated matrix memory
         Buf expand_f32, expand_keys, expand_values;      // a prompt pass's expanded latents: f32 [rows, heads * (dim + vdim)], then bf16 keys and values
         uint32_t expand_rows = 0;                        // rows the three hold
@@ -853,6 +887,7 @@ static void load_gamanex_model(uzu_engine* e, const Json& cfg, const std::string
 static void load_vugipel_model(uzu_engine* e, const Json& cfg, const std::string& dir);
 static void load_vakesun_model(uzu_engine* e, const Json& cfg, const std::string& dir);
 static void load_relidra_model(uzu_engine* e, const Json& cfg, const std::string& dir);
+static void load_bonolorn_model(uzu_engine* e, const Json& cfg, const std::string& dir);
 static void load_language_model_config(uzu_engine* e, const Json& cfg, const std::string& dir);
 
 // Model registry: config.json names its family, either by the reference's type tag or by an "architecture" string.
@@ -868,6 +903,7 @@ static const ModelFamily kModelFamilies[] = {
     {"Vugipel", [](const Json& c) { const Json* a = c.get("architecture"); return a && a->str == "Vugipel"; }, load_vugipel_model},
     {"Vakesun", [](const Json& c) { const Json* a = c.get("architecture"); return a && a->str == "Vakesun"; }, load_vakesun_model},
     {"Relidra", [](const Json& c) { const Json* a = c.get("architecture"); return a && a->str == "Relidra"; }, load_relidra_model},
+    {"Bonolorn", [](const Json& c) { const Json* a = c.get("architecture"); return a && a->str == "Bonolorn"; }, load_bonolorn_model},
 };
 
 static void load_model(uzu_engine* e, const std::string& dir) {

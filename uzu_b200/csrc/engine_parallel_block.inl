@@ -1,4 +1,4 @@
-// Parallel-block families (Punilix, Gamanex) and the sequential-sublayer families (Vugipel, Vakesun, Relidra) inside the host engine: configuration, weights, scratch and the encoding of one pass.
+// Parallel-block families (Punilix, Gamanex) and the sequential-sublayer families (Vugipel, Vakesun, Relidra, Bonolorn) inside the host engine: configuration, weights, scratch and the encoding of one pass.
 // Included by engine.cu; the pass driver, the state / cache manager, sampling, CUDA-graph decode and the sequence slots are the engine's own.
 //
 //   x = embed[token]                                                      (f32 residual stream)
@@ -6,6 +6,7 @@
 //   Gamanex layer:  h1 = rms(x) n1, h2 = rms(x) n2;  x <- x + ls1 sigmoid(G1 h1 + b1) mixer(h1) + ls2 sigmoid(G2 h2 + b2) mlp(h2)
 //   Vugipel layer:  x <- x + mixer(rms(x) (1 + n1));  x <- x + mlp(rms(x) (1 + n2))     (Layer::sequential)
 //   Vakesun layer:  x <- x + m post1(mixer(pre1(x)));  x <- x + m post2(mlp(pre2(x)));  x <- x + m rms(token input(x))    (Layer::sandwich)
+//   Bonolorn layer: x <- x + m post1(mixer(x));  x <- x + m post2(mlp(x))      (Layer::output_normed)
 //   Relidra layer:  u = sum_s in_s x_s;  x_t <- sum_s mix_st x_s + out_t sublayer(norm(u)), for the mixer and then the feed-forward (Layer::streamed)
 //   logits = cap * tanh(head . group_rms(x) / cap)   |   logit_scale * head . rms(x)
 //
@@ -518,6 +519,7 @@ static void load_vugipel_model(uzu_engine* e, const Json& cfg, const std::string
             R.dim = cfg_u32(rj, "dim");
             R.vdim = cfg_u32(rj, "vdim");
             R.share = (float)mc.at("right_scale").number();
+            R.key_scale = 1.0f / sqrtf((float)R.dim);
             if (R.heads == 0 || R.dim == 0 || R.dim > 1024 || R.vdim == 0) throw std::runtime_error(p + "mix.right: heads / vdim must be positive, dim in 1..1024");
             {
                 const auto& dj = rj.at("decay").arr;
@@ -1031,6 +1033,216 @@ static void load_relidra_model(uzu_engine* e, const Json& cfg, const std::string
     }
 }
 
+// Bonolorn: layers that read the residual itself and norm only their sublayers' results (layer norm, weight only, every addition times a fixed
+// factor); a sinusoidal position vector is added to the embedding. One kind of mixer: window attention without rotation (per-head q / k norms, a
+// distance slope per head, a sigmoid gate per head) and lightning attention (retention with silu inputs, one norm over all heads, a sigmoid
+// gate) side by side. Feed-forward: gelu_tanh(gate) * up; clamped experts behind a sigmoid router with corrected, group-limited choice and a
+// shared expert; or none. The readout shares the embedding table.
+// config.json: "width", "vocab", "norm": {"eps"}, "residual_mult", "layers": [{"type": "parallel", "mixer": {"left": {"heads", "kv_heads", "dim",
+// "vdim", "scale", "mask": {"size"}}, "left_scale", "right": {"heads", "dim", "vdim", "decay": [..]}, "right_scale"}, "mlp": null | {"kind": "dense",
+// "ff"} | {"kind": "moe", "expert": {"ff", "limit"}, "router": {"experts", "top", "groups": {"count", "keep"}, "scale"}, "shared": {"ff", "limit"}}}].
+// Tensors: embed, final.norm, l<i>.norm1 / norm2, l<i>.mix.left.{q,k,v,g,o,q.norm,k.norm}, l<i>.mix.right.{q,k,v,g,o,norm}, l<i>.mlp.{gate,up,down} |
+// l<i>.mlp.{router,correction,e<x>.{gate,up,down},shared.{gate,up,down}}.
+static void load_bonolorn_model(uzu_engine* e, const Json& cfg, const std::string& dir) {
+    if (e->opts.tp_size > 1) throw std::runtime_error("tensor parallelism is not built for the parallel-block families");
+    e->parallel_block = true;
+    e->store_dt = e->opts.storage_f32 ? UZU_DT_F32 : UZU_DT_BF16;
+    const uint32_t W = e->model_dim = cfg_u32(cfg, "width");
+    const uint32_t V = e->vocab = cfg_u32(cfg, "vocab");
+    if (W == 0 || V == 0) throw std::runtime_error("config: width and vocab must be positive");
+    e->norm_eps = (float)cfg.at("norm").at("eps").number();
+    e->norm_groups = 1;
+    const float mult = (float)cfg.at("residual_mult").number();
+    ParameterLoader pl(dir + "/model.safetensors");
+    auto layer_norm = [&](const std::string& name) {
+        Norm n;
+        n.present = true;
+        n.kind = 2;
+        n.n = W;
+        n.cfg.epsilon = e->norm_eps;
+        n.scales = upload_f32(e, read_floats(pl, name, {W}).v);
+        return n;
+    };
+    auto present = [](const Json& j, const char* key) -> const Json* {
+        const Json* v = j.get(key);
+        return v && !v->is_null() ? v : nullptr;
+    };
+    e->pb_embed = upload_matrix(e, read_floats(pl, "embed", {V, W}).v, V, W);
+    e->pb_head = e->pb_embed;        // the readout multiplies with the embedding table itself
+    e->pb_out_norm = layer_norm("final.norm");
+    {   // the position vectors' frequencies, in turns per token
+        std::vector<double> turns((W + 1) / 2);
+        for (size_t i = 0; i < turns.size(); ++i) turns[i] = std::pow(10000.0, -2.0 * (double)i / (double)W) / (2.0 * 3.14159265358979323846);
+        e->pb_position_turns = make_buf(e, std::max<size_t>(turns.size() * 8, 16), UZU_BUFFER_DEVICE);
+        cudaMemcpy((void*)e->pb_position_turns.ptr(), turns.data(), turns.size() * 8, cudaMemcpyHostToDevice);
+    }
+    uint64_t wbytes = e->pb_head.bytes, stb = 0, kvb = 0;
+    const auto& lcs = cfg.at("layers").arr;
+    e->layers.resize(lcs.size());
+    for (size_t i = 0; i < lcs.size(); ++i) {
+        const Json& lc = lcs[i];
+        Layer& L = e->layers[i];
+        const std::string p = "l" + std::to_string(i) + ".";
+        L.sequential = true;
+        L.output_normed = true;
+        L.residual_mult = mult;
+        L.post_mixer = layer_norm(p + "norm1");
+        const std::string type = lc.at("type").str;
+        if (type != "parallel") throw std::runtime_error("layer type '" + type + "' is not known to the Bonolorn family");
+        const Json& mc = lc.at("mixer");
+        L.kind = MixSideBySide;
+        L.is_attention = true;
+        WindowAttentionLayer& A = L.wa;
+        RetentionLayer& R = L.rt;
+        const Json& lj = mc.at("left");
+        const Json& rj = mc.at("right");
+        A.heads = cfg_u32(lj, "heads");
+        A.kv_heads = cfg_u32(lj, "kv_heads");
+        A.dim = cfg_u32(lj, "dim");
+        A.vdim = cfg_u32(lj, "vdim");
+        A.scale = (float)lj.at("scale").number();
+        A.share = (float)mc.at("left_scale").number();
+        A.head_gate = true;
+        if (A.heads == 0 || A.kv_heads == 0 || A.heads % A.kv_heads || A.dim == 0 || A.vdim == 0 || A.dim > 512 || A.vdim > 512)
+            throw std::runtime_error(p + "mix.left: kv_heads must divide heads, head sizes must be in 1..512");
+        if (const Json* mk = present(lj, "mask")) {
+            A.window = cfg_u32(*mk, "size");
+            if (A.window == 0) throw std::runtime_error(p + "mix.left: mask.size must be positive");
+        }
+        {
+            std::vector<float> slope;
+            for (uint32_t h = 0; h < A.heads; ++h) slope.push_back((float)std::pow(2.0, -8.0 * (double)(h + 1) / (double)A.heads));
+            A.dist_slope = upload_f32(e, slope);
+        }
+        R.heads = cfg_u32(rj, "heads");
+        R.dim = cfg_u32(rj, "dim");
+        R.vdim = cfg_u32(rj, "vdim");
+        R.share = (float)mc.at("right_scale").number();
+        R.silu_inputs = true;
+        R.joint_norm = true;
+        if (R.heads == 0 || R.dim == 0 || R.dim > 1024 || R.vdim == 0) throw std::runtime_error(p + "mix.right: heads / vdim must be positive, dim in 1..1024");
+        {
+            const auto& dj = rj.at("decay").arr;
+            if (dj.size() != R.heads) throw std::runtime_error(p + "mix.right: one decay per head is expected");
+            std::vector<float> d;
+            for (const Json& x : dj) d.push_back((float)x.number());
+            R.decay = upload_f32(e, d);
+        }
+        const uint32_t lq = A.heads * A.dim, lk = A.kv_heads * A.dim, lv = A.kv_heads * A.vdim, lo = A.heads * A.vdim, rq = R.heads * R.dim, rv = R.heads * R.vdim;
+        const std::string l = p + "mix.left.", r = p + "mix.right.";
+        std::vector<float> in;
+        append(in, read_floats(pl, l + "q", {lq, W}));
+        append(in, read_floats(pl, l + "k", {lk, W}));
+        append(in, read_floats(pl, l + "v", {lv, W}));
+        append(in, read_floats(pl, r + "q", {rq, W}));
+        append(in, read_floats(pl, r + "k", {rq, W}));
+        append(in, read_floats(pl, r + "v", {rv, W}));
+        append(in, read_floats(pl, r + "g", {rv, W}));
+        append(in, read_floats(pl, l + "g", {A.heads, W}));
+        A.q_offset = 0; A.k_offset = lq; A.v_offset = lq + lk;
+        R.q_offset = lq + lk + lv; R.k_offset = R.q_offset + rq; R.v_offset = R.k_offset + rq; R.gate_offset = R.v_offset + rv;
+        A.gate_offset = R.gate_offset + rv;
+        const uint32_t rows = (A.gate_offset + A.heads + 7) & ~7u;      // rows of whole 16-byte pieces in either storage type (zero rows behind the gate)
+        in.resize((size_t)rows * W, 0.0f);
+        L.side_in = upload_matrix(e, in, rows, W);
+        A.q_norm = upload_f32(e, read_floats(pl, l + "q.norm", {A.dim}).v);
+        A.k_norm = upload_f32(e, read_floats(pl, l + "k.norm", {A.dim}).v);
+        R.norm_weight = upload_f32(e, read_floats(pl, r + "norm", {rv}).v);
+        {   // one product for both outputs; the shares multiply its inputs (a share of zero empties its columns: a factor of 0 means 1 to the kernels)
+            HostTensor a = read_floats(pl, l + "o", {W, lo}), b = read_floats(pl, r + "o", {W, rv});
+            for (auto [t, share] : {std::pair<HostTensor*, float*>{&a, &A.share}, {&b, &R.share}})
+                if (*share == 0.0f) { std::fill(t->v.begin(), t->v.end(), 0.0f); *share = 1.0f; }
+            std::vector<float> out((size_t)W * (lo + rv));
+            for (uint32_t c = 0; c < W; ++c) {
+                std::copy_n(a.v.begin() + (size_t)c * lo, lo, out.begin() + (size_t)c * (lo + rv));
+                std::copy_n(b.v.begin() + (size_t)c * rv, rv, out.begin() + (size_t)c * (lo + rv) + lo);
+            }
+            L.side_out = upload_matrix(e, out, W, lo + rv);
+        }
+        wbytes += L.side_in.bytes + L.side_out.bytes;
+        // key / value rows a decode step reads: the window's, or the whole context
+        if (A.window) stb += (uint64_t)A.window * (lk + lv) * storage_size(e->store_dt);
+        else kvb += (uint64_t)(lk + lv) * storage_size(e->store_dt);
+        stb += 2ull * R.heads * R.dim * R.vdim * 4;
+        GatedMlp& M = L.gmlp;
+        const Json* ml = present(lc, "mlp");
+        if (!ml) {
+            if (pl.tensors.count(p + "norm2")) read_floats(pl, p + "norm2", {W});       // a norm without a sublayer: checked, not used
+            continue;
+        }
+        L.post_mlp = layer_norm(p + "norm2");
+        const std::string kind = ml->at("kind").str;
+        if (kind == "dense") {
+            M.kind = GatedMlp::Dense;
+            M.unit = GatedMlp::GeluTanhGlu;
+            M.f = cfg_u32(*ml, "ff");
+            if (M.f == 0) throw std::runtime_error(p + "mlp: ff must be positive");
+            std::vector<float> gu;
+            append(gu, read_floats(pl, p + "mlp.gate", {M.f, W}));
+            append(gu, read_floats(pl, p + "mlp.up", {M.f, W}));
+            M.gate_up = upload_matrix(e, gu, 2 * M.f, W);
+            M.down = upload_matrix(e, read_floats(pl, p + "mlp.down", {W, M.f}).v, W, M.f);
+            wbytes += M.gate_up.bytes + M.down.bytes;
+            continue;
+        }
+        if (kind != "moe") throw std::runtime_error("mlp kind '" + kind + "' is not known to the Bonolorn family");
+        M.kind = GatedMlp::RoutedExperts;
+        M.unit = GatedMlp::ClampedGlu;
+        M.corrected_choice = true;
+        const Json& ro = ml->at("router");
+        M.f = cfg_u32(ml->at("expert"), "ff");
+        M.limit = (float)ml->at("expert").at("limit").number();
+        M.experts = cfg_u32(ro, "experts");
+        M.top = cfg_u32(ro, "top");
+        M.weight_scale = (float)ro.at("scale").number();
+        if (const Json* gr = present(ro, "groups")) { M.choice_groups = cfg_u32(*gr, "count"); M.choice_keep = cfg_u32(*gr, "keep"); }
+        const Json* sh = present(*ml, "shared");
+        const uint32_t sf = sh ? cfg_u32(*sh, "ff") : 0u;
+        if (sh) M.shared_limit = (float)sh->at("limit").number();
+        if (M.f == 0 || M.experts == 0 || M.top == 0 || M.top > M.experts || M.experts > 8192 || M.top > 64) throw std::runtime_error(p + "mlp: bad expert / top counts");
+        if (M.choice_groups == 0 || M.choice_groups > 256 || M.experts % M.choice_groups || M.choice_keep == 0 || M.choice_keep > M.choice_groups ||
+            M.top > M.experts / M.choice_groups * M.choice_keep)
+            throw std::runtime_error(p + "mlp: router.groups.count must divide the experts (at most 256), and the kept groups must hold router.top of them");
+        M.shared = (sf + M.f - 1) / M.f;
+        M.shared_in_list = M.shared > 0 && M.shared <= 8;
+        M.router = upload_matrix(e, read_floats(pl, p + "mlp.router", {M.experts, W}).v, M.experts, W);
+        M.correction = upload_f32(e, read_floats(pl, p + "mlp.correction", {M.experts}).v);
+        std::vector<float> gu, dn;
+        for (uint32_t x = 0; x < M.experts; ++x) {
+            const std::string q = p + "mlp.e" + std::to_string(x) + ".";
+            append(gu, read_floats(pl, q + "gate", {M.f, W}));
+            append(gu, read_floats(pl, q + "up", {M.f, W}));
+            append(dn, read_floats(pl, q + "down", {W, M.f}));
+        }
+        if (sf) {
+            HostTensor g = read_floats(pl, p + "mlp.shared.gate", {sf, W}), u = read_floats(pl, p + "mlp.shared.up", {sf, W}), d = read_floats(pl, p + "mlp.shared.down", {W, sf});
+            const uint32_t padded = M.shared * M.f;
+            g.v.resize((size_t)padded * W, 0.0f);
+            u.v.resize((size_t)padded * W, 0.0f);
+            std::vector<float> wide((size_t)W * padded, 0.0f);
+            for (uint32_t c = 0; c < W; ++c) std::copy_n(d.v.begin() + (size_t)c * sf, sf, wide.begin() + (size_t)c * padded);
+            const size_t block = (size_t)M.f * W;
+            for (uint32_t s = 0; s < M.shared; ++s) {
+                gu.insert(gu.end(), g.v.begin() + s * block, g.v.begin() + (s + 1) * block);
+                gu.insert(gu.end(), u.v.begin() + s * block, u.v.begin() + (s + 1) * block);
+                for (uint32_t c = 0; c < W; ++c) dn.insert(dn.end(), wide.begin() + (size_t)c * padded + s * M.f, wide.begin() + (size_t)c * padded + (s + 1) * M.f);
+            }
+            M.shared_down = upload_matrix(e, wide, W, padded);
+        }
+        M.gate_up = upload_matrix(e, gu, 2 * M.f, W, M.experts + M.shared);
+        M.down = upload_matrix(e, dn, W, M.f, M.experts + M.shared);
+        wbytes += M.router.bytes + (M.gate_up.bytes + M.down.bytes) / (M.experts + M.shared) * (M.top + M.shared);
+    }
+    pl.assert_all_validated();
+    e->info.model_dim = W;
+    e->info.hidden_dim = 0;
+    e->info.vocab_size = V;
+    e->info.num_layers = e->info.num_attention_layers = e->info.num_delta_net_layers = (uint32_t)e->layers.size();
+    e->info.weight_bytes_per_token = wbytes;
+    e->info.kv_bytes_per_token_per_ctx = kvb;
+    e->info.state_bytes_per_token = stb;
+}
+
 constexpr uint32_t kPromptChunks = 8;  // most key chunks of a row tile of a sigmoid-attention prompt pass
 constexpr uint32_t kSplitRows = 256;   // query rows x key splits of one latent-attention launch that leaves partial softmax states
 
@@ -1039,11 +1251,12 @@ static void create_parallel_block_scratch(uzu_engine* e) {
     if (!e->parallel_block) return;
     const uint32_t W = e->model_dim;
     uint32_t proj = 1, lat = 1, wide = 1, query = 1, mixed = 1, gated = 1, gu = 1, act = 1, top = 1, experts = 1, partial = 1, kmax = e->model_dim;
-    uint32_t proj2 = 1, tickets = 1, prompt_partial = 0, factor_heads = 0, expand_cols = 0, expand_rows = 0;
-    bool second_norm = false, sandwich = false;
+    uint32_t proj2 = 1, tickets = 1, prompt_partial = 0, factor_heads = 0, expand_cols = 0, expand_rows = 0, shared_act = 0;
+    bool second_norm = false, sandwich = false, output_normed = false;
     for (const Layer& L : e->layers) {
         second_norm = second_norm || L.pre_mlp.present;
         sandwich = sandwich || L.sandwich;
+        output_normed = output_normed || L.output_normed;
         if (L.side.present) { lat = std::max(lat, L.side.dim); kmax = std::max(kmax, L.side.dim); }
         if (L.kind == MixSigmoidAttention) {
             const SigmoidAttentionLayer& A = L.sa;
@@ -1089,6 +1302,10 @@ static void create_parallel_block_scratch(uzu_engine* e) {
                 gated = std::max(gated, L.rt.heads * L.rt.vdim);
                 kmax = std::max(kmax, L.rt.heads * L.rt.vdim);
             }
+            if (L.side_out.w.b) {          // both outputs lie side by side
+                mixed = std::max(mixed, L.side_out.cols);
+                kmax = std::max(kmax, L.side_out.cols);
+            }
         } else if (L.kind == MixGeneralDelta) {
             const uint32_t HD = L.gd.heads * L.gd.dim;
             proj = std::max(proj, L.gd.in.rows);
@@ -1118,8 +1335,10 @@ static void create_parallel_block_scratch(uzu_engine* e) {
             gu = std::max(gu, 2 * L.gmlp.f);
             act = std::max(act, L.gmlp.f);
             kmax = std::max(kmax, L.gmlp.f);
-            top = std::max(top, L.gmlp.top);
-            experts = std::max(experts, L.gmlp.experts);
+            top = std::max(top, L.gmlp.slots());
+            experts = std::max(experts, L.gmlp.experts + L.gmlp.shared);
+            shared_act = std::max(shared_act, L.gmlp.shared * L.gmlp.f);
+            kmax = std::max(kmax, L.gmlp.shared * L.gmlp.f);
         }
     }
     auto dev = [&](size_t bytes) { return make_buf(e, std::max<size_t>(bytes, 256), UZU_BUFFER_DEVICE); };
@@ -1129,7 +1348,8 @@ static void create_parallel_block_scratch(uzu_engine* e) {
     if (e->streams) P.stream_u = dev(R * W * 4);
     P.normed = dev(R * W * 4);
     if (second_norm) P.normed2 = dev(R * W * 4);
-    if (sandwich || e->streams) P.sub_out = dev(R * W * 4);
+    if (output_normed) P.resid2 = dev((size_t)W * 4);       // (one row: only the decode step's products move the residual)
+    if (sandwich || output_normed || e->streams) P.sub_out = dev(R * W * 4);
     if (factor_heads) P.token_factors = dev(4 * R * factor_heads * 4);
     if (expand_cols) {
         P.expand_rows = std::min(expand_rows, 16384u);      // longer ranges take the kernel that reads the latents directly
@@ -1152,8 +1372,8 @@ static void create_parallel_block_scratch(uzu_engine* e) {
     P.attn_partial = dev(std::max((size_t)kSplitRows * partial, (size_t)prompt_partial * kPromptChunks * R) * 4);
     P.mixed = dev(R * mixed * 4);
     P.gated_mix = dev(R * std::max(gated, mixed) * 4);
-    P.gate_up = dev(R * top * gu * 4);
-    P.act = dev(R * top * act * 4);
+    P.gate_up = dev(R * std::max(top * gu, 2 * shared_act) * 4);
+    P.act = dev(R * std::max(top * act, shared_act) * 4);
     P.pair_out = dev(R * top * W * 4);
     P.group_offsets = dev((size_t)(experts + 1) * 4);
     P.rows_map = dev(R * top * 4);
@@ -1201,11 +1421,62 @@ static void set_norm(uzu_norm_add_args& a, const Norm& n, bool next) {
     else { a.kind = n.kind; a.weight = n.scales.ptr(); a.bias = n.bias.ptr(); a.alpha = n.alpha; }
 }
 
+// Output-normed layers: takes the waiting result into `rows` rows of the residual from row `begin` on, optionally norming them for a reader.
+static void take_pending(uzu_engine* e, uzu_command_buffer* cmd, uint32_t begin, uint32_t rows, const Norm* next, uint64_t output) {
+    auto& P = e->pb;
+    const uint32_t W = e->model_dim;
+    uzu_norm_add_args a{};
+    a.input = P.sub_out.ptr() + (uint64_t)begin * W * 4; a.residual = P.residual() + (uint64_t)begin * W * 4;
+    a.rows = rows; a.n = W; a.in_stride = W; a.epsilon = e->norm_eps; a.mult = P.pending_mult;
+    set_norm(a, *P.pending, false);
+    a.output = output;
+    if (next) set_norm(a, *next, true);
+    else if (output) a.residual_bf16 = 1;
+    uzu_norm_add_encode(cmd, &a);
+    P.pending = nullptr;
+}
+
+// A product of an output-normed layer that reads the residual. If a result still waits to be taken in: a single row's product does it as it
+// stages its row; otherwise a launch does, which in long passes also leaves bf16 rows for the tcgen05 products of the sublayer.
+static void residual_input(uzu_engine* e, uzu_command_buffer* cmd, uzu_dense_linear_args& x) {
+    auto& P = e->pb;
+    const uint32_t W = e->model_dim;
+    x.lda = W;
+    if (P.pending) {
+        uzu_dense_linear_args fused = x;
+        fused.a = P.sub_out.ptr();
+        fused.a_residual = P.residual();
+        fused.a_residual_out = P.residual() == P.resid.ptr() ? P.resid2.ptr() : P.resid.ptr();
+        if (x.m == 1 && dense_takes_residual(fused)) {
+            fused.a_norm_weight = P.pending->scales.ptr(); fused.a_norm_epsilon = e->norm_eps; fused.a_residual_mult = P.pending_mult;
+            x = fused;
+            P.resid_at = fused.a_residual_out;
+            P.pending = nullptr;
+            return;
+        }
+        uzu_dense_linear_args any = x;         // a plain product of this sublayer (the first one may be too narrow for tcgen05)
+        any.a = P.normed.ptr(); any.n = std::max(64u, x.n); any.ldd = any.n; any.batch = 1; any.group_offsets = 0; any.rows_map = 0; any.pair_rows = 0;
+        any.d = P.proj.ptr(); any.d_op = 0;
+        P.normed_bf16 = dense_umma_applicable(any);
+        take_pending(e, cmd, 0, x.m, nullptr, P.normed_bf16 ? P.normed.ptr() : 0);
+    }
+    x.a = P.residual();
+    if (P.normed_bf16) {
+        uzu_dense_linear_args narrow = x;
+        narrow.a = P.normed.ptr();
+        if (dense_umma_applicable(narrow)) { x.a = P.normed.ptr(); x.a_bf16 = 1; }
+    }
+}
+
 // A sublayer's first product: its A rows are the normed input. A streamed layer's short pass norms them inside the product where that can be
 // done (and in a launch of its own otherwise); its long pass may have left them as bf16.
 static void sublayer_input(uzu_engine* e, uzu_command_buffer* cmd, uzu_dense_linear_args& x) {
     auto& P = e->pb;
     const uint32_t W = e->model_dim;
+    if (P.reads_residual) {
+        residual_input(e, cmd, x);
+        return;
+    }
     x.a = P.normed.ptr(); x.lda = W;
     if (P.normed_bf16) { x.a_bf16 = 1; return; }
     if (!P.input_norm) return;
@@ -1327,6 +1598,9 @@ static void encode_side_by_side(uzu_engine* e, uzu_command_buffer* cmd, const La
         aa.head_temp = A.head_temp.ptr(); aa.v_cosines = vcos; aa.v_sines = vsin; aa.v_pairs = v_pairs;
         aa.rows = m; aa.heads = A.heads; aa.kv_heads = A.kv_heads; aa.dim = A.dim; aa.vdim = A.vdim; aa.prefix = S.length; aa.cache_dt = e->store_dt;
         aa.window = A.window; aa.keep_first = A.keep_first; aa.chunk = A.chunk; aa.scale = A.scale; aa.softcap = A.softcap; aa.sinks = A.sink.ptr();
+        aa.dist_slope = A.dist_slope.ptr();
+        if (A.head_gate) { aa.head_gate = P.proj.ptr() + (uint64_t)A.gate_offset * 4; aa.head_gate_stride = ld; }
+        if (L.side_out.w.b) { aa.out_stride = L.side_out.cols; aa.out_scale = A.share; }
         {   // few query rows: cut the visible keys (in tiles of 16) so that about eight small CTAs per SM run (the captured step sizes the
             // cut for the largest context its graph serves; a window bounds it)
             uint32_t bound = pc.dynamic ? attention_bucket(S.length + m) : S.length + m;
@@ -1339,11 +1613,13 @@ static void encode_side_by_side(uzu_engine* e, uzu_command_buffer* cmd, const La
             if (aa.splits < 2 || m > kSplitRows) aa.splits = 1;
         }
         uzu_window_attention_encode(cmd, &aa);
-        uzu_dense_linear_args x = dense_args(e, A.out, P.mixed.ptr(), m, P.redirect ? P.sub_out.ptr() : P.resid.ptr());
-        x.lda = A.heads * A.vdim; x.accumulate = P.redirect ? 0 : 1; x.scale = A.share;
-        if (A.out_bias.b) x.bias = A.out_bias.ptr();
-        sublayer_epilogue(e, x);
-        uzu_dense_linear_encode(cmd, &x);
+        if (!L.side_out.w.b) {
+            uzu_dense_linear_args x = dense_args(e, A.out, P.mixed.ptr(), m, P.redirect ? P.sub_out.ptr() : P.resid.ptr());
+            x.lda = A.heads * A.vdim; x.accumulate = P.redirect ? 0 : 1; x.scale = A.share;
+            if (A.out_bias.b) x.bias = A.out_bias.ptr();
+            sublayer_epilogue(e, x);
+            uzu_dense_linear_encode(cmd, &x);
+        }
     }
     if (L.has_retention()) {
         const RetentionLayer& R = L.rt;
@@ -1352,13 +1628,19 @@ static void encode_side_by_side(uzu_engine* e, uzu_command_buffer* cmd, const La
         ra.q = P.proj.ptr() + (uint64_t)R.q_offset * 4; ra.k = P.proj.ptr() + (uint64_t)R.k_offset * 4; ra.v = P.proj.ptr() + (uint64_t)R.v_offset * 4;
         ra.decay = R.decay.ptr(); ra.state = S.ssm_state.ptr(); ra.out = P.wide.ptr();
         ra.rows = m; ra.heads = R.heads; ra.dim = R.dim; ra.vdim = R.vdim; ra.q_stride = ra.k_stride = ra.v_stride = ld; ra.out_stride = rv;
-        ra.key_scale = 1.0f / sqrtf((float)R.dim);
+        ra.key_scale = R.key_scale; ra.input_op = R.silu_inputs ? 1 : 0;
         uzu_retention_encode(cmd, &ra);
         uzu_head_norm_gate_args na{};
         na.x = P.wide.ptr(); na.gate = P.proj.ptr() + (uint64_t)R.gate_offset * 4; na.out = P.gated_mix.ptr();
         na.rows = m; na.heads = R.heads; na.dim = R.vdim; na.x_stride = rv; na.gate_stride = ld; na.out_stride = rv; na.normalize = 1;
         na.epsilon = e->norm_eps; na.gate_op = 1;
+        if (R.joint_norm) { na.heads = 1; na.dim = rv; na.scales = R.norm_weight.ptr(); na.gate_op = 0; }
+        if (L.side_out.w.b) { na.out = P.mixed.ptr() + (uint64_t)L.wa.heads * L.wa.vdim * 4; na.out_stride = L.side_out.cols; na.out_scale = R.share; }
         uzu_head_norm_gate_encode(cmd, &na);
+        if (L.side_out.w.b) {
+            encode_into_residual(e, cmd, L.side_out, P.mixed.ptr(), L.side_out.cols, m);
+            return;
+        }
         uzu_dense_linear_args x = dense_args(e, R.out, P.gated_mix.ptr(), m, P.redirect ? P.sub_out.ptr() : P.resid.ptr());
         x.lda = rv; x.accumulate = (P.redirect && !L.has_window_attention()) ? 0 : 1; x.scale = R.share;       // the second of two mixers adds to the first
         if (!L.has_window_attention()) sublayer_epilogue(e, x);
@@ -1565,16 +1847,23 @@ static void encode_gated_mlp(uzu_engine* e, uzu_command_buffer* cmd, const Layer
     const uint32_t m = pc.m, W = e->model_dim;
     constexpr float kGateSlope = 1.702f;
     const bool paired = m <= 8;
+    const uint32_t unit_kind = M.unit == GatedMlp::SiluGlu ? 1 : M.unit == GatedMlp::GeluTanhGlu ? 2 : 0;
+    // a shared expert: slices of it among the experts of the pair lists, or (long passes) two plain products
+    const bool shared_listed = M.shared_in_list && m < 128;
+    const uint32_t slots = M.top + (shared_listed ? M.shared : 0u), lists = M.experts + (shared_listed ? M.shared : 0u);
     auto gate_up_args = [&]() {
         uzu_dense_linear_args up = dense_args(e, M.gate_up, h, m, paired ? P.act.ptr() : P.gate_up.ptr());
         up.lda = W;
+        if (M.kind == GatedMlp::Dense && P.reads_residual) residual_input(e, cmd, up);
         if (M.weight_on_input) up.row_scale = P.pair_weight_compact.ptr();      // expert(w h): the first product is linear in its input
-        if (paired) { up.n = M.f; up.ldd = M.f; up.pair_rows = M.f; up.glu_limit = M.limit; up.glu_alpha = kGateSlope; up.glu_kind = M.unit == GatedMlp::SiluGlu ? 1 : 0; }
+        if (paired) { up.n = M.f; up.ldd = M.f; up.pair_rows = M.f; up.glu_limit = M.limit; up.glu_alpha = kGateSlope; up.glu_kind = unit_kind; }
         return up;
     };
     auto unit = [&](uint32_t rows) {
-        if (M.unit == GatedMlp::SiluGlu) uzu_silu_glu_encode(cmd, P.gate_up.ptr(), P.act.ptr(), rows, M.f);
-        else uzu_clamped_glu_encode(cmd, P.gate_up.ptr(), P.act.ptr(), rows, M.f, M.limit, kGateSlope);
+        uzu_glu_args ga{};
+        ga.gate_up = P.gate_up.ptr(); ga.output = P.act.ptr(); ga.rows = rows; ga.f = M.f; ga.kind = unit_kind; ga.limit = M.limit; ga.alpha = kGateSlope;
+        if (shared_listed) { ga.group_offsets = P.group_offsets.ptr(); ga.last_group = M.experts; ga.limit_last = M.shared_limit; }
+        uzu_glu_encode(cmd, &ga);
     };
     if (M.kind == GatedMlp::Dense && M.unit == GatedMlp::ReluSquared) {
         const uint32_t ld = M.gate_up.rows;                                       // [up | gate logits]
@@ -1602,18 +1891,38 @@ static void encode_gated_mlp(uzu_engine* e, uzu_command_buffer* cmd, const Layer
     if (M.kind == GatedMlp::Dense) {
         uzu_dense_linear_args up = gate_up_args();
         uzu_dense_linear_encode(cmd, &up);
-        if (!paired) unit(m);
+        if (!paired) {
+            // long passes keep the unit's rows in bf16, as the down projection's A rows
+            uzu_dense_linear_args dn = dense_args(e, M.down, P.act.ptr(), m, P.sub_out.ptr());
+            uzu_glu_args ga{};
+            ga.gate_up = P.gate_up.ptr(); ga.output = P.act.ptr(); ga.rows = m; ga.f = M.f; ga.kind = unit_kind; ga.limit = M.limit; ga.alpha = kGateSlope;
+            ga.output_bf16 = dn.a_bf16 = P.redirect && dense_umma_applicable(dn) ? 1 : 0;
+            uzu_glu_encode(cmd, &ga);
+            if (dn.a_bf16) {
+                uzu_dense_linear_encode(cmd, &dn);
+                return;
+            }
+        }
         encode_into_residual(e, cmd, M.down, P.act.ptr(), M.f, m);
         return;
     }
     // routed experts: expert-sorted (token, slot) pairs, grouped products over the pairs, weighted combine per token
     if (M.kind == GatedMlp::RoutedExperts) {
-        encode_dense(e, cmd, M.router, h, W, m, P.proj2.ptr());                   // [router logits | gate logits]
+        {
+            uzu_dense_linear_args x = dense_args(e, M.router, h, m, P.proj2.ptr());              // [router logits | gate logits]
+            x.lda = W;
+            if (P.reads_residual) { residual_input(e, cmd, x); h = P.residual(); }
+            uzu_dense_linear_encode(cmd, &x);
+        }
         uzu_topk_route_args ra{};
         ra.logits = P.proj2.ptr(); ra.bias = M.router_bias.ptr(); ra.group_offsets = P.group_offsets.ptr(); ra.rows_map = P.rows_map.ptr();
         ra.pair_pos = P.pair_pos.ptr(); ra.pair_weight = P.pair_weight.ptr(); ra.rows = m; ra.top = M.top; ra.experts = M.experts;
         ra.logits_stride = M.router.rows;
-        ra.weight_kind = M.sigmoid_weights ? 1 : 0;
+        ra.weight_kind = M.corrected_choice ? 2 : M.sigmoid_weights ? 1 : 0;
+        if (M.corrected_choice) {
+            ra.correction = M.correction.ptr(); ra.choice_groups = M.choice_groups; ra.choice_keep = M.choice_keep; ra.weight_scale = M.weight_scale;
+            ra.always = slots - M.top;
+        }
         ra.scratch = P.route_scratch.ptr();
         if (M.weight_on_input) ra.compact_weight = P.pair_weight_compact.ptr();
         if (!M.router_bias.b) ra.bias = 0;
@@ -1625,26 +1934,44 @@ static void encode_gated_mlp(uzu_engine* e, uzu_command_buffer* cmd, const Layer
         uzu_table_route_encode(cmd, &ra);
     }
     // a single expert takes every row in row order: its two products are plain ones (no row groups), so long passes run them on tcgen05
-    const bool grouped = M.experts > 1;
+    const bool grouped = lists > 1;
     uzu_dense_linear_args up = gate_up_args();
     if (grouped) {
-        up.batch = M.experts; up.w_z_stride = M.gate_up.stride();
+        up.batch = lists; up.w_z_stride = M.gate_up.stride();
         up.group_offsets = P.group_offsets.ptr(); up.rows_map = P.rows_map.ptr();
+        if (shared_listed) { up.glu_last_group = M.experts; up.glu_limit_last = M.shared_limit; }
     }
     uzu_dense_linear_encode(cmd, &up);
-    if (!paired) unit(m * M.top);
+    if (!paired) unit(m * slots);
     // ... and, when its weight already sits on its input and no sublayer gate follows, its down projection adds straight into the residual
     const bool direct = !grouped && M.weight_on_input && !L.mlp_gate.present;
     uzu_dense_linear_args dn = dense_args(e, M.down, P.act.ptr(), m, direct ? P.resid.ptr() : P.pair_out.ptr());
     dn.lda = M.f; dn.accumulate = direct ? 1 : 0;
     if (grouped) {
-        dn.batch = M.experts; dn.w_z_stride = M.down.stride();
+        dn.batch = lists; dn.w_z_stride = M.down.stride();
         dn.group_offsets = P.group_offsets.ptr();
     }
     uzu_dense_linear_encode(cmd, &dn);
     if (direct) return;
+    // the shared expert as plain products: its slices' [gate | up] rows lie back to back, so the unit sees m * slices rows of one slice each
+    const bool shared_plain = M.shared > 0 && !shared_listed;
+    if (shared_plain) {
+        uzu_dense_linear_args sx = dense_args(e, M.gate_up, h, m, P.gate_up.ptr());
+        sx.w = M.gate_up.w.ptr() + (uint64_t)M.experts * M.gate_up.stride() * storage_size(e->store_dt);
+        sx.n = M.shared * 2 * M.f; sx.ldd = sx.n; sx.lda = W;
+        if (P.reads_residual) residual_input(e, cmd, sx);
+        uzu_dense_linear_encode(cmd, &sx);
+        uzu_dense_linear_args sd = dense_args(e, M.shared_down, P.act.ptr(), m, P.redirect ? P.sub_out.ptr() : P.resid.ptr());
+        sd.accumulate = P.redirect ? 0 : 1;
+        uzu_glu_args ga{};
+        ga.gate_up = P.gate_up.ptr(); ga.output = P.act.ptr(); ga.rows = m * M.shared; ga.f = M.f; ga.kind = unit_kind; ga.limit = M.shared_limit; ga.alpha = kGateSlope;
+        ga.output_bf16 = sd.a_bf16 = dense_umma_applicable(sd) ? 1 : 0;
+        uzu_glu_encode(cmd, &ga);
+        uzu_dense_linear_encode(cmd, &sd);
+    }
     uzu_routed_combine_args ca{};
-    ca.pairs = P.pair_out.ptr(); ca.pair_pos = P.pair_pos.ptr(); ca.output = P.resid.ptr(); ca.rows = m; ca.top = M.top; ca.n = W; ca.accumulate = 1;
+    ca.pairs = P.pair_out.ptr(); ca.pair_pos = P.pair_pos.ptr(); ca.output = P.redirect ? P.sub_out.ptr() : P.resid.ptr(); ca.rows = m; ca.top = slots; ca.n = W;
+    ca.accumulate = P.redirect && !shared_plain ? 0 : 1;
     if (M.kind == GatedMlp::RoutedExperts) { ca.pair_weight = M.weight_on_input ? 0 : P.pair_weight.ptr(); ca.weight = 1.0f; }
     else ca.weight = 1.0f / (float)M.top;
     if (L.mlp_gate.present) {
@@ -1721,6 +2048,20 @@ static void encode_sandwich_layer(uzu_engine* e, uzu_command_buffer* cmd, const 
         rms.kind = 0; rms.scales = T.norm;
         add(rms, next);
     }
+}
+
+// An output-normed layer: the sublayers read the residual and leave their results in P.sub_out, where they wait for the next reader.
+static void encode_output_normed_layer(uzu_engine* e, uzu_command_buffer* cmd, const Layer& L, LayerState& S, const PassCtx& pc) {
+    auto& P = e->pb;
+    auto sublayer = [&](const Norm& post, auto&& encode) {
+        P.redirect = P.reads_residual = true;
+        encode();
+        P.redirect = P.reads_residual = P.normed_bf16 = false;
+        P.pending = &post;
+        P.pending_mult = L.residual_mult;
+    };
+    sublayer(L.post_mixer, [&] { encode_mixer(e, cmd, L, S, pc); });
+    if (L.gmlp.kind != GatedMlp::None) sublayer(L.post_mlp, [&] { encode_gated_mlp(e, cmd, L, pc, P.residual()); });
 }
 
 // A pass over streamed layers. Between two sublayers the residual's copies take the first one's result and the second one's input is formed:
@@ -1806,11 +2147,27 @@ static void encode_parallel_block_decoder(uzu_engine* e, uzu_command_buffer* cmd
         encode_parallel_block_readout(e, cmd, row_begin, row_end);
         return;
     }
-    uzu_embedding_f32_scaled_encode(cmd, e->token_ids.ptr(), e->pb_embed.w.ptr(), e->store_dt, P.resid.ptr(), m, e->vocab, W, e->input_scale);
+    {
+        uzu_embedding_f32_args ea{};
+        ea.token_ids = e->token_ids.ptr(); ea.table = e->pb_embed.w.ptr(); ea.output = P.resid.ptr();
+        ea.position_turns = e->pb_position_turns.ptr(); ea.dynamic_position = pc.dynamic ? e->decode_state.ptr() : 0; ea.prefix = e->context_length;
+        ea.rows = m; ea.vocab = e->vocab; ea.n = W; ea.weights_dt = e->store_dt; ea.scale = e->input_scale;
+        uzu_embedding_f32_position_encode(cmd, &ea);
+    }
+    P.resid_at = 0;
+    P.pending = nullptr;
     bool normed_ready = false;
     for (size_t i = 0; i < e->layers.size(); ++i) {
         Layer& L = e->layers[i];
         LayerState& S = e->state[i];
+        if (L.output_normed) {
+            encode_output_normed_layer(e, cmd, L, S, pc);
+            if (dump) {
+                take_pending(e, cmd, 0, m, nullptr, 0);
+                uzu_command_buffer_encode_copy(cmd, P.residual(), P.layer_dump.ptr() + (uint64_t)i * MAX_ROWS * W * 4, (size_t)m * W * 4);
+            }
+            continue;
+        }
         if (L.sandwich) {
             const Norm* next = (i + 1 < e->layers.size() && e->layers[i + 1].sandwich) ? &e->layers[i + 1].pre_mixer : nullptr;
             encode_sandwich_layer(e, cmd, L, S, pc, next, normed_ready);
@@ -1834,6 +2191,7 @@ static void encode_parallel_block_decoder(uzu_engine* e, uzu_command_buffer* cmd
         if (dump) uzu_command_buffer_encode_copy(cmd, P.resid.ptr(), P.layer_dump.ptr() + (uint64_t)i * MAX_ROWS * W * 4, (size_t)m * W * 4);
     }
     if (dump) P.dump_rows = m;
+    if (P.pending && row_end <= row_begin) take_pending(e, cmd, 0, m, nullptr, 0);      // rows may be read out by launches of their own later
     encode_parallel_block_readout(e, cmd, row_begin, row_end);
 }
 
@@ -1841,13 +2199,15 @@ static void encode_parallel_block_readout(uzu_engine* e, uzu_command_buffer* cmd
     if (row_end <= row_begin) return;
     const uint32_t rows = row_end - row_begin, W = e->model_dim;
     auto& P = e->pb;
-    const uint64_t rows_in = (e->streams ? P.stream_u : P.resid).ptr() + (uint64_t)row_begin * W * 4;
+    const uint64_t rows_in = (e->streams ? P.stream_u.ptr() : P.residual()) + (uint64_t)row_begin * W * 4;
     uzu_dense_linear_args x = dense_args(e, e->pb_head, P.normed_rows.ptr(), rows, P.logits_f32.ptr());
     x.lda = W;
     if (e->has_logit_scale) x.scale = e->logit_scale;
     uzu_dense_linear_args direct = x;
     direct.a = rows_in;
-    if (e->pb_out_norm.present && e->pb_out_norm.kind == 2 && dense_rows_takes_norm(direct)) {      // few rows: normed inside the readout product
+    if (P.pending) {                // only the rows that are read out take the last sublayer's result in
+        take_pending(e, cmd, row_begin, rows, &e->pb_out_norm, P.normed_rows.ptr());
+    } else if (e->pb_out_norm.present && e->pb_out_norm.kind == 2 && dense_rows_takes_norm(direct)) {      // few rows: normed inside the readout product
         x.a = rows_in; x.a_norm_weight = e->pb_out_norm.scales.ptr(); x.a_norm_epsilon = e->norm_eps;
     } else if (e->pb_out_norm.present) {
         uzu_norm_add_args a{};

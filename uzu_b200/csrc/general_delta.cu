@@ -159,11 +159,14 @@ __global__ void __launch_bounds__(128) general_delta_prepare_kernel(const uzu_ge
 }
 
 // one warp per (row, head)
-__global__ void __launch_bounds__(128) head_norm_gate_kernel(const uzu_head_norm_gate_args a) {
+// WIDE: a CTA per (row, head) instead of a warp: long heads (a norm over all heads at once)
+template <bool WIDE>
+__global__ void __launch_bounds__(WIDE ? 512 : 128) head_norm_gate_kernel(const uzu_head_norm_gate_args a) {
     pdl_launch_dependents();
     pdl_wait();
-    const int lane = threadIdx.x & 31;
-    const uint32_t unit = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    __shared__ float red[32];
+    const uint32_t lane = WIDE ? threadIdx.x : threadIdx.x & 31, step = WIDE ? blockDim.x : 32u;
+    const uint32_t unit = WIDE ? blockIdx.x : blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
     if (unit >= a.rows * a.heads) return;
     const uint32_t row = unit / a.heads, h = unit % a.heads;
     const float* x = reinterpret_cast<const float*>(a.x) + (size_t)row * a.x_stride + (size_t)h * a.dim;
@@ -178,15 +181,16 @@ __global__ void __launch_bounds__(128) head_norm_gate_kernel(const uzu_head_norm
     }
     if (a.normalize) {
         float ss = 0.0f;
-        for (uint32_t i = lane; i < a.dim; i += 32) { const float y = x[i] * pre; ss = fmaf(y, y, ss); }
-        ss = warp_sum(ss);
+        for (uint32_t i = lane; i < a.dim; i += step) { const float y = x[i] * pre; ss = fmaf(y, y, ss); }
+        ss = WIDE ? block_sum(ss, red) : warp_sum(ss);
         inv = 1.0f / sqrtf(ss / (float)a.dim + a.epsilon);
     }
-    for (uint32_t i = lane; i < a.dim; i += 32) {
+    const float out_scale = a.out_scale != 0.0f ? a.out_scale : 1.0f;
+    for (uint32_t i = lane; i < a.dim; i += step) {
         float v = x[i] * pre * inv;
         if (sc) v *= sc[i];
         if (gate) v *= a.gate_op == 1 ? gate[i] / (1.0f + expf(-gate[i])) : 1.0f / (1.0f + expf(-gate[i]));
-        out[i] = v;
+        out[i] = v * out_scale;
     }
 }
 
@@ -242,7 +246,10 @@ void uzu_head_norm_gate_encode(uzu_command_buffer* cmd, const uzu_head_norm_gate
     if (!b.gate_stride) b.gate_stride = b.heads * b.dim;
     if (!b.out_stride) b.out_stride = b.heads * b.dim;
     const uint32_t units = b.rows * b.heads;
-    launch(cmd, "head_norm_gate_kernel", head_norm_gate_kernel, dim3((units + 3) / 4), dim3(128), 0, b);
+    if (b.dim > 512)
+        launch(cmd, "head_norm_gate_kernel", head_norm_gate_kernel<true>, dim3(units), dim3(b.dim > 2048 ? 512 : 256), 0, b);
+    else
+        launch(cmd, "head_norm_gate_kernel", head_norm_gate_kernel<false>, dim3((units + 3) / 4), dim3(128), 0, b);
 }
 
 }  // extern "C"

@@ -25,6 +25,7 @@ namespace uzu {
 namespace {
 
 __device__ __forceinline__ float lr_sigmoid(float x) { return 1.0f / (1.0f + expf(-x)); }
+__device__ __forceinline__ float lr_input(uint32_t op, float x) { return op == 1 ? x * lr_sigmoid(x) : x; }
 
 struct GruStep { float a, b; };     // S <- a S + b
 
@@ -170,8 +171,8 @@ __global__ void __launch_bounds__(PART == 32 ? 1024 : 512) retention_kernel(cons
             pre_q[u] = pre_k[u] = 0.0f;
             if (i < nb * dim) {
                 const uint32_t r = i / dim, ch = i - r * dim;
-                pre_q[u] = pq[(size_t)(tb + r) * a.q_stride + ch] * qscale;
-                pre_k[u] = pk[(size_t)(tb + r) * a.k_stride + ch] * a.key_scale;
+                pre_q[u] = pq[(size_t)(tb + r) * a.q_stride + ch];
+                pre_k[u] = pk[(size_t)(tb + r) * a.k_stride + ch];
             }
         }
 #pragma unroll
@@ -194,12 +195,12 @@ __global__ void __launch_bounds__(PART == 32 ? 1024 : 512) retention_kernel(cons
 #pragma unroll
         for (int u = 0; u < STAGE; ++u) {
             const uint32_t i = tid + (uint32_t)u * blockDim.x;
-            if (i < RT_BATCH * dim) { qs[i] = pre_q[u]; ks[i] = pre_k[u]; }
+            if (i < RT_BATCH * dim) { qs[i] = lr_input(a.input_op, pre_q[u]) * qscale; ks[i] = lr_input(a.input_op, pre_k[u]) * a.key_scale; }
         }
 #pragma unroll
         for (int u = 0; u < 4; ++u) {
             const uint32_t i = tid + (uint32_t)u * blockDim.x;
-            if (i < RT_BATCH * 32) vs[i] = pre_v[u];
+            if (i < RT_BATCH * 32) vs[i] = lr_input(a.input_op, pre_v[u]);
         }
         if constexpr (GATED) { if (tid < RT_BATCH) ds[tid] = pre_d; }
         __syncthreads();
@@ -284,7 +285,7 @@ void uzu_retention_encode(uzu_command_buffer* cmd, const uzu_retention_args* a) 
     if (!encodable(cmd, "retention")) return;
     const bool gated = a->token_decay != 0;
     if (!a->q || !a->k || !a->v || (!gated && !a->decay) || (gated && !a->token_gain) || (!gated && a->norm_out) || !a->state || !a->out || a->dim == 0 ||
-        a->dim > 1024 || a->vdim == 0 || a->heads == 0) {
+        a->dim > 1024 || a->vdim == 0 || a->heads == 0 || a->input_op > 1 || (gated && a->input_op)) {
         cmd->record_error(UZU_ERROR_INVALID_ARGUMENT, "retention: null operand, per-token factors without their pair, or key size outside 1..1024");
         return;
     }

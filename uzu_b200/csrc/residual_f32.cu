@@ -118,6 +118,7 @@ __global__ void __launch_bounds__(256) norm_add_kernel(const uzu_norm_add_args a
         inv = 1.0f / sqrtf(ss / (float)a.n + a.epsilon);
     }
     // first norm, and the residual add
+    __nv_bfloat16* copy = a.residual_bf16 ? reinterpret_cast<__nv_bfloat16*>(a.output) + (size_t)row * a.n : nullptr;
     float s2 = 0.0f, ss2 = 0.0f;
 #pragma unroll
     for (int j = 0; j < KEEP; ++j) {
@@ -130,16 +131,18 @@ __global__ void __launch_bounds__(256) norm_add_kernel(const uzu_norm_add_args a
             s2 += v;
             if (res) res[i] = v;
             else out[i] = v;
+            if (copy) copy[i] = __float2bfloat16_rn(v);
         }
     }
     for (uint32_t i = threadIdx.x + KEEP * blockDim.x; i < a.n; i += blockDim.x) {
         float v = norm_add_value(a.kind, in[i], mean, inv, a.alpha, w, b, i);
         if (res) { v = fmaf(a.mult, v, res[i]); res[i] = v; }          // read back below by the thread that wrote it
         else out[i] = v;
+        if (copy) copy[i] = __float2bfloat16_rn(v);
         ss2 = fmaf(v, v, ss2);
         s2 += v;
     }
-    if (!res || !out) return;
+    if (!res || !out || copy) return;
     float inv2 = 1.0f, mean2 = 0.0f;
     if (a.next_kind == 2) {         // the deviations need the mean: a second sum over the row
         mean2 = block_sum(s2, red) / (float)a.n;
@@ -378,20 +381,75 @@ __global__ void token_gate_kernel(const uzu_token_gate_args a) {
     reinterpret_cast<float*>(a.out)[idx] = g * e;
 }
 
+// a thread per channel pair (2i, 2i + 1): the two share the angle of a sinusoidal position vector
 template <typename TW>
-__global__ void embedding_f32_kernel(const uint32_t* tokens, const TW* table, float* out, uint32_t vocab, uint32_t n, float scale) {
+__global__ void embedding_f32_kernel(const uzu_embedding_f32_args a) {
     pdl_launch_dependents();
     pdl_wait();
-    const uint32_t row = blockIdx.y;
-    const uint32_t tok = tokens[row];
-    const uint32_t i = blockIdx.x * blockDim.x + threadIdx.x;
-    if (i >= n) return;
-    float v = 0.0f;
-    if (tok < vocab) {
-        if constexpr (sizeof(TW) == 2) v = __bfloat162float(table[(size_t)tok * n + i]);
-        else v = table[(size_t)tok * n + i];
+    const uint32_t row = blockIdx.y, i = blockIdx.x * blockDim.x + threadIdx.x, c0 = 2 * i, n = a.n;
+    const uint32_t tok = reinterpret_cast<const uint32_t*>(a.token_ids)[row];
+    if (c0 >= n) return;
+    const bool two = c0 + 1 < n;
+    float v[2] = {0.0f, 0.0f};
+    if (tok < a.vocab) {
+        const TW* t = reinterpret_cast<const TW*>(a.table) + (size_t)tok * n + c0;
+        if constexpr (sizeof(TW) == 2) { v[0] = __bfloat162float(t[0]); if (two) v[1] = __bfloat162float(t[1]); }
+        else { v[0] = t[0]; if (two) v[1] = t[1]; }
     }
-    out[(size_t)row * n + i] = v * scale;
+    v[0] *= a.scale; v[1] *= a.scale;
+    if (a.position_turns) {
+        const uint32_t p = (a.dynamic_position ? *reinterpret_cast<const uint32_t*>(a.dynamic_position) : a.prefix) + row;
+        const double turns = (double)p * reinterpret_cast<const double*>(a.position_turns)[i];
+        float s, c;
+        sincospif(2.0f * (float)(turns - rint(turns)), &s, &c);
+        v[0] += s; v[1] += c;
+    }
+    float* out = reinterpret_cast<float*>(a.output) + (size_t)row * n + c0;
+    out[0] = v[0];
+    if (two) out[1] = v[1];
+    if (a.rows_bf16) {
+        __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(a.rows_bf16) + (size_t)row * n + c0;
+        o[0] = __float2bfloat16_rn(v[0]);
+        if (two) o[1] = __float2bfloat16_rn(v[1]);
+    }
+}
+
+__device__ __forceinline__ float glu_value(uint32_t kind, float g, float u, float limit, float alpha) {
+    if (kind == 0) {
+        g = fminf(g, limit);
+        u = fminf(fmaxf(u, -limit), limit) + 1.0f;
+        return g * (1.0f / (1.0f + expf(-alpha * g))) * u;
+    }
+    if (kind == 1) return g * (1.0f / (1.0f + expf(-g))) * u;
+    return 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
+}
+
+// VEC elements of one row per thread (f a multiple of VEC, 16-byte aligned operands when VEC = 4)
+template <int VEC>
+__global__ void __launch_bounds__(256) glu_kernel(const uzu_glu_args a) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const size_t idx = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * VEC;
+    if (idx >= (size_t)a.rows * a.f) return;
+    const uint32_t r = (uint32_t)(idx / a.f), c = (uint32_t)(idx % a.f);
+    const float* src = reinterpret_cast<const float*>(a.gate_up) + (size_t)r * 2 * a.f + c;
+    const float limit = (a.group_offsets && r >= reinterpret_cast<const uint32_t*>(a.group_offsets)[a.last_group]) ? a.limit_last : a.limit;
+    float v[VEC];
+    if constexpr (VEC == 4) {
+        const float4 g = *reinterpret_cast<const float4*>(src), u = *reinterpret_cast<const float4*>(src + a.f);
+        v[0] = glu_value(a.kind, g.x, u.x, limit, a.alpha); v[1] = glu_value(a.kind, g.y, u.y, limit, a.alpha);
+        v[2] = glu_value(a.kind, g.z, u.z, limit, a.alpha); v[3] = glu_value(a.kind, g.w, u.w, limit, a.alpha);
+        if (a.output_bf16) {
+            const __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
+            *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(a.output) + idx) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+        } else {
+            *reinterpret_cast<float4*>(reinterpret_cast<float*>(a.output) + idx) = make_float4(v[0], v[1], v[2], v[3]);
+        }
+    } else {
+        v[0] = glu_value(a.kind, src[0], src[a.f], limit, a.alpha);
+        if (a.output_bf16) reinterpret_cast<__nv_bfloat16*>(a.output)[idx] = __float2bfloat16_rn(v[0]);
+        else reinterpret_cast<float*>(a.output)[idx] = v[0];
+    }
 }
 
 __global__ void rows_to_bf16_kernel(const float* src, uint32_t src_stride, __nv_bfloat16* dst, uint32_t rows, uint32_t n) {
@@ -401,27 +459,6 @@ __global__ void rows_to_bf16_kernel(const float* src, uint32_t src_stride, __nv_
     if (idx >= (size_t)rows * n) return;
     const size_t r = idx / n, c = idx % n;
     dst[idx] = __float2bfloat16_rn(src[r * src_stride + c]);
-}
-
-__global__ void clamped_glu_kernel(const float* gate_up, float* out, uint32_t rows, uint32_t f, float limit, float alpha) {
-    pdl_launch_dependents();
-    pdl_wait();
-    const size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
-    if (idx >= (size_t)rows * f) return;
-    const size_t r = idx / f, c = idx % f;
-    const float g = fminf(gate_up[r * 2 * f + c], limit);
-    const float u = fminf(fmaxf(gate_up[r * 2 * f + f + c], -limit), limit);
-    out[idx] = g * (1.0f / (1.0f + expf(-alpha * g))) * (u + 1.0f);
-}
-
-__global__ void silu_glu_kernel(const float* gate_up, float* out, uint32_t rows, uint32_t f) {
-    pdl_launch_dependents();
-    pdl_wait();
-    const size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
-    if (idx >= (size_t)rows * f) return;
-    const size_t r = idx / f, c = idx % f;
-    const float g = gate_up[r * 2 * f + c], u = gate_up[r * 2 * f + f + c];
-    out[idx] = g * (1.0f / (1.0f + expf(-g))) * u;
 }
 
 __global__ void unary_f32_kernel(const float* in, uint32_t in_stride, float* out, uint32_t out_stride, uint32_t rows, uint32_t n, uint32_t op) {
@@ -560,16 +597,20 @@ __global__ void __launch_bounds__(1024) table_route_kernel(const uzu_table_route
 
 // One CTA, a warp per row: `top` rounds, each picking the best (logit, lower index first) that comes after the previous pick in that
 // order, so no list of the picked experts is kept. Weights: exp(z - z_first) over the sum of the picked ones, or (weight_kind 1) the
-// sigmoid of every picked logit on its own. compact_weight gets the same weights in the expert-sorted order of the pair list.
+// sigmoid of every picked logit on its own, or (weight_kind 2) the sigmoids of the picked ones over their sum, picked by sigmoid + correction
+// among the experts of the best groups. compact_weight gets the same weights in the expert-sorted order of the pair list.
 // MODE 0: choice and pair lists in one CTA (short passes). Long passes with a scratch: MODE 1 makes the choice over many CTAs (a warp per
 // row, the picked experts go to the scratch), MODE 2 is the one CTA that sorts them into the pair lists.
+constexpr int ROUTE_GROUPS = 8;      // words of 32 groups
+constexpr size_t ROUTE_SMEM = 192 * 1024;   // the experts' counters and the pairs of a pass
+
 template <int MODE>
-__global__ void __launch_bounds__(1024) topk_route_kernel(const uzu_topk_route_args a) {
+__global__ void __launch_bounds__(MODE == 1 ? 256 : 1024) topk_route_kernel(const uzu_topk_route_args a) {
     pdl_launch_dependents();
     pdl_wait();
     extern __shared__ uint32_t counts[];   // [experts + 1]
-    const uint32_t pairs = a.rows * a.top;
-    uint16_t* pe_shared = reinterpret_cast<uint16_t*>(counts + a.experts + 1);
+    const uint32_t slots = a.top + a.always, experts = a.experts + a.always, pairs = a.rows * slots;      // with the experts that every row uses
+    uint16_t* pe_shared = reinterpret_cast<uint16_t*>(counts + experts + 1);
     uint16_t* pe = MODE == 1 ? reinterpret_cast<uint16_t*>(a.scratch) : pe_shared;
     const float* bias = reinterpret_cast<const float*>(a.bias);
     float* weight = reinterpret_cast<float*>(a.pair_weight);
@@ -582,19 +623,76 @@ __global__ void __launch_bounds__(1024) topk_route_kernel(const uzu_topk_route_a
     auto first_logit = [&](uint32_t r) {
         return (r < a.rows && lane < a.experts) ? reinterpret_cast<const float*>(a.logits)[(size_t)r * a.logits_stride + lane] + (bias ? bias[lane] : 0.0f) : 0.0f;
     };
+    const bool corrected = a.weight_kind == 2;
+    const float* correction = reinterpret_cast<const float*>(a.correction);
+    const uint32_t groups = corrected && a.choice_groups > 1 ? a.choice_groups : 1u, group_size = a.experts / groups;
+    const float own_correction = corrected && correction && lane < a.experts ? correction[lane] : 0.0f;
+    // what the choice goes by: the logit, or its sigmoid plus the expert's correction
+    auto score_of = [&](float z, uint32_t e) {
+        return corrected ? 1.0f / (1.0f + expf(-z)) + (e == lane ? own_correction : correction ? correction[e] : 0.0f) : z;
+    };
     float next_z = first_logit(warp);
     for (uint32_t r = warp; r < a.rows; r += warps) {
         const float* z = reinterpret_cast<const float*>(a.logits) + (size_t)r * a.logits_stride;
-        const float own_z = next_z;
+        const float own_z = score_of(next_z, lane);
         next_z = first_logit(r + warps);
+        // lane g % 32 holds group g's score and whether its experts can be chosen (at most 32 * GROUPS groups)
+        float group_score[ROUTE_GROUPS];
+        uint32_t open_groups = 0xFFFFFFFFu;                  // bit g / 32 of lane g % 32
+        if (groups > 1) {
+#pragma unroll
+            for (int q = 0; q < ROUTE_GROUPS; ++q) group_score[q] = -INFINITY;
+            for (uint32_t g = 0; g < groups; ++g) {          // the two largest choice scores of the group, over the warp
+                float hi = -INFINITY, lo = -INFINITY;
+                for (uint32_t e0 = g * group_size; e0 < (g + 1) * group_size; e0 += 32) {
+                    // lane l looks at the expert of this batch that it also owns in the rounds below (e % 32 == l), so own_z serves batch 0
+                    const uint32_t base = e0 & ~31u, e = base + lane + (base + lane < e0 ? 32u : 0u);
+                    if (e < (g + 1) * group_size && e < e0 + 32) {
+                        const float v = e == lane ? own_z : score_of(z[e] + (bias ? bias[e] : 0.0f), e);
+                        if (v > hi) { lo = hi; hi = v; }
+                        else if (v > lo) lo = v;
+                    }
+                }
+#pragma unroll
+                for (int o = 16; o > 0; o >>= 1) {
+                    const float oh = __shfl_xor_sync(0xffffffffu, hi, o), ol = __shfl_xor_sync(0xffffffffu, lo, o);
+                    lo = fmaxf(fminf(hi, oh), fmaxf(lo, ol));
+                    hi = fmaxf(hi, oh);
+                }
+                if (group_size == 1) lo = 0.0f;
+#pragma unroll
+                for (int q = 0; q < ROUTE_GROUPS; ++q)
+                    if (g == 32u * q + lane) group_score[q] = hi + lo;
+            }
+            open_groups = 0;
+            for (uint32_t k = 0; k < a.choice_keep; ++k) {   // the best group that is not open yet, the lower index first
+                float best = -INFINITY;
+                uint32_t at = 0xFFFFFFFFu;
+#pragma unroll
+                for (int q = 0; q < ROUTE_GROUPS; ++q) {
+                    const uint32_t g = 32u * q + lane;
+                    if (g < groups && !(open_groups >> q & 1u) && (at == 0xFFFFFFFFu || group_score[q] > best)) { best = group_score[q]; at = g; }
+                }
+#pragma unroll
+                for (int o = 16; o > 0; o >>= 1) {
+                    const float ov = __shfl_xor_sync(0xffffffffu, best, o);
+                    const uint32_t oi = __shfl_xor_sync(0xffffffffu, at, o);
+                    if (oi != 0xFFFFFFFFu && (at == 0xFFFFFFFFu || ov > best || (ov == best && oi < at))) { best = ov; at = oi; }
+                }
+                if (at != 0xFFFFFFFFu && (at & 31u) == lane) open_groups |= 1u << (at >> 5);
+            }
+        }
         float prev_v = INFINITY, first = 0.0f, sum = 0.0f;
         uint32_t prev_i = 0;
         bool any = false;
         for (uint32_t s = 0; s < a.top; ++s) {
             float best_v = -INFINITY;
             uint32_t best_i = 0xFFFFFFFFu;
-            for (uint32_t e = lane; e < a.experts; e += 32) {
-                const float v = e == lane ? own_z : z[e] + (bias ? bias[e] : 0.0f);
+            for (uint32_t e0 = 0; e0 < a.experts; e0 += 32) {
+                const uint32_t e = e0 + lane, g = groups > 1 ? min(e, a.experts - 1) / group_size : 0u;
+                const uint32_t open = __shfl_sync(0xffffffffu, open_groups, g & 31u);
+                if (e >= a.experts || !(open >> (g >> 5) & 1u)) continue;
+                const float v = e == lane ? own_z : score_of(z[e] + (bias ? bias[e] : 0.0f), e);
                 const bool after = !any || v < prev_v || (v == prev_v && e > prev_i);
                 if (after && (best_i == 0xFFFFFFFFu || v > best_v)) { best_v = v; best_i = e; }    // ascending e: the first of equals stays
             }
@@ -608,22 +706,30 @@ __global__ void __launch_bounds__(1024) topk_route_kernel(const uzu_topk_route_a
             if (!any) first = best_v;
             any = true;
             prev_v = best_v; prev_i = best_i;
-            const float w = a.weight_kind == 1 ? 1.0f / (1.0f + expf(-best_v)) : expf(best_v - first);
+            const float w = corrected ? 1.0f / (1.0f + expf(-(z[best_i] + (bias ? bias[best_i] : 0.0f))))
+                                      : a.weight_kind == 1 ? 1.0f / (1.0f + expf(-best_v)) : expf(best_v - first);
             sum += w;
             if (lane == 0) {
-                pe[r * a.top + s] = (uint16_t)best_i;
-                weight[r * a.top + s] = w;
+                pe[r * slots + s] = (uint16_t)best_i;
+                weight[r * slots + s] = w;
             }
         }
         __syncwarp();
-        if (lane < a.top && a.weight_kind == 0) {
-            for (uint32_t s = lane; s < a.top; s += 32) weight[r * a.top + s] /= sum;
+        if (lane < a.top && a.weight_kind != 1) {
+            for (uint32_t s = lane; s < a.top; s += 32) {
+                const float w = weight[r * slots + s];
+                weight[r * slots + s] = corrected ? w / (sum + 1e-20f) * a.weight_scale : w / sum;
+            }
+        }
+        for (uint32_t s = lane; s < a.always; s += 32) {
+            pe[r * slots + a.top + s] = (uint16_t)(a.experts + s);
+            weight[r * slots + a.top + s] = 1.0f;
         }
     }
     }
     if constexpr (MODE == 1) return;
     __syncthreads();
-    route_sort_pairs(pe_shared, counts, pairs, a.top, a.experts, reinterpret_cast<uint32_t*>(a.group_offsets), reinterpret_cast<uint32_t*>(a.rows_map),
+    route_sort_pairs(pe_shared, counts, pairs, slots, experts, reinterpret_cast<uint32_t*>(a.group_offsets), reinterpret_cast<uint32_t*>(a.rows_map),
                      reinterpret_cast<uint32_t*>(a.pair_pos));
     if (a.compact_weight) {
         __syncthreads();
@@ -680,12 +786,32 @@ void uzu_group_rms_norm_encode(uzu_command_buffer* cmd, const uzu_group_rms_norm
 
 void uzu_embedding_f32_scaled_encode(uzu_command_buffer* cmd, uint64_t token_ids, uint64_t table, uint32_t weights_dt, uint64_t output, uint32_t rows,
                                      uint32_t vocab, uint32_t n, float scale) {
-    if (!encodable(cmd, "embedding_f32") || rows == 0 || n == 0) return;
-    dim3 grid(blocks256(n), rows);
-    if (weights_dt == UZU_DT_BF16)
-        launch(cmd, "embedding_f32_kernel", embedding_f32_kernel<__nv_bfloat16>, grid, dim3(256), 0, (const uint32_t*)token_ids, (const __nv_bfloat16*)table, (float*)output, vocab, n, scale);
-    else
-        launch(cmd, "embedding_f32_kernel", embedding_f32_kernel<float>, grid, dim3(256), 0, (const uint32_t*)token_ids, (const float*)table, (float*)output, vocab, n, scale);
+    uzu_embedding_f32_args a{};
+    a.token_ids = token_ids; a.table = table; a.output = output; a.rows = rows; a.vocab = vocab; a.n = n; a.weights_dt = weights_dt; a.scale = scale;
+    uzu_embedding_f32_position_encode(cmd, &a);
+}
+
+void uzu_embedding_f32_position_encode(uzu_command_buffer* cmd, const uzu_embedding_f32_args* a) {
+    if (!encodable(cmd, "embedding_f32") || a->rows == 0 || a->n == 0) return;
+    if (!a->token_ids || !a->table || !a->output || (a->weights_dt != UZU_DT_BF16 && a->weights_dt != UZU_DT_F32)) {
+        cmd->record_error(UZU_ERROR_INVALID_ARGUMENT, "embedding_f32: null operand or bad table type");
+        return;
+    }
+    const dim3 grid(blocks256((a->n + 1) / 2), a->rows);
+    if (a->weights_dt == UZU_DT_BF16) launch(cmd, "embedding_f32_kernel", embedding_f32_kernel<__nv_bfloat16>, grid, dim3(256), 0, *a);
+    else launch(cmd, "embedding_f32_kernel", embedding_f32_kernel<float>, grid, dim3(256), 0, *a);
+}
+
+void uzu_glu_encode(uzu_command_buffer* cmd, const uzu_glu_args* a) {
+    if (!encodable(cmd, "glu")) return;
+    if (!a->gate_up || !a->output || a->kind > 2) {
+        cmd->record_error(UZU_ERROR_INVALID_ARGUMENT, "glu: null operand or unknown unit");
+        return;
+    }
+    if (a->rows == 0 || a->f == 0) return;
+    const size_t n = (size_t)a->rows * a->f;
+    if (a->f % 4 == 0 && (a->gate_up & 15) == 0 && (a->output & 15) == 0) launch(cmd, "glu_kernel", glu_kernel<4>, dim3(blocks256(n / 4)), dim3(256), 0, *a);
+    else launch(cmd, "glu_kernel", glu_kernel<1>, dim3(blocks256(n)), dim3(256), 0, *a);
 }
 
 void uzu_embedding_f32_encode(uzu_command_buffer* cmd, uint64_t token_ids, uint64_t table, uint32_t weights_dt, uint64_t output, uint32_t rows,
@@ -695,14 +821,14 @@ void uzu_embedding_f32_encode(uzu_command_buffer* cmd, uint64_t token_ids, uint6
 
 void uzu_norm_add_encode(uzu_command_buffer* cmd, const uzu_norm_add_args* a) {
     if (!encodable(cmd, "norm_add")) return;
-    if (!a->input || (!a->residual && !a->output) || a->kind > 2 || a->next_kind > 2) {
+    if (!a->input || (!a->residual && !a->output) || a->kind > 2 || a->next_kind > 2 || (a->residual_bf16 && (!a->residual || !a->output))) {
         cmd->record_error(UZU_ERROR_INVALID_ARGUMENT, "norm_add: null operand or unknown norm kind");
         return;
     }
     if (a->rows == 0 || a->n == 0) return;
     uzu_norm_add_args b = *a;
     if (!b.in_stride) b.in_stride = b.n;
-    if (b.kind == 1 && (!b.residual || !b.output || b.next_kind == 1))
+    if (b.kind == 1 && !b.residual_bf16 && (!b.residual || !b.output || b.next_kind == 1))
         launch(cmd, "norm_add_elementwise_kernel", norm_add_elementwise_kernel, dim3((b.n + 255) / 256, b.rows), dim3(256), 0, b);
     else
         launch(cmd, "norm_add_kernel", norm_add_kernel, dim3(b.rows), dim3(256), 0, b);
@@ -753,13 +879,15 @@ void uzu_token_gate_encode(uzu_command_buffer* cmd, const uzu_token_gate_args* a
 }
 
 void uzu_clamped_glu_encode(uzu_command_buffer* cmd, uint64_t gate_up, uint64_t output, uint32_t rows, uint32_t f, float limit, float alpha) {
-    if (!encodable(cmd, "clamped_glu") || rows == 0 || f == 0) return;
-    launch(cmd, "clamped_glu_kernel", clamped_glu_kernel, dim3(blocks256((size_t)rows * f)), dim3(256), 0, (const float*)gate_up, (float*)output, rows, f, limit, alpha);
+    uzu_glu_args a{};
+    a.gate_up = gate_up; a.output = output; a.rows = rows; a.f = f; a.kind = 0; a.limit = limit; a.alpha = alpha;
+    uzu_glu_encode(cmd, &a);
 }
 
 void uzu_silu_glu_encode(uzu_command_buffer* cmd, uint64_t gate_up, uint64_t output, uint32_t rows, uint32_t f) {
-    if (!encodable(cmd, "silu_glu") || rows == 0 || f == 0) return;
-    launch(cmd, "silu_glu_kernel", silu_glu_kernel, dim3(blocks256((size_t)rows * f)), dim3(256), 0, (const float*)gate_up, (float*)output, rows, f);
+    uzu_glu_args a{};
+    a.gate_up = gate_up; a.output = output; a.rows = rows; a.f = f; a.kind = 1;
+    uzu_glu_encode(cmd, &a);
 }
 
 void uzu_unary_f32_encode(uzu_command_buffer* cmd, uint64_t input, uint32_t in_stride, uint64_t output, uint32_t out_stride, uint32_t rows,
@@ -796,21 +924,30 @@ void uzu_table_route_encode(uzu_command_buffer* cmd, const uzu_table_route_args*
 void uzu_topk_route_encode(uzu_command_buffer* cmd, const uzu_topk_route_args* a) {
     if (!encodable(cmd, "topk_route")) return;
     if (!a->logits || !a->group_offsets || !a->rows_map || !a->pair_pos || !a->pair_weight || a->top == 0 || a->experts == 0 || a->experts > 8192 ||
-        a->top > a->experts || a->logits_stride < a->experts) {
+        a->top > a->experts || a->logits_stride < a->experts || a->weight_kind > 2 || (a->always && a->weight_kind != 2)) {
         cmd->record_error(UZU_ERROR_INVALID_ARGUMENT, "topk_route: null operand or bad expert / top count");
         return;
     }
+    if (a->weight_kind == 2 && a->choice_groups > 1 &&
+        (a->choice_groups > 32 * ROUTE_GROUPS || a->experts % a->choice_groups || a->choice_keep == 0 || a->choice_keep > a->choice_groups ||
+         a->top > a->experts / a->choice_groups * a->choice_keep)) {
+        cmd->record_error(UZU_ERROR_INVALID_ARGUMENT, "topk_route: the groups must divide the experts (at most 256 groups), and the kept ones hold at least `top` experts");
+        return;
+    }
     if (a->rows == 0) return;
-    const size_t smem = (a->experts + 1) * sizeof(uint32_t) + (size_t)a->rows * a->top * sizeof(uint16_t);
-    if (smem > 48 * 1024) {
+    const size_t smem = (a->experts + a->always + 1) * sizeof(uint32_t) + (size_t)a->rows * (a->top + a->always) * sizeof(uint16_t);
+    if (smem > ROUTE_SMEM) {
         cmd->record_error(UZU_ERROR_UNSUPPORTED, "topk_route: rows * top too large for one pass");
         return;
     }
+    static std::atomic<uint64_t> done[2];
     if (a->scratch && a->rows >= 64) {          // the choice over many CTAs (8 rows each), then the one CTA that builds the lists
+        opt_in_dynamic_smem(cmd, topk_route_kernel<2>, (int)ROUTE_SMEM, done[1]);
         launch(cmd, "topk_route_kernel", topk_route_kernel<1>, dim3((a->rows + 7) / 8), dim3(256), 0, *a);
         launch(cmd, "topk_route_kernel", topk_route_kernel<2>, dim3(1), dim3(1024), smem, *a);
         return;
     }
+    opt_in_dynamic_smem(cmd, topk_route_kernel<0>, (int)ROUTE_SMEM, done[0]);
     launch(cmd, "topk_route_kernel", topk_route_kernel<0>, dim3(1), dim3(1024), smem, *a);
 }
 

@@ -1,7 +1,8 @@
 // Windowed softmax attention with kept first tokens, rotated keys AND rotated values.
 //   visibility:  key j is seen from position p when j <= p and (p - j < window or j < keep_first); kept tokens keep their true positions;
 //                with a chunk size also only from inside its own chunk, floor(j / chunk) = floor(p / chunk), counted from position 0
-//   score:       s = scale * temp[h] * q . k, then softcap * tanh(s / softcap); ordinary softmax over the visible keys
+//   score:       s = scale * temp[h] * q . k, then softcap * tanh(s / softcap), then less slope[h] per position of distance; ordinary softmax
+//                over the visible keys
 //   rotation:    q and k turn by their position over the first 2 * rot_pairs channels (pairs (2i, 2i+1), or (i, i + rot_pairs) with
 //                rot_halves); the value of position j turns
 //                by j over 2 * v_pairs channels with its own frequencies and is cached so; a head's weighted sum at position p is turned
@@ -160,6 +161,7 @@ __global__ void __launch_bounds__(WA_WARPS * 32) window_attention_kernel(const u
     const uint32_t dwords = (a.dim + EPW - 1) / EPW, vwords = (a.vdim + EPW - 1) / EPW;
     const float qscale = a.scale * (a.head_temp ? reinterpret_cast<const float*>(a.head_temp)[h] : 1.0f);
     const float cap = a.softcap, inv_cap = a.softcap > 0.0f ? 1.0f / a.softcap : 0.0f;
+    const float slope = a.dist_slope ? reinterpret_cast<const float*>(a.dist_slope)[h] : 0.0f;
     float q[WPL][EPW], acc[WPL][EPW];
     {
         const float* qrow = reinterpret_cast<const float*>(a.query) + ((size_t)t * a.heads + h) * a.dim;
@@ -206,6 +208,7 @@ __global__ void __launch_bounds__(WA_WARPS * 32) window_attention_kernel(const u
 #pragma unroll
         for (int u = 0; u < WA_UNROLL; ++u) {
             if (cap > 0.0f) s[u] = cap * tanhf(s[u] * inv_cap);
+            s[u] -= slope * (float)(p - key[u]);
             if (i0 + u >= i_end) s[u] = -INFINITY;
             batch_m = fmaxf(batch_m, s[u]);
         }
@@ -258,7 +261,8 @@ __global__ void __launch_bounds__(WA_WARPS * 32) window_attention_kernel(const u
     float* result = wa_smem + WA_WARPS * a.vdim;     // [vdim]
     // a sink adds exp(sink - max) to the denominator; a head gate multiplies the head's result by its sigmoid
     const float sink = a.sinks ? reinterpret_cast<const float*>(a.sinks)[h] : -INFINITY;
-    const float gate = a.head_gate ? 1.0f / (1.0f + expf(-reinterpret_cast<const float*>(a.head_gate)[(size_t)t * a.head_gate_stride + h])) : 1.0f;
+    const float gate = (a.head_gate ? 1.0f / (1.0f + expf(-reinterpret_cast<const float*>(a.head_gate)[(size_t)t * a.head_gate_stride + h])) : 1.0f) *
+                       (a.out_scale != 0.0f ? a.out_scale : 1.0f);
     if (splits == 1) {
         const float norm = gate / (a.sinks ? cta_l + expf(sink - cta_m) : cta_l);
         for (uint32_t c = tid; c < a.vdim; c += blockDim.x) {
@@ -298,7 +302,6 @@ __global__ void __launch_bounds__(WA_WARPS * 32) window_attention_kernel(const u
         float all_l = 0.0f;
         for (uint32_t sp = 0; sp < splits; ++sp) all_l = fmaf(split_l[sp], split_f[sp], all_l);      // in split order
         if (a.sinks) all_l += expf(sink - all_m);
-        all_l /= gate;
         for (uint32_t c = tid; c < a.vdim; c += blockDim.x) {
             float v = 0.0f;
             uint32_t sp = 0;
@@ -310,13 +313,13 @@ __global__ void __launch_bounds__(WA_WARPS * 32) window_attention_kernel(const u
                 for (int u = 0; u < 8; ++u) v = fmaf(x[u], split_f[sp + u], v);
             }
             for (; sp < splits; ++sp) v = fmaf(__ldcg(parts + (size_t)sp * pw + 2 + c), split_f[sp], v);
-            result[c] = v / all_l;
+            result[c] = v / all_l * gate;
         }
         if (tid == 0) *ticket = 0;
     }
     __syncthreads();
     // the head's sum turns back by its own position
-    float* out = reinterpret_cast<float*>(a.out) + ((size_t)t * a.heads + h) * a.vdim;
+    float* out = reinterpret_cast<float*>(a.out) + (size_t)t * (a.out_stride ? a.out_stride : a.heads * a.vdim) + (size_t)h * a.vdim;
     const float* vc = a.v_pairs ? reinterpret_cast<const float*>(a.v_cosines) + (size_t)p * a.v_pairs : nullptr;
     const float* vs = a.v_pairs ? reinterpret_cast<const float*>(a.v_sines) + (size_t)p * a.v_pairs : nullptr;
     for (uint32_t i = tid; 2 * i < a.vdim; i += blockDim.x) {
@@ -364,7 +367,7 @@ void uzu_window_attention_encode(uzu_command_buffer* cmd, const uzu_window_atten
     if (!encodable(cmd, "window_attention")) return;
     if (!a->query || !a->keys || !a->values || !a->out || a->heads == 0 || a->kv_heads == 0 || a->heads % a->kv_heads || a->dim == 0 || a->vdim == 0 ||
         a->dim > 512 || a->vdim > 512 || (a->cache_dt != UZU_DT_BF16 && a->cache_dt != UZU_DT_F32) || 2 * a->v_pairs > a->vdim ||
-        (a->v_pairs && (!a->v_cosines || !a->v_sines))) {
+        (a->v_pairs && (!a->v_cosines || !a->v_sines)) || (a->out_stride && a->out_stride < a->heads * a->vdim)) {
         cmd->record_error(UZU_ERROR_INVALID_ARGUMENT, "window_attention: null operand, kv_heads not dividing heads, head size outside 1..512, or bad cache type");
         return;
     }

@@ -3,7 +3,7 @@
 // first the tiles of the kept first tokens that lie before the window, then the tiles from the window's start of the CTA's first row up
 // to its last row; the next tile's keys and values arrive by cp.async while the current one is used. mma.sync.m16n8k16 (bf16 x bf16 -> f32):
 //   S = (q * scale * temp) . K^T   with q = q_hi + q_lo, two bf16 numbers per f32 query entry (two MMAs per tile of S);
-//   soft cap, mask (j <= i and (inside the window and chunk of i, or j < keep_first)) and the running (max, sum) of the softmax in f32 on the accumulator
+//   soft cap, distance slope, mask (j <= i and (inside the window and chunk of i, or j < keep_first)) and the running (max, sum) of the softmax in f32 on the accumulator
 //   fragment, in units of ln 2; the accumulators of O are rescaled when a row's maximum moves;
 //   O += p . V                     with p = p_hi + p_lo again, the fragment of S re-used as the A fragment, V by ldmatrix.trans.
 // The split keeps the error of the query and of the weights below 2^-16 relative, so only the cache's own bf16 rounding remains.
@@ -77,6 +77,7 @@ __global__ void __launch_bounds__(128) window_attention_mma_kernel(const uzu_win
     const float qscale = a.scale * (a.head_temp ? reinterpret_cast<const float*>(a.head_temp)[h] : 1.0f);
     const bool capped = a.softcap > 0.0f;
     const float cap2 = a.softcap * kLog2e, inv_cap2 = capped ? 2.0f * kLog2e / a.softcap : 0.0f;      // tanh(x) = 1 - 2 / (2^(2 x log2 e) + 1)
+    const float slope2 = a.dist_slope ? reinterpret_cast<const float*>(a.dist_slope)[h] * kLog2e : 0.0f;
     const __nv_bfloat16* keys = reinterpret_cast<const __nv_bfloat16*>(a.keys) + (size_t)kvh * dim;
     const __nv_bfloat16* values = reinterpret_cast<const __nv_bfloat16*>(a.values) + (size_t)kvh * vdim;
     const size_t kstride = (size_t)a.kv_heads * dim, vstride = (size_t)a.kv_heads * vdim;
@@ -188,8 +189,9 @@ __global__ void __launch_bounds__(128) window_attention_mma_kernel(const uzu_win
                 float x = s[n][c];
                 if (capped) x = cap2 * (1.0f - __fdividef(2.0f, exp2f(x * inv_cap2) + 1.0f));
                 else x *= kLog2e;
+                const uint32_t i = i_lo + 8 * (c >> 1), j = j0 + n * 8 + t4 * 2 + (c & 1);
+                x = fmaf(-slope2, (float)(int)(i - j), x);
                 if (!all_visible) {
-                    const uint32_t i = i_lo + 8 * (c >> 1), j = j0 + n * 8 + t4 * 2 + (c & 1);
                     if (!(j <= i && (j >= lo_row[c >> 1] || j < keep))) x = -INFINITY;
                 }
                 s[n][c] = x;
@@ -258,12 +260,12 @@ __global__ void __launch_bounds__(128) window_attention_mma_kernel(const uzu_win
         l += __shfl_xor_sync(0xffffffffu, l, 1);
         l += __shfl_xor_sync(0xffffffffu, l, 2);
         if (a.sinks) l += exp2f(reinterpret_cast<const float*>(a.sinks)[h] * kLog2e - run_m[r]);      // the sink's term (the maximum is in units of ln 2)
-        inv_l[r] = 1.0f / l;
+        inv_l[r] = (a.out_scale != 0.0f ? a.out_scale : 1.0f) / l;
         const uint32_t row = row_lo + 8 * r;
         if (a.head_gate && row < rows_here)
             inv_l[r] *= 1.0f / (1.0f + expf(-reinterpret_cast<const float*>(a.head_gate)[(size_t)(m0 + row) * a.head_gate_stride + h]));
     }
-    const size_t row_stride = (size_t)a.heads * vdim;
+    const size_t row_stride = a.out_stride ? a.out_stride : (size_t)a.heads * vdim;
     float* out = reinterpret_cast<float*>(a.out) + (size_t)m0 * row_stride + (size_t)h * vdim;
 #pragma unroll
     for (int n = 0; n < 2 * DV; ++n) {
@@ -302,7 +304,7 @@ static void launch_window_attention_mma(uzu_command_buffer* cmd, const uzu_windo
 bool encode_window_attention_mma(uzu_command_buffer* cmd, const uzu_window_attention_args& a) {
     static const bool off = getenv("UZU_WINDOW_NO_MMA") != nullptr;       // A/B runs
     if (off || a.cache_dt != UZU_DT_BF16 || a.rows < WM_BM || a.dim % 16 || a.vdim % 16 || a.dim > 128 || a.vdim > 128) return false;
-    if ((a.keys & 15) || (a.values & 15) || (a.query & 7) || (a.out & 7) || a.dynamic_position || ((a.heads * a.vdim) & 1)) return false;
+    if ((a.keys & 15) || (a.values & 15) || (a.query & 7) || (a.out & 7) || a.dynamic_position || ((a.heads * a.vdim) & 1) || (a.out_stride & 1)) return false;
     const bool k8 = a.dim > 64, v8 = a.vdim > 64;
     if (k8 && v8) launch_window_attention_mma<8, 8>(cmd, a);
     else if (k8) launch_window_attention_mma<8, 4>(cmd, a);
