@@ -720,13 +720,14 @@ def family_models(size: str, family: str = "punilix"):
     feed-forward in its recurrent layers and 2 of 8 table-routed experts in its attention layers; Vakesun (windowed latent attention that
     keeps or borrows its latents, full attention, matrix memory; relu^2 feed-forwards, a per-layer token input) beside Punilix with the
     same number of layers (at least four); Relidra (gated delta rule layers and chunked attention layers over two residual streams, two-matrix
-    gelu feed-forwards) beside Punilix with the same number of layers."""
+    gelu feed-forwards) beside Punilix with the same number of layers; Bonolorn (window attention beside lightning attention in every layer,
+    dense and routed feed-forwards in turn) beside Vugipel with window attention beside retention in every layer and the same active sizes."""
     from uzu_b200 import synth
     width, ff, blocks, vocab = FAMILY_SIZES[size]
     base = Path(os.environ.get("UZU_MODEL_CACHE", "/dev/shm/uzu_b200_models"))
     base.mkdir(parents=True, exist_ok=True)
     pdir = base / f"punilix-{size}"
-    if not (pdir / ".done").exists():
+    if family in ("punilix", "gamanex", "relidra") and not (pdir / ".done").exists():
         synth.write_punilix_model(synth.punilix_preset(width=width, vocab=vocab, blocks=blocks, ff=ff), pdir, seed=0)
         (pdir / ".done").write_text("ok")
     if family == "gamanex":
@@ -741,6 +742,15 @@ def family_models(size: str, family: str = "punilix"):
             synth.write_relidra_model(synth.relidra_preset(width=width, vocab=vocab, layers=2 * blocks, ff=ff, chunk=512, streams=2), rdir, seed=0)
             (rdir / ".done").write_text("ok")
         return [("relidra", rdir, 2.0), ("closest_existing", pdir, 2.0)]
+    if family == "bonolorn":    # beside Vugipel: the same two mixers side by side, routed experts in every other layer, the same active sizes
+        bdir, vdir = base / f"bonolorn-{size}", base / f"vugipel-side-{size}"
+        if not (bdir / ".done").exists():
+            synth.write_bonolorn_model(synth.bonolorn_preset(width=width, vocab=vocab, layers=2 * blocks, ff=ff), bdir, seed=0)
+            (bdir / ".done").write_text("ok")
+        if not (vdir / ".done").exists():
+            synth.write_vugipel_model(synth.vugipel_side_by_side_preset(width=width, vocab=vocab, layers=2 * blocks, ff=ff), vdir, seed=0)
+            (vdir / ".done").write_text("ok")
+        return [("bonolorn", bdir, 2.0), ("closest_existing", vdir, 2.0)]
     if family == "vakesun":     # beside Punilix (latent attention + a matrix-state recurrence, dense feed-forwards) with the same number of layers
         layers = max(4, 2 * blocks)
         vdir, mdir = base / f"vakesun-{size}", base / f"punilix-{size}-{layers}"
@@ -789,7 +799,7 @@ def family_compare(args):
     with B.Context(0) as ctx:
         for size in sizes:
             models = family_models(size, args.family)
-            line = {"family_compare": size, "family": args.family, "closest_existing": {"gamanex": "punilix (bf16)", "vugipel": "punilix with 2 of 8 table-routed experts (bf16)", "vakesun": "punilix with the same number of layers (bf16)", "relidra": "punilix (bf16)"}.get(args.family, "gated attention + DeltaNet hybrid (int4)"), "prefill_tokens": prompt_len, "decode_steps": steps, "peaks": {"hbm_gbs": hbm, "hbm_source": hbm_src,
+            line = {"family_compare": size, "family": args.family, "closest_existing": {"gamanex": "punilix (bf16)", "vugipel": "punilix with 2 of 8 table-routed experts (bf16)", "vakesun": "punilix with the same number of layers (bf16)", "relidra": "punilix (bf16)", "bonolorn": "vugipel with the same two kinds of mixers in every layer (bf16)"}.get(args.family, "gated attention + DeltaNet hybrid (int4)"), "prefill_tokens": prompt_len, "decode_steps": steps, "peaks": {"hbm_gbs": hbm, "hbm_source": hbm_src,
                                                                                                          "tensor_tflops": tens, "tensor_source": tens_src}}
             for name, d, bytes_per_weight in models:
                 with B.Engine(ctx, d, max_context_length=prompt_len + steps + 64, use_cuda_graph=not args.no_graph) as eng:
@@ -837,7 +847,7 @@ def main():
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--batch", type=int, default=1, help="decode this many independent sequences together (<= 16), one weight pass per step")
     ap.add_argument("--tp", type=int, default=1, help="tensor-parallel size: shard ONE model over this many ranks (= --gpus) instead of replicas")
-    ap.add_argument("--family", choices=["punilix", "gamanex", "vugipel", "vakesun", "relidra"], default=None,
+    ap.add_argument("--family", choices=["punilix", "gamanex", "vugipel", "vakesun", "relidra", "bonolorn"], default=None,
                     help="instead of the headline workload: prefill / decode throughput of this model family beside the closest existing one at equal layer sizes (1 GPU)")
     ap.add_argument("--family-sizes", default="", help="comma list of " + ", ".join(sorted(FAMILY_SIZES)) + " (default 1k,2k)")
     args = ap.parse_args()

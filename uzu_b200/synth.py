@@ -830,3 +830,109 @@ def relidra_preset(width=2048, vocab=32768, layers=6, ff=None, chunk=512, stream
         else:
             out.append(relidra_attention_layer(heads, max(heads // 4, 1), 128, chunk, relidra_dense_mlp(ff), rot_dims=64, rot_base=1e6, factor=4.0))
     return relidra_config(width, vocab, out, streams=streams, loop=loop)
+
+
+# ---- Bonolorn: window attention with distance slopes beside lightning attention, output-normed layers, group-limited routed experts ----------
+
+def bonolorn_dense_mlp(ff: int) -> dict:
+    return {"kind": "dense", "ff": ff}
+
+
+def bonolorn_moe_mlp(ff: int, experts: int, top: int, groups: tuple = (1, 1), scale: float = 1.0, limit: float = 7.0, shared: int = 0,
+                     shared_limit: float | None = None) -> dict:
+    ml = {"kind": "moe", "expert": {"ff": ff, "limit": float(limit)},
+          "router": {"experts": experts, "top": top, "scale": float(scale), "groups": {"count": groups[0], "keep": groups[1]}}}
+    if shared:
+        ml["shared"] = {"ff": shared, "limit": float(limit if shared_limit is None else shared_limit)}
+    return ml
+
+
+def bonolorn_layer(heads: int, kv_heads: int, dim: int, vdim: int, window: int, r_heads: int, r_dim: int, r_vdim: int, mlp: dict | None,
+                   scale: float | None = None, decay: list | None = None, left_scale: float = 1.0, right_scale: float = 1.0) -> dict:
+    left = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": float(dim ** -0.5 if scale is None else scale),
+            "mask": {"size": int(window)}}
+    if decay is None:
+        decay = [1.0 - 1.0 / (20.0 * (h % 8 + 1)) for h in range(r_heads)]
+    right = {"heads": r_heads, "dim": r_dim, "vdim": r_vdim, "decay": [float(d) for d in decay]}
+    return {"type": "parallel", "mixer": {"left": left, "left_scale": float(left_scale), "right": right, "right_scale": float(right_scale)}, "mlp": mlp}
+
+
+def bonolorn_config(width: int, vocab: int, layers: list, eps: float = 1e-6, residual_mult: float = 0.5) -> dict:
+    return {"architecture": "Bonolorn", "width": width, "vocab": vocab, "norm": {"eps": eps}, "residual_mult": residual_mult, "layers": layers}
+
+
+def bonolorn_tensors(config: dict, seed: int = 0) -> dict:
+    """Seeded random tensors of a Bonolorn config: f32 values that bf16 holds exactly."""
+    rng = np.random.default_rng(seed)
+    W, V = config["width"], config["vocab"]
+
+    def bf(x):
+        return st_bits_to_f32(f32_to_bf16_bits(np.asarray(x, np.float32)))
+
+    def mat(rows, cols, gain=1.0):
+        return bf(rng.standard_normal((rows, cols), dtype=np.float32) * (gain / np.sqrt(cols)))
+
+    def vec(n, mean=0.0, spread=0.1):
+        return bf(mean + spread * rng.standard_normal(n, dtype=np.float32))
+
+    def unit(p, f):
+        t[p + "gate"], t[p + "up"], t[p + "down"] = mat(f, W, 1.3), mat(f, W, 1.3), mat(W, f)
+
+    t = {"embed": mat(V, W, np.sqrt(W)), "final.norm": vec(W, 1.0)}
+    for i, L in enumerate(config["layers"]):
+        p = f"l{i}."
+        A, R = L["mixer"]["left"], L["mixer"]["right"]
+        H, G, D, Dv = A["heads"], A["kv_heads"], A["dim"], A["vdim"]
+        Hr, Dr, Dvr = R["heads"], R["dim"], R["vdim"]
+        l, r = p + "mix.left.", p + "mix.right."
+        t[p + "norm1"] = vec(W, 1.0)
+        t[l + "q"], t[l + "k"], t[l + "v"] = mat(H * D, W), mat(G * D, W), mat(G * Dv, W)
+        t[l + "q.norm"], t[l + "k.norm"] = vec(D, 1.0, 0.2), vec(D, 1.0, 0.2)
+        t[l + "g"], t[l + "o"] = mat(H, W, 1.5), mat(W, H * Dv)
+        t[r + "q"], t[r + "k"], t[r + "v"] = mat(Hr * Dr, W), mat(Hr * Dr, W), mat(Hr * Dvr, W)
+        t[r + "g"], t[r + "o"], t[r + "norm"] = mat(Hr * Dvr, W, 1.5), mat(W, Hr * Dvr), vec(Hr * Dvr, 1.0)
+        ml = L.get("mlp")
+        if ml is None:
+            continue
+        t[p + "norm2"] = vec(W, 1.0)
+        if ml["kind"] == "dense":
+            unit(p + "mlp.", ml["ff"])
+            continue
+        E = ml["router"]["experts"]
+        t[p + "mlp.router"], t[p + "mlp.correction"] = mat(E, W, 1.5), vec(E, 0.0, 0.2)
+        for x in range(E):
+            unit(f"{p}mlp.e{x}.", ml["expert"]["ff"])
+        if ml.get("shared"):
+            unit(p + "mlp.shared.", ml["shared"]["ff"])
+    return t
+
+
+def write_bonolorn_model(config: dict, path, seed: int = 0, tensors: dict | None = None) -> Path:
+    """config.json + model.safetensors (bf16). `tensors` overrides the seeded random ones (values are rounded to bf16)."""
+    return write_punilix_model(config, path, seed, tensors if tensors is not None else bonolorn_tensors(config, seed))
+
+
+def bonolorn_preset(width=2048, vocab=32768, layers=6, ff=None, experts=8, top=2, window=1024) -> dict:
+    """A layer stack of realistic sizes for benchmarks: every layer has 128-channel window attention and half as many lightning heads of 128 x 128;
+    the feed-forward is dense in one layer and in the next `top` of `experts` experts (two of four groups stay) beside a shared expert, of the
+    same active size."""
+    ff = ff or 4 * width
+    heads = max(width // 128, 1)
+    out = []
+    for i in range(layers):
+        mlp = bonolorn_dense_mlp(ff) if i % 2 == 0 else bonolorn_moe_mlp(ff // (2 * top), experts, top, groups=(4, 2), scale=1.5, shared=ff // 2)
+        out.append(bonolorn_layer(heads, max(heads // 4, 1), 128, 128, window, max(heads // 2, 1), 128, 128, mlp, left_scale=0.9, right_scale=1.2))
+    return bonolorn_config(width, vocab, out)
+
+
+def vugipel_side_by_side_preset(width=2048, vocab=32768, layers=6, ff=None, experts=8, top=2, window=1024, keep_first=4) -> dict:
+    """Vugipel with window attention and retention side by side in every layer; the feed-forward is a single expert of size `ff` in one layer and
+    `top` of `experts` routed experts of the same active size in the next."""
+    ff = ff or 4 * width
+    heads = max(width // 128, 1)
+    out = []
+    for i in range(layers):
+        mlp = vugipel_moe_mlp(ff, 1, 1) if i % 2 == 0 else vugipel_moe_mlp(ff // top, experts, top)
+        out.append(vugipel_parallel_layer(heads, max(heads // 4, 1), 128, 128, window, keep_first, max(heads // 2, 1), 128, 128, mlp,
+                                          softcap=30.0, left_scale=0.9, right_scale=1.2))
+    return vugipel_config(width, vocab, out, eps=1e-6)
