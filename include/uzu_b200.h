@@ -476,7 +476,7 @@ typedef struct uzu_dense_linear_args {
     float scale;                   /* applied to the product before gate / bias / accumulation */
     uint32_t a_op;                 /* applied to every A element as it is read: 0 none, 1 tanh, 2 max(x, 0)^2 */
     uint32_t gate_ld;
-    uint32_t pair_rows;            /* m <= 8 only. Non-zero: W has a second block of rows `pair_rows` below the first; feature col forms
+    uint32_t pair_rows;            /* m <= 8, or the tcgen05 form. Non-zero: W has a second block of rows `pair_rows` below the first; feature col forms
                                       g = A.W[col], u = A.W[col + pair_rows] and stores the clamped gated unit
                                       min(g, limit) * sigmoid(alpha * min(g, limit)) * (clamp(u, -limit, limit) + 1) */
     float glu_limit, glu_alpha;
@@ -497,7 +497,7 @@ typedef struct uzu_dense_linear_args {
     uint64_t token_ids, token_table;   /* token_table of type token_gate_dt [vocab, token_table_stride], token_ids u32 [rows] (ids >= token_vocab read 0) */
     uint32_t token_table_stride, token_column, token_vocab;
     uint32_t a_bf16;               /* 1: A is bf16 [m, k] (lda = k, 16-byte aligned), e.g. rows of a bf16 cache; only the tcgen05 form takes it
-                                      (bf16 weights, batch 1, m >= 128, k a multiple of 64, n >= 64), no A operation */
+                                      (bf16 weights, batch 1 or row groups, m >= 128, k a multiple of 64, n >= 8), no A operation */
     /* Stream epilogue (streams 1..4; batch = 1, no accumulate; not on the tcgen05 form): the finished product y is a sublayer's result over a
      * residual kept as `streams` copies x_s (f32 [rows, streams, n], stream_x). Element by element, from the old copies,
      *   x_t <- sum_s stream_mix[s, t] x_s + stream_out[t] y,   stream_u[row, col] = sum_t stream_in[t] x_t   (stream_in 0: all ones)

@@ -56,6 +56,13 @@ def close(got, ref, tol, what=""):
     assert err <= tol, f"{what}: max error {err:.3e} of the rms exceeds {tol:.1e}"
 
 
+def close_bf16(bits, ref, what=""):
+    """a value whose f32 form is accurate, rounded to bf16 once"""
+    ref = np.asarray(ref, np.float64)
+    err = np.abs(from_bits(bits) - ref) - 2.0 ** -8 * np.abs(ref)
+    assert err.max() <= 5e-5 * np.sqrt((ref ** 2).mean()), what
+
+
 # ---- embedding and norms -----------------------------------------------------------------------------------------------------------------
 @pytest.mark.parametrize("n", [7, 64, 514])
 @pytest.mark.parametrize("prefix,dynamic", [(0, False), (1000, False), (123457, True)])
@@ -171,7 +178,62 @@ def test_gated_units(ctx, rows, f, kind):
     run(ctx, "uzu_glu_encode", C.byref(B.GluArgs(gate_up=bg.ptr, output=bh.ptr, group_offsets=bl.ptr, rows=rows, f=f, kind=kind, output_bf16=1, last_group=2, limit=1.5,
                                                  limit_last=0.3, alpha=1.702)))
     ref = torch.cat([pair_ref(kind, g[:split], u[:split], 1.5), pair_ref(kind, g[split:], u[split:], 0.3)]).numpy()
-    close(from_bits(bh.numpy(np.uint16, (rows, f))), ref, 3e-2, "bf16 unit, two limits")
+    close_bf16(bh.numpy(np.uint16, (rows, f)), ref, "bf16 unit, two limits")
+
+
+@pytest.mark.parametrize("m,n,k", [(128, 64, 64), (300, 200, 192), (129, 36, 128), (1000, 8, 64)])
+@pytest.mark.parametrize("kind", [0, 1, 2])
+@pytest.mark.parametrize("out_bf16", [True, False])
+def test_gated_units_as_the_epilogue_of_a_long_product(ctx, m, n, k, kind, out_bf16):
+    rng = np.random.default_rng(m + kind)
+    x, w, rs = bf16_exact(f32(rng, m, k)), bf16_exact(f32(rng, 2 * n, k, spread=2 * k ** -0.5)), f32(rng, m)
+    bx, bw, ws, br = ctx.upload(x), ctx.upload(bf16_bits(w)), ctx.upload(np.zeros((m, k), np.uint16)), ctx.upload(rs)
+    for row_scale in (False, True):
+        bd = ctx.upload(np.zeros((m, n), np.uint16 if out_bf16 else np.float32))
+        run(ctx, "uzu_dense_linear_encode", C.byref(B.DenseLinearArgs(a=bx.ptr, w=bw.ptr, d=bd.ptr, workspace=ws.ptr, row_scale=br.ptr if row_scale else 0, m=m, n=n, k=k, lda=k,
+                                                                      ldd=n, batch=1, weights_dt=B.DT_BF16, scale=1.0, pair_rows=n, glu_kind=kind, glu_limit=0.7, glu_alpha=1.702,
+                                                                      d_bf16=int(out_bf16))))
+        z = t64(x) @ t64(w).T * (t64(rs)[:, None] if row_scale else 1.0)
+        ref = pair_ref(kind, z[:, :n], z[:, n:], 0.7).numpy()
+        if out_bf16:
+            close_bf16(bd.numpy(np.uint16, (m, n)), ref, f"row scale {row_scale}")
+        else:
+            close(bd.numpy(np.float32, (m, n)), ref, 5e-5, f"row scale {row_scale}")
+    assert ctx.lib.uzu_debug_dense_umma_error() == 0
+
+
+@pytest.mark.parametrize("m,n,k,groups", [(128, 64, 64, 3), (300, 72, 192, 5), (513, 200, 64, 2)])
+def test_row_groups_of_long_products(ctx, m, n, k, groups):
+    """Compact rows gathered from bf16 activation rows, groups from empty to all rows: plain and as gated units; then compact rows in their own order."""
+    rng = np.random.default_rng(m)
+    x, w = bf16_exact(f32(rng, m, k)), bf16_exact(f32(rng, groups, 2 * n, k, spread=2 * k ** -0.5))
+    of = np.sort(rng.integers(0, groups, 2 * m))
+    of[of == 1] = 0 if groups > 2 else 1                       # one group stays empty
+    sizes = [int((of == g).sum()) for g in range(groups)]
+    sizes[-1] = min(sizes[-1], m)
+    sizes = [min(s, m) for s in sizes]
+    total = sum(sizes)
+    rows_map = np.concatenate([np.sort(rng.permutation(m)[:s]) for s in sizes]).astype(np.uint32)
+    off = np.cumsum([0] + sizes).astype(np.uint32)
+    bx, bw, bo, bm, ws = ctx.upload(bf16_bits(x)), ctx.upload(bf16_bits(w)), ctx.upload(off), ctx.upload(rows_map), ctx.upload(np.zeros(8, np.uint16))
+    base = dict(w=bw.ptr, workspace=ws.ptr, m=m, k=k, lda=k, weights_dt=B.DT_BF16, scale=1.0, batch=groups, w_z_stride=2 * n * k, group_offsets=bo.ptr, a_bf16=1)
+    z = torch.cat([t64(x[rows_map[off[g]:off[g + 1]]]) @ t64(w[g]).T for g in range(groups)])
+    bd = ctx.upload(np.full((total + 1, 2 * n), 7.0, np.float32))
+    run(ctx, "uzu_dense_linear_encode", C.byref(B.DenseLinearArgs(a=bx.ptr, rows_map=bm.ptr, d=bd.ptr, n=2 * n, ldd=2 * n, **base)))
+    got = bd.numpy(np.float32, (total + 1, 2 * n))
+    close(got[:total], z.numpy(), 3e-5, "plain")
+    assert (got[total] == 7.0).all()
+    bd = ctx.upload(np.zeros((total, n), np.float32))
+    run(ctx, "uzu_dense_linear_encode", C.byref(B.DenseLinearArgs(a=bx.ptr, rows_map=bm.ptr, d=bd.ptr, n=n, ldd=n, pair_rows=n, glu_kind=0, glu_limit=0.9, glu_alpha=1.702,
+                                                                  glu_last_group=groups - 1, glu_limit_last=0.3, **base)))
+    last = off[groups - 1]
+    ref = torch.cat([pair_ref(0, z[:last, :n], z[:last, n:], 0.9), pair_ref(0, z[last:, :n], z[last:, n:], 0.3)])
+    close(bd.numpy(np.float32, (total, n)), ref.numpy(), 3e-5, "gated units")
+    y = bf16_exact(f32(rng, total, k))
+    by, bd = ctx.upload(bf16_bits(y)), ctx.upload(np.zeros((total, 2 * n), np.float32))
+    run(ctx, "uzu_dense_linear_encode", C.byref(B.DenseLinearArgs(a=by.ptr, d=bd.ptr, n=2 * n, ldd=2 * n, **base)))
+    close(bd.numpy(np.float32, (total, 2 * n)), torch.cat([t64(y[off[g]:off[g + 1]]) @ t64(w[g]).T for g in range(groups)]).numpy(), 3e-5, "compact rows")
+    assert ctx.lib.uzu_debug_dense_umma_error() == 0
 
 
 # ---- router --------------------------------------------------------------------------------------------------------------------------------

@@ -815,7 +815,7 @@ extern "C" void uzu_dense_linear_encode(uzu_command_buffer* cmd, const uzu_dense
         cmd->record_error(UZU_ERROR_INVALID_ARGUMENT, "dense_linear: the sandwich / token-gate epilogues take one plain product (no accumulate, no pairs, no batch)");
         return;
     }
-    if (a.d_op > 1 || (a.pair_rows && a.d_op) || (a.d_bf16 && a.accumulate) ||
+    if (a.d_op > 1 || (a.pair_rows && a.d_op) || (a.d_bf16 && (a.accumulate || a.m <= (uint32_t)DL_MAX_ROWS)) ||
         (a.streams && (a.streams > (uint32_t)DL_MAX_STREAMS || !a.stream_x || !a.stream_mix || !a.stream_out || !a.stream_u || a.accumulate || a.batch != 1 || a.pair_rows ||
                        a.group_offsets || a.rows_map || a.post_weight || a.token_table || a.d_bf16))) {
         cmd->record_error(UZU_ERROR_INVALID_ARGUMENT, "dense_linear: unknown D operation, a bf16 D that accumulates, or a stream epilogue that is not one plain product");
@@ -838,9 +838,10 @@ extern "C" void uzu_dense_linear_encode(uzu_command_buffer* cmd, const uzu_dense
         const bool dense_rows = a.lda == 0 || a.lda == a.k;
         a.lda = a.k;
         if (!dense_rows || a.a_op || a.post_weight || a.token_table || a.streams || !dense_umma_applicable(a)) {
-            cmd->record_error(UZU_ERROR_UNSUPPORTED, "dense_linear: bf16 activations need the tcgen05 form (bf16 weights, dense rows, a workspace pointer, m >= 128, k a multiple of 64, n >= 64, no A operation)");
+            cmd->record_error(UZU_ERROR_UNSUPPORTED, "dense_linear: bf16 activations need the tcgen05 form (bf16 weights, dense rows, a workspace pointer, m >= 128, k a multiple of 64, n >= 8, no A operation)");
             return;
         }
+        if (a.ldd == 0) a.ldd = a.n;
         encode_dense_umma(cmd, a);
         return;
     }
@@ -900,12 +901,12 @@ extern "C" void uzu_dense_linear_encode(uzu_command_buffer* cmd, const uzu_dense
         else by_ks(float{});
         return;
     }
-    if (a.pair_rows) {
-        cmd->record_error(UZU_ERROR_UNSUPPORTED, "dense_linear: the paired gated-unit epilogue covers passes of at most 8 rows");
-        return;
-    }
     if (!a.post_weight && !a.token_table && !a.streams && dense_umma_applicable(a)) {
         encode_dense_umma(cmd, a);
+        return;
+    }
+    if (a.pair_rows) {
+        cmd->record_error(UZU_ERROR_UNSUPPORTED, "dense_linear: the paired gated-unit epilogue covers passes of at most 8 rows and the tcgen05 form");
         return;
     }
     static const bool no_tensor128 = getenv("UZU_DENSE_NO_TENSOR128") != nullptr;     // A/B runs

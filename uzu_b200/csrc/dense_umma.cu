@@ -11,6 +11,10 @@
 //   warp 4, one lane: MMA ISSUER. Per K block 4 x tcgen05.mma.cta_group::1.kind::f16 (128 x 128 x 16) into 128 TMEM columns, then
 //     tcgen05.commit on the stage's `empty` barrier; after the last block a commit on the accumulator barrier.
 //   warps 0..3 again: EPILOGUE. tcgen05.ld 32 lanes x 32 columns, scale / factors / bias / gelu / accumulate, 16-byte stores (f32 or bf16).
+// Row groups (routed experts): grid z is the group, its compact rows [off[z], off[z+1]) use weight block z; the producers gather the activation
+// rows by the map as they copy them, CTAs past a group's end return at once.
+// Gated units (pair_rows): a CTA's 128 weight rows are 64 gate rows and the 64 up rows that belong to them, the epilogue reads both halves of
+// the accumulator and stores the finished unit of 64 features: the [gate | up] rows never go to memory.
 // Every barrier wait is bounded (about a second): a wait that runs out sets an error word, the CTA stops working, still meets at the
 // final barrier, frees its tensor memory and returns.
 #include "common.cuh"
@@ -26,7 +30,12 @@ struct DenseUmmaParams {
     const float* col_scale;    // optional [n]
     const float* bias;         // optional [n], added after scale / gate / col_scale
     const float* row_scale;    // optional [m]
+    const uint32_t* group_offsets;   // optional [groups + 1]
+    const uint32_t* rows_map;        // optional: the activation row of a compact row
+    uint64_t w_z_stride;
     uint32_t m, n, k, ldd, gate_ld, accumulate, d_op, d_bf16;
+    uint32_t pair_rows, glu_kind, glu_last_group;
+    float glu_limit, glu_limit_last, glu_alpha;
     float scale;
     uint32_t desc_hi, desc_lbo, k_step, idesc;
     unsigned int* error;
@@ -74,7 +83,31 @@ __device__ __forceinline__ void du_cp_async16(uint32_t dst_smem, const void* src
 }
 __device__ __forceinline__ uint32_t du_tile_off(uint32_t row, uint32_t ch) { return row * 128u + ((ch ^ (row & 7u)) << 4); }
 
-enum DuEpilogue : int { DuPlain = 0 /* scale, bias, accumulate */, DuGelu = 1 /* the exact gelu besides */, DuGeneral = 2 /* gate, row and column factors besides */ };
+enum DuEpilogue : int { DuPlain = 0 /* scale, bias, accumulate */, DuGelu = 1 /* the exact gelu besides */, DuGeneral = 2 /* gate, row and column factors besides */,
+                        DuPair = 3 /* the gated unit of the tile's two halves */ };
+
+__device__ __forceinline__ float du_unit(uint32_t kind, float g, float u, float limit, float alpha) {
+    if (kind == 0) {
+        g = fminf(g, limit);
+        return g * (1.0f / (1.0f + expf(-alpha * g))) * (fminf(fmaxf(u, -limit), limit) + 1.0f);
+    }
+    if (kind == 1) return g * (1.0f / (1.0f + expf(-g))) * u;
+    return 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
+}
+
+// 32 accumulator columns of this warp's 32 rows (one row per lane)
+__device__ __forceinline__ void du_tmem_load(uint32_t (&v)[32], uint32_t taddr) {
+    asm volatile(
+        "tcgen05.ld.sync.aligned.32x32b.x32.b32 "
+        "{%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31}, "
+        "[%32];"
+        : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]), "=r"(v[4]), "=r"(v[5]), "=r"(v[6]), "=r"(v[7]), "=r"(v[8]), "=r"(v[9]),
+          "=r"(v[10]), "=r"(v[11]), "=r"(v[12]), "=r"(v[13]), "=r"(v[14]), "=r"(v[15]), "=r"(v[16]), "=r"(v[17]), "=r"(v[18]),
+          "=r"(v[19]), "=r"(v[20]), "=r"(v[21]), "=r"(v[22]), "=r"(v[23]), "=r"(v[24]), "=r"(v[25]), "=r"(v[26]), "=r"(v[27]),
+          "=r"(v[28]), "=r"(v[29]), "=r"(v[30]), "=r"(v[31])
+        : "r"(taddr)
+        : "memory");
+}
 
 template <int EPI>
 __global__ void __launch_bounds__(DU_NP + 32, 1) dense_umma_kernel(const DenseUmmaParams p) {
@@ -83,7 +116,16 @@ __global__ void __launch_bounds__(DU_NP + 32, 1) dense_umma_kernel(const DenseUm
     __shared__ uint32_t tmem_slot;
     __shared__ uint32_t gave_up;
 
-    const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, z = blockIdx.z;
+    constexpr uint32_t kFeatures = EPI == DuPair ? 64u : 128u;        // output features of a CTA
+    const uint32_t n0 = blockIdx.x * kFeatures, m0 = blockIdx.y * 128u;
+    uint32_t row_begin = 0, rows = p.m;                               // the group's compact rows
+    if (p.group_offsets) {
+        pdl_wait();
+        row_begin = p.group_offsets[z];
+        rows = p.group_offsets[z + 1] - row_begin;
+        if (m0 >= rows) return;                                       // uniform over the CTA, before any barrier or tensor memory
+    }
     uint32_t smem_base = du_smem_u32(du_smem_raw);
     const uint32_t pad = (1024u - (smem_base & 1023u)) & 1023u;    // swizzle atoms sit on 1024-byte boundaries
     smem_base += pad;
@@ -110,7 +152,6 @@ __global__ void __launch_bounds__(DU_NP + 32, 1) dense_umma_kernel(const DenseUm
     __syncthreads();
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
     const uint32_t tmem_base = tmem_slot;
-    const uint32_t n0 = blockIdx.x * 128u, m0 = blockIdx.y * 128u;
     const uint32_t nkb = p.k >> 6;
     auto fail = [&](uint32_t code) {
         gave_up = 1;
@@ -120,18 +161,30 @@ __global__ void __launch_bounds__(DU_NP + 32, 1) dense_umma_kernel(const DenseUm
     if (tid < (uint32_t)DU_NP) {
         // ================================ producers ================================
         constexpr int PA = DU_STAGES - 2;                       // K blocks in flight ahead of the one being handed over
+        pdl_wait();
+        const __nv_bfloat16* wz = p.w + (size_t)z * p.w_z_stride;
+        // this thread's rows of the tiles: 8 activation rows and 8 weight rows, 16 apart; rows past the edge are zero-filled
+        uint32_t a_row[8];
+        uint32_t a_in = 0;
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            const uint32_t r = m0 + ((uint32_t)i * DU_NP + tid) / 8u;
+            const bool in = r < rows;
+            a_in |= (in ? 1u : 0u) << i;
+            a_row[i] = in ? (p.rows_map ? p.rows_map[row_begin + r] : row_begin + r) : 0u;
+        }
         auto issue = [&](uint32_t j, uint32_t stage) {
             const uint32_t st = smem_base + stage * DU_STAGE_BYTES;
 #pragma unroll
             for (int i = 0; i < 8; ++i) {
                 const uint32_t c = (uint32_t)i * DU_NP + tid, row = c >> 3, ch = c & 7u;
-                const bool a_ok = m0 + row < p.m, w_ok = n0 + row < p.n;     // rows past the edge are zero-filled
-                du_cp_async16(st + du_tile_off(row, ch), p.a + (size_t)(a_ok ? m0 + row : 0u) * p.k + (size_t)j * 64u + ch * 8u, a_ok ? 16u : 0u);
-                du_cp_async16(st + DU_TILE_BYTES + du_tile_off(row, ch), p.w + (size_t)(w_ok ? n0 + row : 0u) * p.k + (size_t)j * 64u + ch * 8u,
-                              w_ok ? 16u : 0u);
+                const uint32_t feature = n0 + (EPI == DuPair ? row & 63u : row);
+                const bool a_ok = (a_in >> i & 1u) != 0u, w_ok = feature < p.n;
+                const uint32_t w_row = w_ok ? (EPI == DuPair && row >= 64u ? p.pair_rows + feature : feature) : 0u;
+                du_cp_async16(st + du_tile_off(row, ch), p.a + (size_t)a_row[i] * p.k + (size_t)j * 64u + ch * 8u, a_ok ? 16u : 0u);
+                du_cp_async16(st + DU_TILE_BYTES + du_tile_off(row, ch), wz + (size_t)w_row * p.k + (size_t)j * 64u + ch * 8u, w_ok ? 16u : 0u);
             }
         };
-        pdl_wait();
         uint32_t a_stage = 0, a_parity = 1, c_stage = 0;
         bool ok = true;
         for (uint32_t t = 0; t < nkb + PA && ok; ++t) {
@@ -153,24 +206,16 @@ __global__ void __launch_bounds__(DU_NP + 32, 1) dense_umma_kernel(const DenseUm
         if (ok && !du_mbar_wait(accum_bar, 0)) { fail(2); ok = false; }
         if (ok) {
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-            const uint32_t row = m0 + warp * 32u + lane;
+            const uint32_t in_group = m0 + warp * 32u + lane, row = row_begin + in_group;
 #pragma unroll 1
-            for (uint32_t cb = 0; cb < 4u; ++cb) {
-                uint32_t v[32];
+            for (uint32_t cb = 0; cb < kFeatures / 32u; ++cb) {
+                uint32_t v[32], up[EPI == DuPair ? 32 : 1];
                 const uint32_t taddr = tmem_base + ((warp * 32u) << 16) + cb * 32u;
-                asm volatile(
-                    "tcgen05.ld.sync.aligned.32x32b.x32.b32 "
-                    "{%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31}, "
-                    "[%32];"
-                    : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]), "=r"(v[4]), "=r"(v[5]), "=r"(v[6]), "=r"(v[7]), "=r"(v[8]), "=r"(v[9]),
-                      "=r"(v[10]), "=r"(v[11]), "=r"(v[12]), "=r"(v[13]), "=r"(v[14]), "=r"(v[15]), "=r"(v[16]), "=r"(v[17]), "=r"(v[18]),
-                      "=r"(v[19]), "=r"(v[20]), "=r"(v[21]), "=r"(v[22]), "=r"(v[23]), "=r"(v[24]), "=r"(v[25]), "=r"(v[26]), "=r"(v[27]),
-                      "=r"(v[28]), "=r"(v[29]), "=r"(v[30]), "=r"(v[31])
-                    : "r"(taddr)
-                    : "memory");
+                du_tmem_load(v, taddr);
+                if constexpr (EPI == DuPair) du_tmem_load(up, taddr + 64u);
                 asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
                 const uint32_t col0 = n0 + cb * 32u;
-                if (row >= p.m || col0 >= p.n) continue;
+                if (in_group >= rows || col0 >= p.n) continue;
                 float* out = p.d + (size_t)row * p.ldd + col0;
                 __nv_bfloat16* out16 = reinterpret_cast<__nv_bfloat16*>(p.d) + (size_t)row * p.ldd + col0;
                 const float* gate = p.gate ? p.gate + (size_t)row * p.gate_ld + col0 : nullptr;
@@ -181,6 +226,10 @@ __global__ void __launch_bounds__(DU_NP + 32, 1) dense_umma_kernel(const DenseUm
 #pragma unroll
                 for (int j = 0; j < 32; ++j) {
                     float val = __uint_as_float(v[j]) * p.scale;
+                    if constexpr (EPI == DuPair) {
+                        const float limit = p.glu_last_group && z >= p.glu_last_group ? p.glu_limit_last : p.glu_limit;
+                        val = du_unit(p.glu_kind, val * rs, __uint_as_float(up[j]) * p.scale * rs, limit, p.glu_alpha);
+                    }
                     if constexpr (EPI == DuGeneral) {
                         if (whole || col0 + (uint32_t)j < p.n) {
                             if (p.row_scale) val *= rs;
@@ -299,12 +348,15 @@ __global__ void dense_cast_bf16_kernel(const float* a, uint32_t lda, __nv_bfloat
     *reinterpret_cast<uint2*>(out + idx) = o;
 }
 
-// Shapes the tensor-memory kernel takes: one plain product (no z-batches or row groups), bf16 weights, >= 128 rows, k a multiple
-// of 64, 16-byte aligned operands, and a bf16 workspace of m * k elements from the caller.
+// Shapes the tensor-memory kernel takes: bf16 weights, >= 128 rows (of a group, at most), k a multiple of 64, 16-byte aligned operands; one plain
+// product with a bf16 workspace of m * k elements from the caller, or row groups over activation rows that are bf16 already; plain or paired.
 bool dense_umma_applicable(const uzu_dense_linear_args& a) {
     static const bool off = getenv("UZU_DENSE_NO_UMMA") != nullptr;      // A/B runs
-    if (off || !a.workspace || a.weights_dt != UZU_DT_BF16 || a.batch != 1 || a.group_offsets || a.rows_map || a.pair_rows) return false;
-    if (a.m < 128 || a.k % 64u != 0 || a.n < 64) return false;
+    if (off || !a.workspace || a.weights_dt != UZU_DT_BF16) return false;
+    if (a.group_offsets ? !a.a_bf16 || a.w_z_stride % 8u != 0 : a.batch != 1 || a.rows_map) return false;
+    if (a.m < 128 || a.k % 64u != 0 || a.n < 8) return false;
+    if (a.pair_rows && (a.d_op || a.gate || a.col_scale || a.bias || a.accumulate || a.glu_kind > 2)) return false;
+    if (a.streams || a.post_weight || a.token_table || a.a_norm_weight) return false;
     if ((a.d & 15u) && (a.ldd ? a.ldd : a.n) % 8u == 0) return false;      // rows of whole 16-byte pieces are stored as such
     if (a.d_op && (a.gate || a.row_scale || a.col_scale)) return false;
     if ((a.a & 15u) || (a.w & 15u) || (a.workspace & 15u) || a.lda % 4u != 0) return false;
@@ -326,6 +378,11 @@ void encode_dense_umma(uzu_command_buffer* cmd, const uzu_dense_linear_args& a) 
     p.col_scale = (const float*)a.col_scale;
     p.bias = (const float*)a.bias;
     p.row_scale = (const float*)a.row_scale;
+    p.group_offsets = (const uint32_t*)a.group_offsets;
+    p.rows_map = (const uint32_t*)a.rows_map;
+    p.w_z_stride = a.w_z_stride;
+    p.pair_rows = a.pair_rows; p.glu_kind = a.glu_kind; p.glu_last_group = a.glu_last_group;
+    p.glu_limit = a.glu_limit; p.glu_limit_last = a.glu_limit_last; p.glu_alpha = a.glu_alpha;
     p.m = a.m; p.n = a.n; p.k = a.k; p.ldd = a.ldd; p.gate_ld = a.gate_ld; p.accumulate = a.accumulate; p.d_op = a.d_op; p.d_bf16 = a.d_bf16;
     p.scale = a.scale;
     // shared-memory matrix descriptor: start address >> 4 @ [0,14), LBO >> 4 @ [16,30), SBO >> 4 @ [32,46), version 1 @ [46,48), layout
@@ -341,10 +398,12 @@ void encode_dense_umma(uzu_command_buffer* cmd, const uzu_dense_linear_args& a) 
     constexpr size_t smem = (size_t)DU_STAGES * DU_STAGE_BYTES + 1024;
     auto go = [&](auto kernel, std::atomic<uint64_t>& opt_in) {
         opt_in_dynamic_smem(cmd, kernel, (int)smem, opt_in);
-        launch(cmd, "dense_umma_kernel", kernel, dim3((a.n + 127u) / 128u, (a.m + 127u) / 128u), dim3(DU_NP + 32), smem, p);
+        const uint32_t features = a.pair_rows ? 64u : 128u;
+        launch(cmd, "dense_umma_kernel", kernel, dim3((a.n + features - 1u) / features, (a.m + 127u) / 128u, a.batch), dim3(DU_NP + 32), smem, p);
     };
-    static std::atomic<uint64_t> opt_in[3];
-    if (a.gate || a.row_scale || a.col_scale) go(dense_umma_kernel<DuGeneral>, opt_in[2]);
+    static std::atomic<uint64_t> opt_in[4];
+    if (a.pair_rows) go(dense_umma_kernel<DuPair>, opt_in[3]);
+    else if (a.gate || a.row_scale || a.col_scale) go(dense_umma_kernel<DuGeneral>, opt_in[2]);
     else if (a.d_op == 1) go(dense_umma_kernel<DuGelu>, opt_in[1]);
     else go(dense_umma_kernel<DuPlain>, opt_in[0]);
 }

@@ -1495,10 +1495,10 @@ static void sublayer_input(uzu_engine* e, uzu_command_buffer* cmd, uzu_dense_lin
 // x += A . W^T: the sublayers' output projections add straight into the residual stream. With a sublayer gate the product is first
 // multiplied by scale[c] * sigmoid(logits[row, c] + bias[c]); the logits are columns [offset, offset + width) of a [rows, gate_ld] block.
 static void encode_into_residual(uzu_engine* e, uzu_command_buffer* cmd, const DenseMatrix& w, uint64_t a, uint32_t lda, uint32_t rows,
-                                 const SublayerGate* g = nullptr, uint64_t gate_block = 0, uint32_t gate_ld = 0, uint32_t a_op = 0) {
+                                 const SublayerGate* g = nullptr, uint64_t gate_block = 0, uint32_t gate_ld = 0, uint32_t a_op = 0, bool a_bf16 = false) {
     // (a sandwich layer's sublayer leaves its result in a scratch block: it goes through a norm of its own before it is added)
     uzu_dense_linear_args x = dense_args(e, w, a, rows, e->pb.redirect ? e->pb.sub_out.ptr() : e->pb.resid.ptr());
-    x.lda = lda; x.accumulate = e->pb.redirect ? 0 : 1; x.a_op = a_op;
+    x.lda = lda; x.accumulate = e->pb.redirect ? 0 : 1; x.a_op = a_op; x.a_bf16 = a_bf16 ? 1 : 0;
     sublayer_epilogue(e, x);
     if (g && g->present) {
         if (g->bias.b) { x.gate = gate_block + (uint64_t)g->offset * 4; x.gate_ld = gate_ld; x.gate_bias = g->bias.ptr(); }
@@ -1859,6 +1859,16 @@ static void encode_gated_mlp(uzu_engine* e, uzu_command_buffer* cmd, const Layer
         if (paired) { up.n = M.f; up.ldd = M.f; up.pair_rows = M.f; up.glu_limit = M.limit; up.glu_alpha = kGateSlope; up.glu_kind = unit_kind; }
         return up;
     };
+    // Long bf16 passes: the unit is the first product's epilogue and its rows stay in bf16, as the down projection's A rows.
+    auto unit_on_tcgen05 = [&](uzu_dense_linear_args& up, uzu_dense_linear_args dn) {
+        uzu_dense_linear_args x = up;
+        x.d = P.act.ptr(); x.n = M.f; x.ldd = M.f; x.pair_rows = M.f; x.d_bf16 = 1;
+        x.glu_limit = M.limit; x.glu_alpha = kGateSlope; x.glu_kind = unit_kind;
+        dn.a_bf16 = 1;
+        if (paired || !dense_umma_applicable(x) || !dense_umma_applicable(dn)) return false;
+        up = x;
+        return true;
+    };
     auto unit = [&](uint32_t rows) {
         uzu_glu_args ga{};
         ga.gate_up = P.gate_up.ptr(); ga.output = P.act.ptr(); ga.rows = rows; ga.f = M.f; ga.kind = unit_kind; ga.limit = M.limit; ga.alpha = kGateSlope;
@@ -1890,20 +1900,10 @@ static void encode_gated_mlp(uzu_engine* e, uzu_command_buffer* cmd, const Layer
     }
     if (M.kind == GatedMlp::Dense) {
         uzu_dense_linear_args up = gate_up_args();
+        const bool fused = unit_on_tcgen05(up, dense_args(e, M.down, P.act.ptr(), m, P.sub_out.ptr()));
         uzu_dense_linear_encode(cmd, &up);
-        if (!paired) {
-            // long passes keep the unit's rows in bf16, as the down projection's A rows
-            uzu_dense_linear_args dn = dense_args(e, M.down, P.act.ptr(), m, P.sub_out.ptr());
-            uzu_glu_args ga{};
-            ga.gate_up = P.gate_up.ptr(); ga.output = P.act.ptr(); ga.rows = m; ga.f = M.f; ga.kind = unit_kind; ga.limit = M.limit; ga.alpha = kGateSlope;
-            ga.output_bf16 = dn.a_bf16 = P.redirect && dense_umma_applicable(dn) ? 1 : 0;
-            uzu_glu_encode(cmd, &ga);
-            if (dn.a_bf16) {
-                uzu_dense_linear_encode(cmd, &dn);
-                return;
-            }
-        }
-        encode_into_residual(e, cmd, M.down, P.act.ptr(), M.f, m);
+        if (!paired && !fused) unit(m);
+        encode_into_residual(e, cmd, M.down, P.act.ptr(), M.f, m, nullptr, 0, 0, 0, fused);
         return;
     }
     // routed experts: expert-sorted (token, slot) pairs, grouped products over the pairs, weighted combine per token
@@ -1941,16 +1941,35 @@ static void encode_gated_mlp(uzu_engine* e, uzu_command_buffer* cmd, const Layer
         up.group_offsets = P.group_offsets.ptr(); up.rows_map = P.rows_map.ptr();
         if (shared_listed) { up.glu_last_group = M.experts; up.glu_limit_last = M.shared_limit; }
     }
+    auto down_args = [&](uint64_t d) {
+        uzu_dense_linear_args dn = dense_args(e, M.down, P.act.ptr(), m, d);
+        dn.lda = M.f;
+        if (grouped) {
+            dn.batch = lists; dn.w_z_stride = M.down.stride();
+            dn.group_offsets = P.group_offsets.ptr();
+        }
+        return dn;
+    };
+    // Long bf16 passes run the row groups on tcgen05 too, over bf16 copies of the activation rows (left by the norm, or made here).
+    bool fused = false;
+    if (grouped && !paired) {
+        uzu_dense_linear_args x = up;
+        x.a_bf16 = 1;
+        x.a = P.reads_residual && P.normed_bf16 ? P.normed.ptr() : P.operand_bf16.ptr();
+        fused = unit_on_tcgen05(x, down_args(P.pair_out.ptr()));
+        if (fused) {
+            if (x.a == P.operand_bf16.ptr()) uzu_rows_to_bf16_encode(cmd, h, W, x.a, m, W);
+            up = x;
+        }
+    } else if (!grouped) {
+        fused = unit_on_tcgen05(up, down_args(P.pair_out.ptr()));
+    }
     uzu_dense_linear_encode(cmd, &up);
-    if (!paired) unit(m * slots);
+    if (!paired && !fused) unit(m * slots);
     // ... and, when its weight already sits on its input and no sublayer gate follows, its down projection adds straight into the residual
     const bool direct = !grouped && M.weight_on_input && !L.mlp_gate.present;
-    uzu_dense_linear_args dn = dense_args(e, M.down, P.act.ptr(), m, direct ? P.resid.ptr() : P.pair_out.ptr());
-    dn.lda = M.f; dn.accumulate = direct ? 1 : 0;
-    if (grouped) {
-        dn.batch = lists; dn.w_z_stride = M.down.stride();
-        dn.group_offsets = P.group_offsets.ptr();
-    }
+    uzu_dense_linear_args dn = down_args(direct ? P.resid.ptr() : P.pair_out.ptr());
+    dn.accumulate = direct ? 1 : 0; dn.a_bf16 = fused ? 1 : 0;
     uzu_dense_linear_encode(cmd, &dn);
     if (direct) return;
     // the shared expert as plain products: its slices' [gate | up] rows lie back to back, so the unit sees m * slices rows of one slice each
@@ -1960,9 +1979,9 @@ static void encode_gated_mlp(uzu_engine* e, uzu_command_buffer* cmd, const Layer
         sx.w = M.gate_up.w.ptr() + (uint64_t)M.experts * M.gate_up.stride() * storage_size(e->store_dt);
         sx.n = M.shared * 2 * M.f; sx.ldd = sx.n; sx.lda = W;
         if (P.reads_residual) residual_input(e, cmd, sx);
-        uzu_dense_linear_encode(cmd, &sx);
         uzu_dense_linear_args sd = dense_args(e, M.shared_down, P.act.ptr(), m, P.redirect ? P.sub_out.ptr() : P.resid.ptr());
         sd.accumulate = P.redirect ? 0 : 1;
+        uzu_dense_linear_encode(cmd, &sx);
         uzu_glu_args ga{};
         ga.gate_up = P.gate_up.ptr(); ga.output = P.act.ptr(); ga.rows = m * M.shared; ga.f = M.f; ga.kind = unit_kind; ga.limit = M.shared_limit; ga.alpha = kGateSlope;
         ga.output_bf16 = sd.a_bf16 = dense_umma_applicable(sd) ? 1 : 0;
