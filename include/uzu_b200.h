@@ -776,6 +776,9 @@ typedef struct uzu_retention_args {
     uint64_t norm_out;                     /* optional f32 [rows, heads] */
     float query_scale;                     /* 0 = 1 */
     uint32_t reserved1;
+    uint64_t chunk_scratch;                /* optional f32 [heads, ceil(rows / 64), dim, vdim]: with it (not in the gated form), passes of >= 64 tokens with head
+                                              sizes that are multiples of 16 (dim <= 128, vdim <= 256) take chunks of 64 tokens at a time on the tensor pipe,
+                                              q, k and v rounded to bf16 there (states, decays and sums stay f32) */
 } uzu_retention_args;
 UZU_API void uzu_retention_encode(uzu_command_buffer* cmd, const uzu_retention_args* args);
 

@@ -416,19 +416,24 @@ class Memory:
         self.S0 = f32(self.rng, heads, dim, vdim, spread=start)
         self.bdecay, self.bstate = ctx.upload(self.decay), ctx.upload(self.S0)
 
-    def feed(self, proj):
+    def feed(self, proj, chunks=False):
         T = proj.shape[0]
         qn, vn = self.H * self.d, self.H * self.dv
         ld = proj.shape[1]
         bp, bo = self.ctx.upload(proj), self.ctx.upload(np.zeros((T, vn), np.float32))
         a = B.RetentionArgs(q=bp.ptr, k=bp.ptr + qn * 4, v=bp.ptr + 2 * qn * 4, decay=self.bdecay.ptr, state=self.bstate.ptr, out=bo.ptr, rows=T, heads=self.H, dim=self.d, vdim=self.dv,
                             q_stride=ld, k_stride=ld, v_stride=ld, out_stride=vn, key_scale=1.0, input_op=1)
+        if chunks:
+            scratch = self.ctx.upload(np.full(self.H * ((T + 63) // 64) * self.d * self.dv, np.nan, np.float32))
+            a.chunk_scratch = scratch.ptr
         run(self.ctx, "uzu_retention_encode", C.byref(a))
         return bo.numpy(np.float32, (T, self.H, self.dv))
 
-    def plain(self, proj):
+    def plain(self, proj, rounded=False):
         T, qn = proj.shape[0], self.H * self.d
         x = P.silu(t64(proj))
+        if rounded:
+            x = t64(bf16_exact(x.numpy()))
         return P.memory_scan(x[:, :qn].reshape(T, self.H, -1), x[:, qn:2 * qn].reshape(T, self.H, -1), x[:, 2 * qn:2 * qn + self.H * self.dv].reshape(T, self.H, -1),
                              t64(self.decay), t64(self.S0))
 
@@ -457,6 +462,29 @@ def test_lightning_attention_in_portions(ctx, heads, dim, vdim):
     close(M.bstate.numpy(np.float32, M.S0.shape), S.numpy(), 2e-5, "state after portions")
 
 
+@pytest.mark.parametrize("heads,dim,vdim", [(4, 128, 128), (2, 64, 64), (6, 32, 128), (3, 48, 16), (2, 16, 80), (1, 112, 192), (2, 96, 256), (1, 64, 48)])
+def test_lightning_attention_in_chunks(ctx, heads, dim, vdim):
+    """Long passes on the tensor pipe, cut anywhere (also passes too short for it between them), against the recurrence on the rounded inputs; the
+    inputs' rounding is the only one that shows."""
+    decay = [(0.3, 0.9, 0.999, 1.0, 0.97, 0.0)[h % 6] for h in range(heads)]
+    ld = heads * (2 * dim + vdim) + 8
+    for cuts in ([400], [64, 64], [65, 130, 64, 127], [100, 3, 1, 90, 30, 129]):
+        M = Memory(ctx, heads, dim, vdim, decay, seed=dim + vdim)
+        T = sum(cuts)
+        proj = f32(M.rng, T, ld)
+        proj[:, :heads * dim] = bf16_exact(proj[:, :heads * dim])
+        o, S = M.plain(proj, rounded=True)
+        got, at = [], 0
+        for c in cuts:
+            got.append(M.feed(proj[at:at + c], chunks=True))
+            at += c
+        short = any(c < 64 for c in cuts)                  # those passes do not round their inputs
+        for g, r, what in ((np.concatenate(got), o.numpy(), "outputs"), (M.bstate.numpy(np.float32, M.S0.shape), S.numpy(), "state")):
+            close(g, r, 8e-2 if short else 4e-3, f"{what}, cuts {cuts}")
+            # (a silu that lies at a rounding's border may round the other way: rare)
+            assert np.sqrt(((g - r) ** 2).mean() / (r ** 2).mean()) < (6e-3 if short else 1e-4), f"{what}, cuts {cuts}"
+
+
 def test_lightning_attention_recalls_a_far_write(ctx):
     """One key channel that a single early token writes and the last one reads, no decay: its value comes back exactly among hundreds of others."""
     heads, dim, vdim, T = 1, 64, 64, 700
@@ -470,6 +498,8 @@ def test_lightning_attention_recalls_a_far_write(ctx):
         v = proj[place, 2 * dim:]
         want = 400.0 * v / (1.0 + np.exp(-v))
         close(M.feed(proj)[T - 1, 0], want, 1e-5, f"write at {place}, prompt")
+        M = Memory(ctx, heads, dim, vdim, [1.0], seed=3, start=0.0)
+        close(M.feed(proj, chunks=True)[T - 1, 0], want, 1e-2, f"write at {place}, prompt in chunks")
         M = Memory(ctx, heads, dim, vdim, [1.0], seed=3, start=0.0)
         M.feed(proj[:T - 1])
         close(M.feed(proj[T - 1:])[0, 0], want, 1e-5, f"write at {place}, decoded")

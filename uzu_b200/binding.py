@@ -210,7 +210,7 @@ MinGruArgs = _struct("uzu_min_gru_args", [
 RetentionArgs = _struct("uzu_retention_args", [
     ("q", u64), ("k", u64), ("v", u64), ("decay", u64), ("state", u64), ("out", u64),
     ("rows", u32), ("heads", u32), ("dim", u32), ("vdim", u32), ("q_stride", u32), ("k_stride", u32), ("v_stride", u32), ("out_stride", u32),
-    ("key_scale", f32), ("input_op", u32), ("token_decay", u64), ("token_gain", u64), ("norm_out", u64), ("query_scale", f32), ("reserved1", u32)])
+    ("key_scale", f32), ("input_op", u32), ("token_decay", u64), ("token_gain", u64), ("norm_out", u64), ("query_scale", f32), ("reserved1", u32), ("chunk_scratch", u64)])
 
 ExpGatesArgs = _struct("uzu_exp_gates_args", [
     ("i_pre", u64), ("f_pre", u64), ("state", u64), ("token_decay", u64), ("token_gain", u64), ("floor", u64),

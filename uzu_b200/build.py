@@ -46,6 +46,7 @@ SOURCES = {
     "window_attention.cu": [],
     "window_attention_mma.cu": [],
     "linear_recurrence.cu": [],
+    "retention_chunked.cu": [],
     "gated_delta.cu": [],
     "engine.cu": [],
 }

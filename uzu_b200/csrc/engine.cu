@@ -414,6 +414,7 @@ struct RetentionLayer {         // retention: per head S <- decay S + (key_scale
     Buf norm_weight;            // f32 [heads * vdim] (joint_norm)
     bool joint_norm = false;
     bool silu_inputs = false;   // q, k and v pass a silu first
+    bool chunked = false;       // long bf16 passes run in chunks on the tensor pipe (q, k and v rounded to bf16)
     float key_scale = 1.0f;
     uint32_t heads = 0, dim = 0, vdim = 0;
     uint32_t q_offset = 0, k_offset = 0, v_offset = 0, gate_offset = 0;
@@ -611,6 +612,7 @@ struct uzu_engine {
         // Output-normed layers: the last sublayer's result waits in sub_out; whoever reads the residual next takes it in with its first launch
         // (a decode step's first product does it itself, from the rows at resid_at into the other of resid / resid2).
         Buf resid2;
+        Buf chunk_states;                                // retention in chunks: the states before every chunk of a pass
         uint64_t resid_at = 0;                           // where the residual's rows are (0: resid)
         const Norm* pending = nullptr;                   // the norm of the waiting result
         float pending_mult = 1.0f;

@@ -1119,6 +1119,7 @@ static void load_bonolorn_model(uzu_engine* e, const Json& cfg, const std::strin
         R.vdim = cfg_u32(rj, "vdim");
         R.share = (float)mc.at("right_scale").number();
         R.silu_inputs = true;
+        R.chunked = e->store_dt == UZU_DT_BF16;
         R.joint_norm = true;
         if (R.heads == 0 || R.dim == 0 || R.dim > 1024 || R.vdim == 0) throw std::runtime_error(p + "mix.right: heads / vdim must be positive, dim in 1..1024");
         {
@@ -1252,6 +1253,7 @@ static void create_parallel_block_scratch(uzu_engine* e) {
     const uint32_t W = e->model_dim;
     uint32_t proj = 1, lat = 1, wide = 1, query = 1, mixed = 1, gated = 1, gu = 1, act = 1, top = 1, experts = 1, partial = 1, kmax = e->model_dim;
     uint32_t proj2 = 1, tickets = 1, prompt_partial = 0, factor_heads = 0, expand_cols = 0, expand_rows = 0, shared_act = 0;
+    size_t chunk_states = 0;
     bool second_norm = false, sandwich = false, output_normed = false;
     for (const Layer& L : e->layers) {
         second_norm = second_norm || L.pre_mlp.present;
@@ -1301,6 +1303,7 @@ static void create_parallel_block_scratch(uzu_engine* e) {
                 wide = std::max(wide, L.rt.heads * L.rt.vdim);
                 gated = std::max(gated, L.rt.heads * L.rt.vdim);
                 kmax = std::max(kmax, L.rt.heads * L.rt.vdim);
+                if (L.rt.chunked && L.rt.dim % 16 == 0 && L.rt.vdim % 16 == 0) chunk_states = std::max<size_t>(chunk_states, (size_t)L.rt.heads * L.rt.dim * L.rt.vdim);
             }
             if (L.side_out.w.b) {          // both outputs lie side by side
                 mixed = std::max(mixed, L.side_out.cols);
@@ -1349,6 +1352,7 @@ static void create_parallel_block_scratch(uzu_engine* e) {
     P.normed = dev(R * W * 4);
     if (second_norm) P.normed2 = dev(R * W * 4);
     if (output_normed) P.resid2 = dev((size_t)W * 4);       // (one row: only the decode step's products move the residual)
+    if (chunk_states) P.chunk_states = dev(chunk_states * (MAX_ROWS / 64) * 4);
     if (sandwich || output_normed || e->streams) P.sub_out = dev(R * W * 4);
     if (factor_heads) P.token_factors = dev(4 * R * factor_heads * 4);
     if (expand_cols) {
@@ -1629,6 +1633,7 @@ static void encode_side_by_side(uzu_engine* e, uzu_command_buffer* cmd, const La
         ra.decay = R.decay.ptr(); ra.state = S.ssm_state.ptr(); ra.out = P.wide.ptr();
         ra.rows = m; ra.heads = R.heads; ra.dim = R.dim; ra.vdim = R.vdim; ra.q_stride = ra.k_stride = ra.v_stride = ld; ra.out_stride = rv;
         ra.key_scale = R.key_scale; ra.input_op = R.silu_inputs ? 1 : 0;
+        if (R.chunked) ra.chunk_scratch = P.chunk_states.ptr();
         uzu_retention_encode(cmd, &ra);
         uzu_head_norm_gate_args na{};
         na.x = P.wide.ptr(); na.gate = P.proj.ptr() + (uint64_t)R.gate_offset * 4; na.out = P.gated_mix.ptr();

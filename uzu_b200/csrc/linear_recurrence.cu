@@ -11,6 +11,7 @@
 //   registers. Tokens are taken in batches of RT_BATCH: q and k rows of the batch go to shared memory (requested one batch ahead), every
 //   thread runs the batch with no barrier, leaving per-warp partial outputs in shared memory, which are then added in warp order (a
 //   fixed order).
+//   Long passes with a scratch: in chunks of 64 tokens on the tensor pipe (retention_chunked.cu).
 //   Gated form (matrix memory with exponential gates): decay and input gain change from token to token and come from exp_gates_kernel,
 //   S_t = decay_t S_(t-1) + gain_t k_t v_t^T; the gain is folded into the staged value row. A normaliser n_t = decay_t n_(t-1) + gain_t k_t
 //   is the same recurrence with the value 1, so it rides along as one more state column whose output n_t . q_t goes to its own array.
@@ -259,6 +260,8 @@ __global__ void __launch_bounds__(PART == 32 ? 1024 : 512) retention_kernel(cons
         if ((uint32_t)i < cnt && col_ok) state[(size_t)(i0 + i) * vcols + col] = S[i];
 }
 
+bool encode_retention_chunked(uzu_command_buffer* cmd, const uzu_retention_args& a);      // retention_chunked.cu
+
 }  // namespace uzu
 
 extern "C" {
@@ -295,6 +298,7 @@ void uzu_retention_encode(uzu_command_buffer* cmd, const uzu_retention_args* a) 
     if (!b.k_stride) b.k_stride = b.heads * b.dim;
     if (!b.v_stride) b.v_stride = b.heads * b.vdim;
     if (!b.out_stride) b.out_stride = b.heads * b.vdim;
+    if (encode_retention_chunked(cmd, b)) return;
     // key channels per warp: about 16 warps per CTA whatever the key size, at most 32 warps
     int part = 4;
     while (part * 16 < (int)b.dim) part *= 2;
