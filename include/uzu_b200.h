@@ -881,6 +881,21 @@ typedef struct uzu_window_attention_args {
 } uzu_window_attention_args;
 UZU_API void uzu_window_attention_encode(uzu_command_buffer* cmd, const uzu_window_attention_args* args);
 
+/* Window attention and retention side by side, their two launches between the input and the output projection of a layer:
+ *   side_step:       uzu_window_attention_prepare and uzu_retention of the same ONE token (prep.rows = retention.rows = 1, not the gated form)
+ *   side_attention:  uzu_window_attention and the norm and gate of the retention's output (uzu_head_norm_gate, normalize = 1, no denominator); passes
+ *                    that run the attention on the tensor pipe take a launch each */
+typedef struct uzu_side_step_args {
+    uzu_window_attention_prepare_args prep;
+    uzu_retention_args retention;
+} uzu_side_step_args;
+UZU_API void uzu_side_step_encode(uzu_command_buffer* cmd, const uzu_side_step_args* args);
+typedef struct uzu_side_attention_args {
+    uzu_window_attention_args attention;
+    uzu_head_norm_gate_args norm;
+} uzu_side_attention_args;
+UZU_API void uzu_side_attention_encode(uzu_command_buffer* cmd, const uzu_side_attention_args* args);
+
 /* ---- Host engine (C++ mirror of the reference's backend-agnostic Rust host code) ---------- *
  * No Rust toolchain exists in the build image, so the layer above the kernels -- Engine /
  * LanguageModel / LanguageModelStream / Decoder / Transformer / TransformerLayer (engine/mod.rs:15-43,

@@ -517,6 +517,45 @@ def test_joint_norm_with_sigmoid_gate_and_share(ctx, rows, dim, pad):
     close(out[:, :dim], (P.unit_rms(t64(x), 1e-3) * t64(w) * torch.sigmoid(t64(gate[:, :dim])) * 1.2).numpy(), 1e-5)
 
 
+@pytest.mark.parametrize("heads,kv_heads,dim,vdim,r_heads,r_dim,r_vdim", [(4, 2, 16, 24, 3, 20, 40), (2, 1, 64, 64, 2, 128, 128), (3, 3, 7, 5, 1, 5, 7), (1, 1, 32, 16, 2, 300, 70)])
+@pytest.mark.parametrize("f32_cache", [True, False])
+def test_both_mixers_of_one_token_in_shared_launches(ctx, heads, kv_heads, dim, vdim, r_heads, r_dim, r_vdim, f32_cache):
+    """side_step and side_attention over 40 decoded tokens against the recurrence and the attention of the restatement; the two outputs lie side by side."""
+    T, window, eps = 40, 13, 1e-3
+    A = Attention(ctx, heads, kv_heads, dim, vdim, window, 1.2 / dim ** 0.5, f32_cache, positions=64, out_scale=0.8)
+    M = Memory(ctx, r_heads, r_dim, r_vdim, [(0.9, 1.0, 0.5)[h % 3] for h in range(r_heads)], seed=dim)
+    rng = np.random.default_rng(dim)
+    q, k, v, gate = attention_inputs(rng, T, heads, kv_heads, dim, vdim)
+    proj, rgate, w = f32(rng, T, r_heads * (2 * r_dim + r_vdim)), f32(rng, T, r_heads * r_vdim), f32(rng, r_heads * r_vdim)
+    o, S = M.plain(proj)
+    left = A.plain(q, k, v, gate).reshape(T, -1)
+    right = (P.unit_rms(o.reshape(T, -1), eps) * t64(w) * torch.sigmoid(t64(rgate)) * 1.3).numpy()
+    lo, ro = heads * vdim, r_heads * r_vdim
+    rows = np.concatenate([q.reshape(T, -1), k.reshape(T, -1), v.reshape(T, -1), gate, proj, rgate], axis=1).astype(np.float32)
+    offs = np.cumsum([0, heads * dim, kv_heads * dim, kv_heads * vdim, heads, r_heads * r_dim, r_heads * r_dim, ro, ro])
+    bq, bw, bo, bm = ctx.upload(np.zeros(heads * dim, np.float32)), ctx.upload(w), ctx.upload(np.zeros(ro, np.float32)), ctx.upload(np.zeros(lo + ro, np.float32))
+    parts, tickets = ctx.upload(np.zeros(heads * 5 * (vdim + 2), np.float32)), ctx.upload(np.zeros(heads, np.uint32))
+    dt = B.DT_F32 if f32_cache else B.DT_BF16
+    got = []
+    for t in range(T):
+        bp, bpos = ctx.upload(rows[t]), ctx.upload(np.array([t, 0], np.uint32))
+        at = lambda i: bp.ptr + int(offs[i]) * 4
+        common = dict(rows=1, heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, prefix=0 if t % 2 else t, cache_dt=dt, dynamic_position=bpos.ptr if t % 2 else 0)
+        pa = B.WindowAttentionPrepareArgs(q=at(0), k=at(1), v=at(2), q_scales=A.bqw.ptr, k_scales=A.bkw.ptr, query=bq.ptr, keys=A.keys.ptr, values=A.values.ptr, q_stride=rows.shape[1],
+                                          k_stride=rows.shape[1], v_stride=rows.shape[1], epsilon=eps, **common)
+        ra = B.RetentionArgs(q=at(4), k=at(5), v=at(6), decay=M.bdecay.ptr, state=M.bstate.ptr, out=bo.ptr, rows=1, heads=r_heads, dim=r_dim, vdim=r_vdim, key_scale=1.0, input_op=1)
+        run(ctx, "uzu_side_step_encode", C.byref(B.SideStepArgs(prep=pa, retention=ra)))
+        aa = B.WindowAttentionArgs(query=bq.ptr, keys=A.keys.ptr, values=A.values.ptr, out=bm.ptr, partials=parts.ptr, tickets=tickets.ptr, scale=A.scale, splits=t % 6, window=window,
+                                   head_gate=at(3), head_gate_stride=rows.shape[1], dist_slope=A.bslope.ptr, out_stride=lo + ro, out_scale=0.8, **common)
+        na = B.HeadNormGateArgs(x=bo.ptr, scales=bw.ptr, gate=at(7), out=bm.ptr + lo * 4, rows=1, heads=1, dim=ro, normalize=1, epsilon=eps, gate_op=0, out_scale=1.3)
+        run(ctx, "uzu_side_attention_encode", C.byref(B.SideAttentionArgs(attention=aa, norm=na)))
+        got.append(bm.numpy(np.float32, (lo + ro,)))
+    got = np.stack(got)
+    close(got[:, :lo], left, 3e-5 if f32_cache else 3e-3, "attention")
+    close(got[:, lo:], right, 5e-5, "memory")
+    close(M.bstate.numpy(np.float32, M.S0.shape), S.numpy(), 2e-5, "state")
+
+
 # ---- whole models ----------------------------------------------------------------------------------------------------------------------------
 def config_a():
     """widths and head sizes that fit no vector load, grouped heads, a layer without feed-forward, shared experts of one and of several slices with a

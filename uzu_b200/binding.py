@@ -238,6 +238,10 @@ WindowAttentionArgs = _struct("uzu_window_attention_args", [
     ("keep_first", u32), ("v_pairs", u32), ("scale", f32), ("softcap", f32), ("splits", u32), ("head_gate_stride", u32), ("sinks", u64), ("head_gate", u64),
     ("chunk", u32), ("out_stride", u32), ("dist_slope", u64), ("out_scale", f32), ("reserved", u32)])
 
+SideStepArgs = _struct("uzu_side_step_args", [("prep", WindowAttentionPrepareArgs), ("retention", RetentionArgs)])
+
+SideAttentionArgs = _struct("uzu_side_attention_args", [("attention", WindowAttentionArgs), ("norm", HeadNormGateArgs)])
+
 StreamMixArgs = _struct("uzu_stream_mix_args", [
     ("x", u64), ("y", u64), ("mix", u64), ("out", u64), ("read", u64), ("u", u64), ("weight", u64), ("output", u64), ("token_ids", u64), ("table", u64),
     ("rows", u32), ("n", u32), ("streams", u32), ("vocab", u32), ("table_dt", u32), ("output_bf16", u32), ("epsilon", f32), ("reserved", u32)])
@@ -255,7 +259,7 @@ GatedDeltaStepArgs = _struct("uzu_gated_delta_step_args", [
 
 MAIN_SLOT = 0xFFFFFFFF
 
-ABI_STRUCTS = [EmbeddingF32Args, GluArgs, StreamMixArgs, DeltaPrepareArgs, GatedDeltaArgs, GatedDeltaStepArgs, ExpGatesArgs, NormAddArgs, TokenGateArgs, MinGruArgs, RetentionArgs, WindowAttentionPrepareArgs, WindowAttentionArgs, TopkRouteArgs, RoutedCombineArgs, SigmoidAttentionPrepareArgs, SigmoidAttentionArgs, DenseLinearArgs, GroupRmsNormArgs, TableRouteArgs, GeneralDeltaArgs, HeadNormGateArgs, LatentPrepareArgs, LatentAttentionArgs,
+ABI_STRUCTS = [SideStepArgs, SideAttentionArgs, EmbeddingF32Args, GluArgs, StreamMixArgs, DeltaPrepareArgs, GatedDeltaArgs, GatedDeltaStepArgs, ExpGatesArgs, NormAddArgs, TokenGateArgs, MinGruArgs, RetentionArgs, WindowAttentionPrepareArgs, WindowAttentionArgs, TopkRouteArgs, RoutedCombineArgs, SigmoidAttentionPrepareArgs, SigmoidAttentionArgs, DenseLinearArgs, GroupRmsNormArgs, TableRouteArgs, GeneralDeltaArgs, HeadNormGateArgs, LatentPrepareArgs, LatentAttentionArgs,
                DeltaNetFusedUpdateArgs, QkNormConfig, AttentionPrepareNormArgs, FusedLinearArgs, RingParams, TrieNode, KvCopy, MatmulArgs, NormalizationArgs, QkvNormArgs, AttentionPrepareArgs, AttentionArgs,
                AttentionTwoPass2Args, KvCacheUpdateArgs, GatedActMulArgs, QuantizedEmbeddingLookupArgs, UnifiedSamplingArgs,
                DeltaNetConvUpdateArgs, DeltaNetUpdateArgs, EngineOptions, SamplingMethod, ModelInfo, TpAllGatherArgs]
@@ -290,7 +294,7 @@ uzu_silu_glu_encode uzu_topk_route_encode uzu_routed_combine_gated_encode uzu_si
 uzu_engine_slot_acquire uzu_engine_slot_release uzu_engine_forward_rows uzu_engine_debug_layer_outputs uzu_debug_dense_umma_error
 uzu_min_gru_encode uzu_retention_encode uzu_window_attention_prepare_encode uzu_window_attention_encode
 uzu_exp_gates_encode uzu_norm_add_encode uzu_token_gate_encode uzu_embedding_f32_scaled_encode uzu_rows_to_bf16_encode
-uzu_embedding_f32_position_encode uzu_glu_encode uzu_stream_mix_encode uzu_delta_prepare_encode uzu_gated_delta_encode uzu_gated_delta_step_encode""".split()
+uzu_side_step_encode uzu_side_attention_encode uzu_embedding_f32_position_encode uzu_glu_encode uzu_stream_mix_encode uzu_delta_prepare_encode uzu_gated_delta_encode uzu_gated_delta_step_encode""".split()
 
 _lib = None
 
@@ -455,6 +459,8 @@ def load() -> C.CDLL:
         "uzu_rows_to_bf16_encode": (None, [vp, u64, u32, u64, u32, u32]),
         "uzu_embedding_f32_scaled_encode": (None, [vp, u64, u64, u32, u64, u32, u32, u32, f32]),
         "uzu_embedding_f32_position_encode": (None, [vp, C.POINTER(EmbeddingF32Args)]),
+        "uzu_side_step_encode": (None, [vp, C.POINTER(SideStepArgs)]),
+        "uzu_side_attention_encode": (None, [vp, C.POINTER(SideAttentionArgs)]),
         "uzu_glu_encode": (None, [vp, C.POINTER(GluArgs)]),
         "uzu_engine_slot_acquire": (C.c_int, [vp, C.POINTER(u32)]),
         "uzu_engine_slot_release": (C.c_int, [vp, u32]),

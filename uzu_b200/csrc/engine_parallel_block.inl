@@ -1581,11 +1581,14 @@ static void encode_side_by_side(uzu_engine* e, uzu_command_buffer* cmd, const La
         if (L.side_in_bias.b) x.bias = L.side_in_bias.ptr();
         uzu_dense_linear_encode(cmd, &x);
     }
+    uzu_window_attention_prepare_args pa{};
+    uzu_window_attention_args aa{};
+    uzu_retention_args ra{};
+    uzu_head_norm_gate_args na{};
     if (L.has_window_attention()) {
         const WindowAttentionLayer& A = L.wa;
         const uint64_t vcos = A.value_rope_index >= 0 ? e->rope_cos[A.value_rope_index].ptr() : 0, vsin = A.value_rope_index >= 0 ? e->rope_sin[A.value_rope_index].ptr() : 0;
         const uint32_t v_pairs = A.value_rope_index >= 0 ? A.vdim / 2 : 0;
-        uzu_window_attention_prepare_args pa{};
         pa.q = P.proj.ptr() + (uint64_t)A.q_offset * 4; pa.k = P.proj.ptr() + (uint64_t)A.k_offset * 4; pa.v = P.proj.ptr() + (uint64_t)A.v_offset * 4;
         pa.q_scales = A.q_norm.ptr(); pa.k_scales = A.k_norm.ptr(); pa.query = P.query.ptr(); pa.keys = S.keys; pa.values = S.values;
         if (A.rope_index >= 0) {
@@ -1596,8 +1599,6 @@ static void encode_side_by_side(uzu_engine* e, uzu_command_buffer* cmd, const La
         pa.rows = m; pa.heads = A.heads; pa.kv_heads = A.kv_heads; pa.dim = A.dim; pa.vdim = A.vdim;
         pa.q_stride = pa.k_stride = pa.v_stride = ld; pa.prefix = S.length; pa.cache_dt = e->store_dt; pa.epsilon = e->norm_eps;
         pa.rot_halves = A.rot_halves ? 1 : 0; pa.unit_rms = A.unit_rms ? 1 : 0;
-        uzu_window_attention_prepare_encode(cmd, &pa);
-        uzu_window_attention_args aa{};
         aa.query = P.query.ptr(); aa.keys = S.keys; aa.values = S.values; aa.out = P.mixed.ptr(); aa.dynamic_position = dyn;
         aa.head_temp = A.head_temp.ptr(); aa.v_cosines = vcos; aa.v_sines = vsin; aa.v_pairs = v_pairs;
         aa.rows = m; aa.heads = A.heads; aa.kv_heads = A.kv_heads; aa.dim = A.dim; aa.vdim = A.vdim; aa.prefix = S.length; aa.cache_dt = e->store_dt;
@@ -1616,38 +1617,54 @@ static void encode_side_by_side(uzu_engine* e, uzu_command_buffer* cmd, const La
             aa.partials = P.attn_partial.ptr(); aa.tickets = P.attn_tickets.ptr();
             if (aa.splits < 2 || m > kSplitRows) aa.splits = 1;
         }
-        uzu_window_attention_encode(cmd, &aa);
-        if (!L.side_out.w.b) {
-            uzu_dense_linear_args x = dense_args(e, A.out, P.mixed.ptr(), m, P.redirect ? P.sub_out.ptr() : P.resid.ptr());
-            x.lda = A.heads * A.vdim; x.accumulate = P.redirect ? 0 : 1; x.scale = A.share;
-            if (A.out_bias.b) x.bias = A.out_bias.ptr();
-            sublayer_epilogue(e, x);
-            uzu_dense_linear_encode(cmd, &x);
-        }
     }
     if (L.has_retention()) {
         const RetentionLayer& R = L.rt;
         const uint32_t rv = R.heads * R.vdim;
-        uzu_retention_args ra{};
         ra.q = P.proj.ptr() + (uint64_t)R.q_offset * 4; ra.k = P.proj.ptr() + (uint64_t)R.k_offset * 4; ra.v = P.proj.ptr() + (uint64_t)R.v_offset * 4;
         ra.decay = R.decay.ptr(); ra.state = S.ssm_state.ptr(); ra.out = P.wide.ptr();
         ra.rows = m; ra.heads = R.heads; ra.dim = R.dim; ra.vdim = R.vdim; ra.q_stride = ra.k_stride = ra.v_stride = ld; ra.out_stride = rv;
         ra.key_scale = R.key_scale; ra.input_op = R.silu_inputs ? 1 : 0;
         if (R.chunked) ra.chunk_scratch = P.chunk_states.ptr();
-        uzu_retention_encode(cmd, &ra);
-        uzu_head_norm_gate_args na{};
         na.x = P.wide.ptr(); na.gate = P.proj.ptr() + (uint64_t)R.gate_offset * 4; na.out = P.gated_mix.ptr();
         na.rows = m; na.heads = R.heads; na.dim = R.vdim; na.x_stride = rv; na.gate_stride = ld; na.out_stride = rv; na.normalize = 1;
         na.epsilon = e->norm_eps; na.gate_op = 1;
         if (R.joint_norm) { na.heads = 1; na.dim = rv; na.scales = R.norm_weight.ptr(); na.gate_op = 0; }
         if (L.side_out.w.b) { na.out = P.mixed.ptr() + (uint64_t)L.wa.heads * L.wa.vdim * 4; na.out_stride = L.side_out.cols; na.out_scale = R.share; }
-        uzu_head_norm_gate_encode(cmd, &na);
-        if (L.side_out.w.b) {
-            encode_into_residual(e, cmd, L.side_out, P.mixed.ptr(), L.side_out.cols, m);
-            return;
-        }
+    }
+    const bool both = L.has_window_attention() && L.has_retention();
+    if (both && m == 1) {
+        uzu_side_step_args sa{};
+        sa.prep = pa; sa.retention = ra;
+        uzu_side_step_encode(cmd, &sa);
+    } else {
+        if (L.has_window_attention()) uzu_window_attention_prepare_encode(cmd, &pa);
+        if (L.has_retention()) uzu_retention_encode(cmd, &ra);
+    }
+    if (both) {
+        uzu_side_attention_args sa{};
+        sa.attention = aa; sa.norm = na;
+        uzu_side_attention_encode(cmd, &sa);
+    } else {
+        if (L.has_window_attention()) uzu_window_attention_encode(cmd, &aa);
+        if (L.has_retention()) uzu_head_norm_gate_encode(cmd, &na);
+    }
+    if (L.side_out.w.b) {
+        encode_into_residual(e, cmd, L.side_out, P.mixed.ptr(), L.side_out.cols, m);
+        return;
+    }
+    if (L.has_window_attention()) {
+        const WindowAttentionLayer& A = L.wa;
+        uzu_dense_linear_args x = dense_args(e, A.out, P.mixed.ptr(), m, P.redirect ? P.sub_out.ptr() : P.resid.ptr());
+        x.lda = A.heads * A.vdim; x.accumulate = P.redirect ? 0 : 1; x.scale = A.share;
+        if (A.out_bias.b) x.bias = A.out_bias.ptr();
+        sublayer_epilogue(e, x);
+        uzu_dense_linear_encode(cmd, &x);
+    }
+    if (L.has_retention()) {
+        const RetentionLayer& R = L.rt;
         uzu_dense_linear_args x = dense_args(e, R.out, P.gated_mix.ptr(), m, P.redirect ? P.sub_out.ptr() : P.resid.ptr());
-        x.lda = rv; x.accumulate = (P.redirect && !L.has_window_attention()) ? 0 : 1; x.scale = R.share;       // the second of two mixers adds to the first
+        x.lda = R.heads * R.vdim; x.accumulate = (P.redirect && !L.has_window_attention()) ? 0 : 1; x.scale = R.share;       // the second of two mixers adds to the first
         if (!L.has_window_attention()) sublayer_epilogue(e, x);
         uzu_dense_linear_encode(cmd, &x);
     }

@@ -948,7 +948,8 @@ void uzu_topk_route_encode(uzu_command_buffer* cmd, const uzu_topk_route_args* a
         return;
     }
     opt_in_dynamic_smem(cmd, topk_route_kernel<0>, (int)ROUTE_SMEM, done[0]);
-    launch(cmd, "topk_route_kernel", topk_route_kernel<0>, dim3(1), dim3(1024), smem, *a);
+    const uint32_t warps = std::min(32u, std::max(2u, a->rows));        // few rows: a small CTA, its barriers meet sooner
+    launch(cmd, "topk_route_kernel", topk_route_kernel<0>, dim3(1), dim3(32 * warps), smem, *a);
 }
 
 void uzu_routed_combine_gated_encode(uzu_command_buffer* cmd, const uzu_routed_combine_args* a) {

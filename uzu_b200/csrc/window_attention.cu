@@ -103,12 +103,8 @@ __device__ __forceinline__ Visible wa_visible(uint32_t p, uint32_t window, uint3
 
 // a warp per (token, unit): units [0, heads) queries, [heads, heads + kv_heads) keys, then values
 template <typename T>
-__global__ void __launch_bounds__(128) window_attention_prepare_kernel(const uzu_window_attention_prepare_args a) {
-    pdl_launch_dependents();
-    pdl_wait();
-    const uint32_t lane = threadIdx.x & 31;
+__device__ __forceinline__ void wa_prepare_unit(const uzu_window_attention_prepare_args& a, uint32_t item, uint32_t lane) {
     const uint32_t units = a.heads + 2 * a.kv_heads;
-    const uint32_t item = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
     if (item >= a.rows * units) return;
     const uint32_t t = item / units, unit = item % units;
     const uint32_t prefix = a.dynamic_position ? *reinterpret_cast<const uint32_t*>(a.dynamic_position) : a.prefix;
@@ -139,13 +135,65 @@ __global__ void __launch_bounds__(128) window_attention_prepare_kernel(const uzu
     }
 }
 
+template <typename T>
+__global__ void __launch_bounds__(128) window_attention_prepare_kernel(const uzu_window_attention_prepare_args a) {
+    pdl_launch_dependents();
+    pdl_wait();
+    wa_prepare_unit<T>(a, blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), threadIdx.x & 31);
+}
+
+// One token of a layer that holds both mixers: the first CTAs take the retention (32 value columns of one head each: 8 warps share the key
+// channels, their partial outputs are added in warp order), the others prepare the attention (a warp per unit).
+constexpr int SS_PART = 16;     // key channels of a warp in flight
+template <typename T>
+__global__ void __launch_bounds__(256) side_step_kernel(const uzu_side_step_args s, uint32_t retention_ctas) {
+    pdl_launch_dependents();
+    pdl_wait();
+    __shared__ float part[8][32];
+    const uint32_t lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    if (blockIdx.x >= retention_ctas) {
+        wa_prepare_unit<T>(s.prep, (blockIdx.x - retention_ctas) * 8 + warp, lane);
+        return;
+    }
+    const uzu_retention_args& a = s.retention;
+    const uint32_t tiles = (a.vdim + 31) / 32, head = blockIdx.x / tiles, col = (blockIdx.x - head * tiles) * 32 + lane;
+    const bool ok = col < a.vdim;
+    const float* q = reinterpret_cast<const float*>(a.q) + (size_t)head * a.dim;
+    const float* k = reinterpret_cast<const float*>(a.k) + (size_t)head * a.dim;
+    float* state = reinterpret_cast<float*>(a.state) + (size_t)head * a.dim * a.vdim + col;
+    auto input = [&](float x) { return a.input_op == 1 ? x * (1.0f / (1.0f + expf(-x))) : x; };
+    const float decay = reinterpret_cast<const float*>(a.decay)[head];
+    const float v = ok ? input(reinterpret_cast<const float*>(a.v)[(size_t)head * a.vdim + col]) : 0.0f;
+    float o = 0.0f;
+    for (uint32_t c0 = warp * SS_PART; c0 < a.dim; c0 += 8 * SS_PART) {
+        // lane i forms channel c0 + i of q and k once for the warp
+        const uint32_t mine = c0 + (lane & (SS_PART - 1));
+        const float qv = mine < a.dim ? input(q[mine]) : 0.0f, kv = mine < a.dim ? input(k[mine]) * a.key_scale : 0.0f;
+        float S[SS_PART];
+#pragma unroll
+        for (int i = 0; i < SS_PART; ++i) S[i] = (ok && c0 + i < a.dim) ? state[(size_t)(c0 + i) * a.vdim] : 0.0f;
+#pragma unroll
+        for (int i = 0; i < SS_PART; ++i) {
+            const float next = fmaf(__shfl_sync(0xffffffffu, kv, i), v, decay * S[i]);
+            o = fmaf(next, __shfl_sync(0xffffffffu, qv, i), o);
+            if (ok && c0 + i < a.dim) state[(size_t)(c0 + i) * a.vdim] = next;
+        }
+    }
+    part[warp][lane] = o;
+    __syncthreads();
+    if (warp == 0 && ok) {
+        float sum = 0.0f;
+#pragma unroll
+        for (int w = 0; w < 8; ++w) sum += part[w][lane];
+        reinterpret_cast<float*>(a.out)[(size_t)head * a.vdim + col] = sum * (a.query_scale != 0.0f ? a.query_scale : 1.0f);
+    }
+}
+
 constexpr int WA_WARPS = 4, WA_TILE = 16, WA_UNROLL = 4, WA_MAX_SPLITS = 128;
 
 // WPL = words of a head's key / value row per lane (the larger of the two)
 template <typename T, int EPW, int WPL>
-__global__ void __launch_bounds__(WA_WARPS * 32) window_attention_kernel(const uzu_window_attention_args a) {
-    pdl_launch_dependents();
-    pdl_wait();
+__device__ __forceinline__ void window_attention_body(const uzu_window_attention_args& a) {
     extern __shared__ float wa_smem[];          // [WA_WARPS][vdim] partial sums, then [vdim] the head's result
     __shared__ float warp_m[WA_WARPS], warp_l[WA_WARPS];
     __shared__ uint32_t is_last;
@@ -336,6 +384,51 @@ __global__ void __launch_bounds__(WA_WARPS * 32) window_attention_kernel(const u
     }
 }
 
+template <typename T, int EPW, int WPL>
+__global__ void __launch_bounds__(WA_WARPS * 32) window_attention_kernel(const uzu_window_attention_args a) {
+    pdl_launch_dependents();
+    pdl_wait();
+    window_attention_body<T, EPW, WPL>(a);
+}
+
+// ... and, in the CTAs behind the query heads', the norm and gate of another mixer's finished output (a CTA per row and norm head)
+template <typename T, int EPW, int WPL>
+__global__ void __launch_bounds__(WA_WARPS * 32) side_attention_kernel(const uzu_side_attention_args s) {
+    pdl_launch_dependents();
+    pdl_wait();
+    if (blockIdx.y < s.attention.heads) {
+        window_attention_body<T, EPW, WPL>(s.attention);
+        return;
+    }
+    if (blockIdx.z) return;
+    __shared__ float red[32];
+    const uzu_head_norm_gate_args& a = s.norm;
+    const uint32_t row = blockIdx.x, h = blockIdx.y - s.attention.heads;
+    const float* x = reinterpret_cast<const float*>(a.x) + (size_t)row * a.x_stride + (size_t)h * a.dim;
+    const float* gate = a.gate ? reinterpret_cast<const float*>(a.gate) + (size_t)row * a.gate_stride + (size_t)h * a.dim : nullptr;
+    const float* sc = a.scales ? reinterpret_cast<const float*>(a.scales) + (size_t)h * a.dim : nullptr;
+    float* out = reinterpret_cast<float*>(a.out) + (size_t)row * a.out_stride + (size_t)h * a.dim;
+    constexpr int KEEP = 16;          // elements of a thread that stay in registers, their gates and weights requested with them
+    float v[KEEP], w[KEEP], ss = 0.0f;
+    auto act = [&](float z) { const float p = 1.0f / (1.0f + expf(-z)); return a.gate_op == 1 ? z * p : p; };
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+        const uint32_t i = threadIdx.x + j * blockDim.x;
+        v[j] = i < a.dim ? x[i] : 0.0f;
+        w[j] = i < a.dim ? (gate ? act(gate[i]) : 1.0f) * (sc ? sc[i] : 1.0f) : 0.0f;
+    }
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) ss = fmaf(v[j], v[j], ss);
+    for (uint32_t i = threadIdx.x + KEEP * blockDim.x; i < a.dim; i += blockDim.x) ss = fmaf(x[i], x[i], ss);
+    const float inv = (a.out_scale != 0.0f ? a.out_scale : 1.0f) / sqrtf(block_sum(ss, red) / (float)a.dim + a.epsilon);
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+        const uint32_t i = threadIdx.x + j * blockDim.x;
+        if (i < a.dim) out[i] = v[j] * inv * w[j];
+    }
+    for (uint32_t i = threadIdx.x + KEEP * blockDim.x; i < a.dim; i += blockDim.x) out[i] = x[i] * inv * (gate ? act(gate[i]) : 1.0f) * (sc ? sc[i] : 1.0f);
+}
+
 bool encode_window_attention_mma(uzu_command_buffer* cmd, const uzu_window_attention_args& a);     // window_attention_mma.cu
 
 }  // namespace uzu
@@ -363,7 +456,35 @@ void uzu_window_attention_prepare_encode(uzu_command_buffer* cmd, const uzu_wind
         launch(cmd, "window_attention_prepare_kernel", window_attention_prepare_kernel<__nv_bfloat16>, dim3((items + 3) / 4), dim3(128), 0, b);
 }
 
-void uzu_window_attention_encode(uzu_command_buffer* cmd, const uzu_window_attention_args* a) {
+static void encode_attention(uzu_command_buffer* cmd, const uzu_window_attention_args* a, const uzu_head_norm_gate_args* norm);
+
+void uzu_window_attention_encode(uzu_command_buffer* cmd, const uzu_window_attention_args* a) { encode_attention(cmd, a, nullptr); }
+
+void uzu_side_attention_encode(uzu_command_buffer* cmd, const uzu_side_attention_args* a) {
+    if (!a->norm.normalize || a->norm.denom || a->norm.rows != a->attention.rows || a->norm.heads == 0 || a->norm.dim == 0 || !a->norm.x || !a->norm.out) {
+        cmd->record_error(UZU_ERROR_INVALID_ARGUMENT, "side_attention: the norm must be of the same rows, with its operands and without a denominator");
+        return;
+    }
+    encode_attention(cmd, &a->attention, &a->norm);
+}
+
+void uzu_side_step_encode(uzu_command_buffer* cmd, const uzu_side_step_args* a) {
+    if (!encodable(cmd, "side_step")) return;
+    const uzu_window_attention_prepare_args& p = a->prep;
+    const uzu_retention_args& r = a->retention;
+    if (p.rows != 1 || r.rows != 1 || !p.q || !p.k || !p.v || !p.query || !p.keys || !p.values || p.heads == 0 || p.kv_heads == 0 || p.dim == 0 || p.vdim == 0 ||
+        (p.cache_dt != UZU_DT_BF16 && p.cache_dt != UZU_DT_F32) || 2 * p.rot_pairs > p.dim || 2 * p.v_pairs > p.vdim || (p.rot_pairs && (!p.cosines || !p.sines)) ||
+        (p.v_pairs && (!p.v_cosines || !p.v_sines)) || !r.q || !r.k || !r.v || !r.decay || !r.state || !r.out || r.heads == 0 || r.dim == 0 || r.vdim == 0 ||
+        r.token_decay || r.norm_out || r.input_op > 1) {
+        cmd->record_error(UZU_ERROR_INVALID_ARGUMENT, "side_step: one token, all operands of both mixers, one decay per head");
+        return;
+    }
+    const uint32_t ret = r.heads * ((r.vdim + 31) / 32), units = p.heads + 2 * p.kv_heads;
+    if (p.cache_dt == UZU_DT_F32) launch(cmd, "side_step_kernel", side_step_kernel<float>, dim3(ret + (units + 7) / 8), dim3(256), 0, *a, ret);
+    else launch(cmd, "side_step_kernel", side_step_kernel<__nv_bfloat16>, dim3(ret + (units + 7) / 8), dim3(256), 0, *a, ret);
+}
+
+static void encode_attention(uzu_command_buffer* cmd, const uzu_window_attention_args* a, const uzu_head_norm_gate_args* norm) {
     if (!encodable(cmd, "window_attention")) return;
     if (!a->query || !a->keys || !a->values || !a->out || a->heads == 0 || a->kv_heads == 0 || a->heads % a->kv_heads || a->dim == 0 || a->vdim == 0 ||
         a->dim > 512 || a->vdim > 512 || (a->cache_dt != UZU_DT_BF16 && a->cache_dt != UZU_DT_F32) || 2 * a->v_pairs > a->vdim ||
@@ -377,25 +498,38 @@ void uzu_window_attention_encode(uzu_command_buffer* cmd, const uzu_window_atten
         cmd->record_error(UZU_ERROR_INVALID_ARGUMENT, "window_attention: key splits need the partials and tickets scratch");
         return;
     }
-    if (splits == 1 && encode_window_attention_mma(cmd, *a)) return;
+    if (splits == 1 && encode_window_attention_mma(cmd, *a)) {
+        if (norm) uzu_head_norm_gate_encode(cmd, norm);
+        return;
+    }
     const bool f32 = a->cache_dt == UZU_DT_F32;
     // bf16 rows of even head sizes are read two elements per word
     const bool pairs = !f32 && a->dim % 2 == 0 && a->vdim % 2 == 0;
     const uint32_t epw = pairs ? 2 : 1;
     const uint32_t words = (std::max(a->dim, a->vdim) + epw - 1) / epw;
     const uint32_t wpl = (words + 31) / 32;
-    const dim3 grid(a->rows, a->heads, splits), block(WA_WARPS * 32);
+    const dim3 grid(a->rows, a->heads + (norm ? norm->heads : 0u), splits), block(WA_WARPS * 32);
     const size_t smem = (size_t)(WA_WARPS + 1) * a->vdim * sizeof(float);
-    auto go = [&](auto kernel) { launch(cmd, "window_attention_kernel", kernel, grid, block, smem, *a); };
+    uzu_side_attention_args both{};
+    if (norm) {
+        both.attention = *a; both.norm = *norm;
+        if (!both.norm.x_stride) both.norm.x_stride = norm->heads * norm->dim;
+        if (!both.norm.gate_stride) both.norm.gate_stride = norm->heads * norm->dim;
+        if (!both.norm.out_stride) both.norm.out_stride = norm->heads * norm->dim;
+    }
+    auto go = [&](auto kernel, auto with_norm) {
+        if (norm) launch(cmd, "side_attention_kernel", with_norm, grid, block, smem, both);
+        else launch(cmd, "window_attention_kernel", kernel, grid, block, smem, *a);
+    };
     auto by_wpl = [&](auto tw, auto epw_c) {
         using T = decltype(tw);
         constexpr int E = decltype(epw_c)::value;
         switch (wpl) {
-            case 1: go(window_attention_kernel<T, E, 1>); break;
-            case 2: go(window_attention_kernel<T, E, 2>); break;
-            case 3: case 4: go(window_attention_kernel<T, E, 4>); break;
-            case 5: case 6: case 7: case 8: go(window_attention_kernel<T, E, 8>); break;
-            default: go(window_attention_kernel<T, E, 16>); break;
+            case 1: go(window_attention_kernel<T, E, 1>, side_attention_kernel<T, E, 1>); break;
+            case 2: go(window_attention_kernel<T, E, 2>, side_attention_kernel<T, E, 2>); break;
+            case 3: case 4: go(window_attention_kernel<T, E, 4>, side_attention_kernel<T, E, 4>); break;
+            case 5: case 6: case 7: case 8: go(window_attention_kernel<T, E, 8>, side_attention_kernel<T, E, 8>); break;
+            default: go(window_attention_kernel<T, E, 16>, side_attention_kernel<T, E, 16>); break;
         }
     };
     if (f32) by_wpl(float{}, std::integral_constant<int, 1>{});
