@@ -88,7 +88,7 @@ def test_embedding_adds_the_sinusoidal_position(ctx, n, prefix, dynamic):
     np.testing.assert_allclose(bo.numpy(np.float32, (rows, n)), rows_ref, rtol=1e-6)
 
 
-@pytest.mark.parametrize("rows,n", [(1, 7), (5, 90), (3, 2500)])
+@pytest.mark.parametrize("rows,n", [(1, 7), (5, 90), (3, 2500), (2, 64), (7, 1028), (2, 4096), (2, 4100)])
 def test_residual_takes_the_normed_result_in_and_leaves_bf16_rows(ctx, rows, n):
     rng = np.random.default_rng(n)
     y, res, w = f32(rng, rows, n) + 4.0, f32(rng, rows, n), f32(rng, n)
@@ -98,6 +98,12 @@ def test_residual_takes_the_normed_result_in_and_leaves_bf16_rows(ctx, rows, n):
     got = br.numpy(np.float32, (rows, n))
     close(got, (t64(res) + 0.7 * P.layer_norm(t64(y), t64(w), 1e-3)).numpy(), 1e-5, "residual")
     np.testing.assert_array_equal(bo.numpy(np.uint16, (rows, n)), bf16_bits(got))
+    b = f32(rng, n)
+    bb, bf = ctx.upload(b), ctx.upload(np.zeros((rows, n), np.float32))
+    for kind in (0, 2):                                 # without a residual, with a bias
+        run(ctx, "uzu_norm_add_encode", C.byref(B.NormAddArgs(input=by.ptr, weight=bw.ptr, bias=bb.ptr, output=bf.ptr, rows=rows, n=n, kind=kind, epsilon=1e-3)))
+        ref = P.layer_norm(t64(y), t64(w), 1e-3) if kind == 2 else P.unit_rms(t64(y), 1e-3) * t64(w)
+        close(bf.numpy(np.float32, (rows, n)), (ref + t64(b)).numpy(), 1e-5, f"kind {kind} alone")
 
 
 # ---- products ------------------------------------------------------------------------------------------------------------------------------

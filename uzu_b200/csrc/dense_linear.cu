@@ -209,10 +209,12 @@ __global__ void __launch_bounds__(256, RMAX == 1 ? 4 : 2) dense_rows_kernel(cons
             }
         }
     };
-    if (vec_ok && col_ok) request(cur, cur2, k_first);
+    const bool early = vec_ok && col_ok && !a.group_offsets;     // (most row groups of a short pass are empty: their weights are not asked for)
+    if (early) request(cur, cur2, k_first);
     pdl_wait();
     const DenseRows R = dense_rows(a, z);
     if (R.count == 0) return;                            // uniform over the CTA
+    if (vec_ok && col_ok && !early) request(cur, cur2, k_first);
     const uint32_t* map = reinterpret_cast<const uint32_t*>(a.rows_map);
     // the group's activation rows, with the A operation applied, go to shared memory once per CTA when they fit
     const bool staged = vec_ok && (size_t)R.count * a.k <= DL_STAGE_FLOATS;

@@ -166,6 +166,59 @@ __global__ void __launch_bounds__(256) norm_add_kernel(const uzu_norm_add_args a
     for (uint32_t i = threadIdx.x + KEEP * blockDim.x; i < a.n; i += blockDim.x) out[i] = norm_add_value(a.next_kind, res[i], mean2, inv2, a.next_alpha, nw, nb, i);
 }
 
+// The same for RMS and layer norms without a second norm over rows of whole float4 that a CTA holds in registers (n <= 8 * threads): 16-byte
+// requests, all of a thread's in flight at once.
+__global__ void __launch_bounds__(512) norm_add_vec_kernel(const uzu_norm_add_args a) {
+    pdl_launch_dependents();
+    __shared__ float red[32];
+    constexpr int KEEP = 2;
+    const float4 zero = make_float4(0.0f, 0.0f, 0.0f, 0.0f), one = make_float4(1.0f, 1.0f, 1.0f, 1.0f);
+    const uint32_t row = blockIdx.x, n4 = a.n / 4;
+    float4 x[KEEP], w[KEEP], b[KEEP], r[KEEP];
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+        const uint32_t i = threadIdx.x + j * blockDim.x;
+        w[j] = (a.weight && i < n4) ? reinterpret_cast<const float4*>(a.weight)[i] : one;
+        b[j] = (a.bias && i < n4) ? reinterpret_cast<const float4*>(a.bias)[i] : zero;
+    }
+    pdl_wait();
+    const float4* in = reinterpret_cast<const float4*>(reinterpret_cast<const float*>(a.input) + (size_t)row * a.in_stride);
+    float4* res = a.residual ? reinterpret_cast<float4*>(a.residual) + (size_t)row * n4 : nullptr;
+    float s = 0.0f, ss = 0.0f, mean = 0.0f;
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+        const uint32_t i = threadIdx.x + j * blockDim.x;
+        x[j] = i < n4 ? in[i] : zero;
+        r[j] = (res && i < n4) ? res[i] : zero;
+        s += (x[j].x + x[j].y) + (x[j].z + x[j].w);
+    }
+    if (a.kind == 2) mean = block_sum(s, red) / (float)a.n;
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+        if (threadIdx.x + j * blockDim.x < n4) {
+            x[j].x -= mean; x[j].y -= mean; x[j].z -= mean; x[j].w -= mean;
+            ss += (x[j].x * x[j].x + x[j].y * x[j].y) + (x[j].z * x[j].z + x[j].w * x[j].w);
+        }
+    }
+    const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)a.n + a.epsilon);
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+        const uint32_t i = threadIdx.x + j * blockDim.x;
+        if (i >= n4) continue;
+        float4 v = make_float4(x[j].x * inv * w[j].x + b[j].x, x[j].y * inv * w[j].y + b[j].y, x[j].z * inv * w[j].z + b[j].z, x[j].w * inv * w[j].w + b[j].w);
+        if (!res) {
+            reinterpret_cast<float4*>(a.output)[(size_t)row * n4 + i] = v;
+            continue;
+        }
+        v = make_float4(fmaf(a.mult, v.x, r[j].x), fmaf(a.mult, v.y, r[j].y), fmaf(a.mult, v.z, r[j].z), fmaf(a.mult, v.w, r[j].w));
+        res[i] = v;
+        if (a.residual_bf16) {
+            const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+            reinterpret_cast<uint2*>(a.output)[(size_t)row * n4 + i] = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+        }
+    }
+}
+
 // One CTA per row of a residual kept as several streams: begin from the embedding, or take a sublayer's result in; then the next reader's
 // weighted sum of the streams and its layer norm. A thread keeps up to KEEP elements of that sum in registers between the passes over it.
 template <int MAXS>
@@ -830,6 +883,9 @@ void uzu_norm_add_encode(uzu_command_buffer* cmd, const uzu_norm_add_args* a) {
     if (!b.in_stride) b.in_stride = b.n;
     if (b.kind == 1 && !b.residual_bf16 && (!b.residual || !b.output || b.next_kind == 1))
         launch(cmd, "norm_add_elementwise_kernel", norm_add_elementwise_kernel, dim3((b.n + 255) / 256, b.rows), dim3(256), 0, b);
+    else if (b.kind != 1 && (!b.residual || !b.output || b.residual_bf16) && b.n % 4 == 0 && b.n <= 4096 && b.in_stride % 4 == 0 &&
+             ((b.input | b.weight | b.bias | b.residual | b.output) & 15) == 0)
+        launch(cmd, "norm_add_kernel", norm_add_vec_kernel, dim3(b.rows), dim3(b.n <= 1024 ? 128 : b.n <= 2048 ? 256 : 512), 0, b);
     else
         launch(cmd, "norm_add_kernel", norm_add_kernel, dim3(b.rows), dim3(256), 0, b);
 }

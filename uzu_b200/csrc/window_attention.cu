@@ -197,7 +197,7 @@ __device__ __forceinline__ void window_attention_body(const uzu_window_attention
     extern __shared__ float wa_smem[];          // [WA_WARPS][vdim] partial sums, then [vdim] the head's result
     __shared__ float warp_m[WA_WARPS], warp_l[WA_WARPS];
     __shared__ uint32_t is_last;
-    __shared__ float split_f[WA_MAX_SPLITS], split_l[WA_MAX_SPLITS];
+    __shared__ float split_f[WA_MAX_SPLITS];
     const uint32_t t = blockIdx.x, h = blockIdx.y, split = blockIdx.z, splits = gridDim.z;
     const uint32_t tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const uint32_t prefix = a.dynamic_position ? *reinterpret_cast<const uint32_t*>(a.dynamic_position) : a.prefix;
@@ -337,30 +337,37 @@ __device__ __forceinline__ void window_attention_body(const uzu_window_attention
         if (!is_last) return;
         __threadfence();
         const float* parts = reinterpret_cast<const float*>(a.partials) + ((size_t)t * a.heads + h) * splits * pw;
-        for (uint32_t sp = tid; sp < splits; sp += blockDim.x) {
-            split_f[sp] = __ldcg(parts + (size_t)sp * pw);
-            split_l[sp] = __ldcg(parts + (size_t)sp * pw + 1);
+        // every warp forms the splits' factors for itself, a lane per split (and 32, 64, 96 on)
+        constexpr int PER = WA_MAX_SPLITS / 32;
+        float sm[PER], sl[PER], all_m = -INFINITY, all_l = 0.0f;
+#pragma unroll
+        for (int i = 0; i < PER; ++i) {
+            const uint32_t sp = lane + 32u * i;
+            sm[i] = sp < splits ? __ldcg(parts + (size_t)sp * pw) : -INFINITY;
+            sl[i] = sp < splits ? __ldcg(parts + (size_t)sp * pw + 1) : 0.0f;
+            all_m = fmaxf(all_m, sm[i]);
         }
+        all_m = warp_max(all_m);
+#pragma unroll
+        for (int i = 0; i < PER; ++i) {
+            const float f = sm[i] == -INFINITY ? 0.0f : expf(sm[i] - all_m);
+            all_l = fmaf(sl[i], f, all_l);
+            if (warp == 0) split_f[lane + 32u * i] = f;
+        }
+        all_l = warp_sum(all_l);
         __syncthreads();
-        float all_m = -INFINITY;
-        for (uint32_t sp = 0; sp < splits; ++sp) all_m = fmaxf(all_m, split_f[sp]);
-        __syncthreads();
-        for (uint32_t sp = tid; sp < splits; sp += blockDim.x) split_f[sp] = split_f[sp] == -INFINITY ? 0.0f : expf(split_f[sp] - all_m);
-        __syncthreads();
-        float all_l = 0.0f;
-        for (uint32_t sp = 0; sp < splits; ++sp) all_l = fmaf(split_l[sp], split_f[sp], all_l);      // in split order
         if (a.sinks) all_l += expf(sink - all_m);
         for (uint32_t c = tid; c < a.vdim; c += blockDim.x) {
             float v = 0.0f;
             uint32_t sp = 0;
-            for (; sp + 8 <= splits; sp += 8) {        // eight loads in flight, added in split order
-                float x[8];
+            constexpr int FLY = 8;
+            for (; sp < splits; sp += FLY) {           // eight loads in flight, added in split order (factors past the last split are 0)
+                float x[FLY];
 #pragma unroll
-                for (int u = 0; u < 8; ++u) x[u] = __ldcg(parts + (size_t)(sp + u) * pw + 2 + c);
+                for (int u = 0; u < FLY; ++u) x[u] = sp + u < splits ? __ldcg(parts + (size_t)(sp + u) * pw + 2 + c) : 0.0f;
 #pragma unroll
-                for (int u = 0; u < 8; ++u) v = fmaf(x[u], split_f[sp + u], v);
+                for (int u = 0; u < FLY; ++u) v = fmaf(x[u], split_f[sp + u], v);
             }
-            for (; sp < splits; ++sp) v = fmaf(__ldcg(parts + (size_t)sp * pw + 2 + c), split_f[sp], v);
             result[c] = v / all_l * gate;
         }
         if (tid == 0) *ticket = 0;
