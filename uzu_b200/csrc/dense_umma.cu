@@ -86,13 +86,18 @@ __device__ __forceinline__ uint32_t du_tile_off(uint32_t row, uint32_t ch) { ret
 enum DuEpilogue : int { DuPlain = 0 /* scale, bias, accumulate */, DuGelu = 1 /* the exact gelu besides */, DuGeneral = 2 /* gate, row and column factors besides */,
                         DuPair = 3 /* the gated unit of the tile's two halves */ };
 
+// All three units are g * sigmoid(s(g)) times something of u: (1 + tanh(y)) / 2 = sigmoid(2 y). (The fast exponential and division are good to about
+// 2^-20; a row of units is rounded to bf16 next.)
 __device__ __forceinline__ float du_unit(uint32_t kind, float g, float u, float limit, float alpha) {
+    float s = g;
     if (kind == 0) {
         g = fminf(g, limit);
-        return g * (1.0f / (1.0f + expf(-alpha * g))) * (fminf(fmaxf(u, -limit), limit) + 1.0f);
+        u = fminf(fmaxf(u, -limit), limit) + 1.0f;
+        s = alpha * g;
+    } else if (kind == 2) {
+        s = 1.5957691216057308f * (g + 0.044715f * g * g * g);
     }
-    if (kind == 1) return g * (1.0f / (1.0f + expf(-g))) * u;
-    return 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
+    return __fdividef(g, 1.0f + __expf(-s)) * u;
 }
 
 // 32 accumulator columns of this warp's 32 rows (one row per lane)

@@ -12,6 +12,7 @@ namespace uzu {
 namespace {
 
 constexpr int RC_ROWS = 64, RC_COLS = 64, RC_PAD = 8;        // tokens of a chunk, value columns of a CTA
+constexpr int RC_THREADS = 256;
 
 __device__ __forceinline__ void rc_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
     asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
@@ -39,7 +40,8 @@ __device__ __forceinline__ void rc_split(float x0, float x1, uint32_t& hi, uint3
     lo = rc_pack(x0 - __uint_as_float(hi << 16), x1 - __uint_as_float(hi & 0xffff0000u));
 }
 
-__device__ __forceinline__ float rc_input(uint32_t op, float x) { return op == 1 ? x / (1.0f + expf(-x)) : x; }
+// (the fast exponential and division are good to about 2^-20; the result is rounded to bf16 next)
+__device__ __forceinline__ float rc_input(uint32_t op, float x) { return op == 1 ? __fdividef(x, 1.0f + __expf(-x)) : x; }
 
 __device__ __forceinline__ float4 rc_input4(uint32_t op, float4 x) {
     return make_float4(rc_input(op, x.x), rc_input(op, x.y), rc_input(op, x.z), rc_input(op, x.w));
@@ -67,8 +69,8 @@ __device__ __forceinline__ void rc_stage(const float* src, size_t stride, uint32
 
 }  // namespace
 
-// (1) scratch[head, chunk] = sum_j g^(n-1-j) k_j v_j^T.  M = key channels (a warp takes 16-row tiles warp, warp + 4), N = 64 value columns, K = tokens.
-__global__ void __launch_bounds__(128) retention_chunk_sums_kernel(const uzu_retention_args a) {
+// (1) scratch[head, chunk] = sum_j g^(n-1-j) k_j v_j^T.  M = key channels (16 per warp), N = 64 value columns, K = tokens.
+__global__ void __launch_bounds__(RC_THREADS) retention_chunk_sums_kernel(const uzu_retention_args a) {
     pdl_launch_dependents();
     extern __shared__ __align__(16) unsigned char rc_raw[];
     __shared__ float power[RC_ROWS];
@@ -100,50 +102,38 @@ __global__ void __launch_bounds__(128) retention_chunk_sums_kernel(const uzu_ret
         *reinterpret_cast<uint2*>(v_s + r * ldv + c) = make_uint2(rc_pack(x.x, x.y), rc_pack(x.z, x.w));
     });
     __syncthreads();
-    float acc[2][8][4];
+    if (warp * 16 >= dim) return;
+    float acc[8][4];
 #pragma unroll
-    for (int m = 0; m < 2; ++m)
+    for (int j = 0; j < 8; ++j)
 #pragma unroll
-        for (int j = 0; j < 8; ++j)
-#pragma unroll
-            for (int c = 0; c < 4; ++c) acc[m][j][c] = 0.0f;
-    const uint32_t mtiles = dim / 16, nblocks = cols / 16;
+        for (int c = 0; c < 4; ++c) acc[j][c] = 0.0f;
+    const uint32_t nblocks = cols / 16;
 #pragma unroll
     for (int kk = 0; kk < RC_ROWS / 16; ++kk) {
         uint32_t b[4][4];
 #pragma unroll
         for (int j = 0; j < 4; ++j)
             if ((uint32_t)j < nblocks) rc_ldmatrix<true>(b[j], v_s + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * ldv + (lane >> 4) * 8 + j * 16);
+        uint32_t hi[4], lo[4];
+        const uint32_t at = (kk * 16 + (lane & 7) + (lane >> 4) * 8) * ldk + warp * 16 + ((lane >> 3) & 1) * 8;
+        rc_ldmatrix<true>(hi, k_hi + at);
+        rc_ldmatrix<true>(lo, k_lo + at);
 #pragma unroll
-        for (int m = 0; m < 2; ++m) {
-            const uint32_t tile = warp + 4 * m;
-            if (tile < mtiles) {
-                uint32_t hi[4], lo[4];
-                const uint32_t at = (kk * 16 + (lane & 7) + (lane >> 4) * 8) * ldk + tile * 16 + ((lane >> 3) & 1) * 8;
-                rc_ldmatrix<true>(hi, k_hi + at);
-                rc_ldmatrix<true>(lo, k_lo + at);
+        for (int j = 0; j < 8; ++j)
+            if ((uint32_t)j < 2 * nblocks) rc_mma(acc[j], hi, b[j >> 1][(j & 1) * 2], b[j >> 1][(j & 1) * 2 + 1]);
 #pragma unroll
-                for (int j = 0; j < 8; ++j)
-                    if ((uint32_t)j < 2 * nblocks) rc_mma(acc[m][j], hi, b[j >> 1][(j & 1) * 2], b[j >> 1][(j & 1) * 2 + 1]);
-#pragma unroll
-                for (int j = 0; j < 8; ++j)
-                    if ((uint32_t)j < 2 * nblocks) rc_mma(acc[m][j], lo, b[j >> 1][(j & 1) * 2], b[j >> 1][(j & 1) * 2 + 1]);
-            }
-        }
+        for (int j = 0; j < 8; ++j)
+            if ((uint32_t)j < 2 * nblocks) rc_mma(acc[j], lo, b[j >> 1][(j & 1) * 2], b[j >> 1][(j & 1) * 2 + 1]);
     }
     float* out = reinterpret_cast<float*>(a.chunk_scratch) + ((size_t)head * chunks + chunk) * dim * vdim + v0;
 #pragma unroll
-    for (int m = 0; m < 2; ++m) {
-        const uint32_t tile = warp + 4 * m;
-        if (tile >= mtiles) continue;
-#pragma unroll
-        for (int j = 0; j < 8; ++j)
-            if ((uint32_t)j < 2 * nblocks) {
-                float* o = out + (size_t)(tile * 16 + g) * vdim + j * 8 + t4 * 2;
-                *reinterpret_cast<float2*>(o) = make_float2(acc[m][j][0], acc[m][j][1]);
-                *reinterpret_cast<float2*>(o + (size_t)8 * vdim) = make_float2(acc[m][j][2], acc[m][j][3]);
-            }
-    }
+    for (int j = 0; j < 8; ++j)
+        if ((uint32_t)j < 2 * nblocks) {
+            float* o = out + (size_t)(warp * 16 + g) * vdim + j * 8 + t4 * 2;
+            *reinterpret_cast<float2*>(o) = make_float2(acc[j][0], acc[j][1]);
+            *reinterpret_cast<float2*>(o + (size_t)8 * vdim) = make_float2(acc[j][2], acc[j][3]);
+        }
 }
 
 // (2) four state elements per thread: the sums become the states before their chunks (hi in the upper half of a word), the last state is stored
@@ -158,7 +148,7 @@ __global__ void __launch_bounds__(256) retention_chunk_scan_kernel(const uzu_ret
     float4* state = reinterpret_cast<float4*>(a.state) + head * size4 + i;
     float4* u = reinterpret_cast<float4*>(a.chunk_scratch) + (size_t)head * chunks * size4 + i;
     float4 s = *state;
-    constexpr int AHEAD = 4;
+    constexpr int AHEAD = 8;
     float4 x[AHEAD];
 #pragma unroll
     for (int q = 0; q < AHEAD; ++q)
@@ -183,8 +173,8 @@ __global__ void __launch_bounds__(256) retention_chunk_scan_kernel(const uzu_ret
     *state = s;
 }
 
-// (3) 64 tokens x 64 value columns of one head; a warp takes 16 tokens
-__global__ void __launch_bounds__(128) retention_chunk_out_kernel(const uzu_retention_args a) {
+// (3) 64 tokens x 64 value columns of one head; a warp takes 16 tokens and half of the columns
+__global__ void __launch_bounds__(RC_THREADS, 2) retention_chunk_out_kernel(const uzu_retention_args a) {
     pdl_launch_dependents();
     extern __shared__ __align__(16) unsigned char rc_raw[];
     __shared__ float power[RC_ROWS + 1];
@@ -196,7 +186,7 @@ __global__ void __launch_bounds__(128) retention_chunk_out_kernel(const uzu_rete
     __nv_bfloat16* s_lo = s_hi + dim * ldv;
     const uint32_t chunk = blockIdx.x, head = blockIdx.y, v0 = blockIdx.z * RC_COLS, chunks = gridDim.x;
     const uint32_t t0 = chunk * RC_ROWS, n = min((uint32_t)RC_ROWS, a.rows - t0), cols = min((uint32_t)RC_COLS, vdim - v0);
-    const uint32_t tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t4 = lane & 3;
+    const uint32_t tid = threadIdx.x, lane = tid & 31, warp = (tid >> 5) & 3, part = tid >> 7, g = lane >> 2, t4 = lane & 3;
     if (tid <= RC_ROWS) power[tid] = powf(reinterpret_cast<const float*>(a.decay)[head], (float)tid);
     pdl_wait();
     auto to_bf16 = [&](__nv_bfloat16* tile, uint32_t ld) {
@@ -212,16 +202,16 @@ __global__ void __launch_bounds__(128) retention_chunk_out_kernel(const uzu_rete
         const uint32_t* src = reinterpret_cast<const uint32_t*>(a.chunk_scratch) + ((size_t)head * chunks + chunk) * dim * vdim + v0;
         const uint32_t c4 = cols / 4, total = dim * c4;
         constexpr int BATCH = 8;
-        for (uint32_t i0 = tid; i0 < total; i0 += BATCH * 128) {
+        for (uint32_t i0 = tid; i0 < total; i0 += BATCH * RC_THREADS) {
             uint4 x[BATCH];
 #pragma unroll
             for (int u = 0; u < BATCH; ++u) {
-                const uint32_t i = i0 + u * 128, r = i / c4, c = (i - r * c4) * 4;
+                const uint32_t i = i0 + u * RC_THREADS, r = i / c4, c = (i - r * c4) * 4;
                 if (i < total) x[u] = *reinterpret_cast<const uint4*>(src + (size_t)r * vdim + c);
             }
 #pragma unroll
             for (int u = 0; u < BATCH; ++u) {
-                const uint32_t i = i0 + u * 128, r = i / c4, c = (i - r * c4) * 4;
+                const uint32_t i = i0 + u * RC_THREADS, r = i / c4, c = (i - r * c4) * 4;
                 if (i < total) {
                     const uint4 w = x[u];
                     *reinterpret_cast<uint2*>(s_hi + r * ldv + c) = make_uint2((w.x >> 16) | (w.y & 0xffff0000u), (w.z >> 16) | (w.w & 0xffff0000u));
@@ -231,30 +221,32 @@ __global__ void __launch_bounds__(128) retention_chunk_out_kernel(const uzu_rete
         }
     }
     __syncthreads();
-    float o[8][4], s[8][4];
+    const uint32_t c_first = part * (RC_COLS / 2);              // this warp's columns
+    if (c_first >= cols) return;
+    float o[4][4], s[8][4];
 #pragma unroll
     for (int j = 0; j < 8; ++j)
 #pragma unroll
-        for (int c = 0; c < 4; ++c) o[j][c] = s[j][c] = 0.0f;
-    const uint32_t dk = dim / 16, nblocks = cols / 16, row_lo = warp * 16 + g;
+        for (int c = 0; c < 4; ++c) { s[j][c] = 0.0f; if (j < 4) o[j][c] = 0.0f; }
+    const uint32_t dk = dim / 16, nblocks = min((uint32_t)RC_COLS / 2, cols - c_first) / 16, row_lo = warp * 16 + g;
     // what the state before the chunk gives, and the scores of the chunk's own keys (only those up to the warp's last token)
     for (uint32_t kk = 0; kk < dk; ++kk) {
         uint32_t q[4];
         rc_ldmatrix<false>(q, q_s + (warp * 16 + (lane & 15)) * ldk + kk * 16 + (lane >> 4) * 8);
-        const uint32_t at = (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * ldv + (lane >> 4) * 8;
-        uint32_t b[4][4];
+        const uint32_t at = (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * ldv + (lane >> 4) * 8 + c_first;
+        uint32_t b[2][4], bl[2][4];
+#pragma unroll
+        for (int j = 0; j < 2; ++j)
+            if ((uint32_t)j < nblocks) {
+                rc_ldmatrix<true>(b[j], s_hi + at + j * 16);
+                rc_ldmatrix<true>(bl[j], s_lo + at + j * 16);
+            }
 #pragma unroll
         for (int j = 0; j < 4; ++j)
-            if ((uint32_t)j < nblocks) rc_ldmatrix<true>(b[j], s_hi + at + j * 16);
-#pragma unroll
-        for (int j = 0; j < 8; ++j)
             if ((uint32_t)j < 2 * nblocks) rc_mma(o[j], q, b[j >> 1][(j & 1) * 2], b[j >> 1][(j & 1) * 2 + 1]);
 #pragma unroll
         for (int j = 0; j < 4; ++j)
-            if ((uint32_t)j < nblocks) rc_ldmatrix<true>(b[j], s_lo + at + j * 16);
-#pragma unroll
-        for (int j = 0; j < 8; ++j)
-            if ((uint32_t)j < 2 * nblocks) rc_mma(o[j], q, b[j >> 1][(j & 1) * 2], b[j >> 1][(j & 1) * 2 + 1]);
+            if ((uint32_t)j < 2 * nblocks) rc_mma(o[j], q, bl[j >> 1][(j & 1) * 2], bl[j >> 1][(j & 1) * 2 + 1]);
         // keys: two tiles of 8 tokens per load: (tokens 0-7, channels 0-7), (0-7, 8-15), (8-15, 0-7), (8-15, 8-15)
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
@@ -272,7 +264,7 @@ __global__ void __launch_bounds__(128) retention_chunk_out_kernel(const uzu_rete
 #pragma unroll
         for (int c = 0; c < 4; ++c) {
             const uint32_t i = row_lo + 8 * (c >> 1), t = j * 8 + t4 * 2 + (c & 1);
-            o[j][c] *= power[i + 1];
+            if (j < 4) o[j][c] *= power[i + 1];
             s[j][c] = t <= i ? s[j][c] * (power[i - t] * key_scale) : 0.0f;
         }
 #pragma unroll
@@ -283,21 +275,21 @@ __global__ void __launch_bounds__(128) retention_chunk_out_kernel(const uzu_rete
         rc_split(s[2 * kk][2], s[2 * kk][3], ph[1], pl[1]);
         rc_split(s[2 * kk + 1][0], s[2 * kk + 1][1], ph[2], pl[2]);
         rc_split(s[2 * kk + 1][2], s[2 * kk + 1][3], ph[3], pl[3]);
-        uint32_t b[4][4];
+        uint32_t b[2][4];
+#pragma unroll
+        for (int j = 0; j < 2; ++j)
+            if ((uint32_t)j < nblocks) rc_ldmatrix<true>(b[j], v_s + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * ldv + (lane >> 4) * 8 + c_first + j * 16);
 #pragma unroll
         for (int j = 0; j < 4; ++j)
-            if ((uint32_t)j < nblocks) rc_ldmatrix<true>(b[j], v_s + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * ldv + (lane >> 4) * 8 + j * 16);
-#pragma unroll
-        for (int j = 0; j < 8; ++j)
             if ((uint32_t)j < 2 * nblocks) rc_mma(o[j], ph, b[j >> 1][(j & 1) * 2], b[j >> 1][(j & 1) * 2 + 1]);
 #pragma unroll
-        for (int j = 0; j < 8; ++j)
+        for (int j = 0; j < 4; ++j)
             if ((uint32_t)j < 2 * nblocks) rc_mma(o[j], pl, b[j >> 1][(j & 1) * 2], b[j >> 1][(j & 1) * 2 + 1]);
     }
     const float qscale = a.query_scale != 0.0f ? a.query_scale : 1.0f;
-    float* out = reinterpret_cast<float*>(a.out) + (size_t)t0 * a.out_stride + (size_t)head * vdim + v0;
+    float* out = reinterpret_cast<float*>(a.out) + (size_t)t0 * a.out_stride + (size_t)head * vdim + v0 + c_first;
 #pragma unroll
-    for (int j = 0; j < 8; ++j)
+    for (int j = 0; j < 4; ++j)
         if ((uint32_t)j < 2 * nblocks) {
 #pragma unroll
             for (int half = 0; half < 2; ++half) {
@@ -319,9 +311,9 @@ bool encode_retention_chunked(uzu_command_buffer* cmd, const uzu_retention_args&
     opt_in_dynamic_smem(cmd, retention_chunk_sums_kernel, (int)(RC_ROWS * (2 * most_k + row_v)), done[0]);
     opt_in_dynamic_smem(cmd, retention_chunk_out_kernel, (int)(RC_ROWS * (2 * most_k + row_v) + 2 * 128 * row_v), done[1]);
     const dim3 grid(chunks, a.heads, tiles);
-    launch(cmd, "retention_chunk_sums_kernel", retention_chunk_sums_kernel, grid, dim3(128), RC_ROWS * (2 * row_k + row_v), a);
+    launch(cmd, "retention_chunk_sums_kernel", retention_chunk_sums_kernel, grid, dim3(RC_THREADS), RC_ROWS * (2 * row_k + row_v), a);
     launch(cmd, "retention_chunk_scan_kernel", retention_chunk_scan_kernel, dim3((unsigned)(((size_t)a.dim * a.vdim / 4 + 255) / 256), a.heads), dim3(256), 0, a);
-    launch(cmd, "retention_chunk_out_kernel", retention_chunk_out_kernel, grid, dim3(128), RC_ROWS * (2 * row_k + row_v) + 2 * a.dim * row_v, a);
+    launch(cmd, "retention_chunk_out_kernel", retention_chunk_out_kernel, grid, dim3(RC_THREADS), RC_ROWS * (2 * row_k + row_v) + 2 * a.dim * row_v, a);
     return true;
 }
 
